@@ -4,6 +4,7 @@ from .engine_config import EngineConfig, resolve_dtype_name
 from .model_spec import LayerCall, LayerSpec, ModelSpec, PartSpec
 from .qwen2_config import ConfigError, Qwen2Config
 from .fovudra_config import FovudraConfig
+from .mekusun_config import MekusunConfig
 from .zelasun_config import ZelasunConfig
 from .zururax_config import ZururaxConfig
 from .zuzunex_config import ZuzunexConfig
@@ -24,6 +25,7 @@ __all__ = [
     "FovudraConfig",
     "LayerCall",
     "LayerSpec",
+    "MekusunConfig",
     "ModelSpec",
     "PartSpec",
     "Qwen2Config",

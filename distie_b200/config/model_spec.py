@@ -37,6 +37,7 @@ class LayerSpec:
     mixer: PartSpec
     feed_forward: PartSpec
     norms: Mapping[str, PartSpec]
+    average: str | None = None  # the tensor of a depth average behind the block (see parts/depth.py)
 
 
 @dataclass(frozen=True)
@@ -89,6 +90,18 @@ class ModelSpec:
                 raise ValueError(f"order[{index}] reads cache slot {call.cache_slot} before any call wrote it")
         if sorted(owners) != list(range(len(owners))):
             raise ValueError("cache slots must be numbered 0..n-1 without gaps")
+
+        averaged = [self.layers[call.layer].average is not None for call in self.order]
+        if any(averaged):
+            if not all(averaged):
+                raise ValueError("a depth average stands behind every layer or behind none")
+            if len({call.layer for call in self.order}) != len(self.order):
+                raise ValueError("a layer with a depth average runs once: its weights are as many as the states so far")
+
+    @property
+    def depth_averaged(self) -> bool:
+        """Whether the residual behind every layer is a weighted sum of all states so far (see parts/depth.py)."""
+        return self.layers[self.order[0].layer].average is not None
 
     @property
     def num_cache_slots(self) -> int:

@@ -1,0 +1,517 @@
+// Recurrences whose decay varies by channel and token: the selective scan (a diagonal state per channel) and the delta
+// rule with a decay and a removal rate per key channel (a matrix state per head).
+//
+// Everything is float32 up to the selective scan's gated read-out, which feeds the next product and is stored as T.
+// State is read and written through a token's seat; nothing reads host-side batch data beyond counts that a step's
+// layout fixes, so captured decode steps replay these kernels.
+#include "recurrent.cuh"
+
+namespace distie {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// 2^x on the special-function unit (results below the smallest normal number become zero).
+__device__ __forceinline__ float exp2_unit(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// ---------------------------------------------------------------------------
+// Selective scan.  Per channel c and state n, with d = softplus(dt[t, c] + dt_bias[c]):
+//   S[n, c] <- exp(d rates[n, c]) S[n, c] + d x[t, c] B[t, n]
+//   out[t, c] = (sum_n S[n, c] C[t, n] + skip[c] x[t, c]) * silu(gate[t, c])
+// State layout [seat, n, c]: neighbouring threads hold neighbouring channels.
+//
+// A channel belongs to LANES threads of one warp, each with PER of its states in registers (LANES * PER >= states; what
+// lies beyond has no input and adds nothing).  Tokens come in tiles of 16: the block makes d and d x for its channels
+// and copies B and C into shared memory, walks the tile, and finishes it element by element (skip, gate, store).
+//
+// A long prompt alone would leave most of the machine idle, since only channels run side by side.  Its portion is then
+// cut into the step's tiles of 128 tokens (`tiles`: first token and length, a request's tiles in a row), and three
+// launches replace the walk: (1) every tile but a request's last from a state of zeros, leaving its state and the sum
+// of its steps; (2) the chain over a request's tiles, S <- exp(rate * sum of steps) S + the tile's state, which turns
+// every tile's state into the one it starts from; (3) every tile from there, with output; a request's last tile leaves
+// the request's state.
+// ---------------------------------------------------------------------------
+constexpr int kSelectTile = 16, kSelectThreads = 128;
+constexpr int kSelectWalk = 0, kSelectLocal = 1, kSelectFinish = 2;
+
+struct SelectArgs {
+  const float* x;
+  int x_stride;
+  Sliced dt, B, C, gate;
+  const float *rates, *skip, *dt_bias;
+  float* state;
+  int out_stride;
+  const int *seq_bounds, *seq_seat, *token_seq, *tiles;
+  int channels, states, first_row, num_tiles;
+  float* tile_state;  // [tiles, states, channels]
+  float* tile_steps;  // [tiles, channels]
+};
+
+template <typename T, int PER, int LANES, int MODE>
+__global__ void __launch_bounds__(kSelectThreads) selective_scan_kernel(SelectArgs a, T* __restrict__ out) {
+  constexpr int CH = kSelectThreads / LANES;  // channels of the block
+  constexpr int PER_WARP = 32 / LANES;        // channels of a warp
+  constexpr int NP = PER * LANES;
+  __shared__ float d_s[kSelectTile][CH];      // the step sizes; a token's read-out takes the place of its step
+  __shared__ float dx_s[kSelectTile][CH];
+  __shared__ __align__(16) float b_s[kSelectTile][NP];
+  __shared__ __align__(16) float c_s[kSelectTile][NP];
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int local = (tid >> 5) * PER_WARP + lane % PER_WARP, part = lane / PER_WARP;
+  const int c0 = blockIdx.x * CH, c = c0 + local;
+  const bool valid = c < a.channels;
+  int first, end, row;
+  bool last = true;
+  if (MODE == kSelectWalk) {
+    row = a.first_row + blockIdx.y;
+    first = a.seq_bounds[row];
+    end = a.seq_bounds[row + 1];
+    if (end <= first) return;
+  } else {
+    const int tile = blockIdx.y;
+    first = a.tiles[2 * tile];
+    end = first + a.tiles[2 * tile + 1];
+    row = a.token_seq[first];
+    last = tile + 1 == a.num_tiles || a.token_seq[a.tiles[2 * tile + 2]] != row;
+    if (MODE == kSelectLocal && last) return;
+  }
+  const size_t plane = (size_t)a.states * a.channels;
+  float* held = MODE == kSelectWalk ? a.state + (size_t)a.seq_seat[row] * plane : a.tile_state + blockIdx.y * plane;
+  float S[PER], rate[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int n = part * PER + i;
+    const bool live = valid && n < a.states;
+    S[i] = (live && MODE != kSelectLocal) ? held[(size_t)n * a.channels + c] : 0.f;
+    rate[i] = live ? a.rates[(size_t)n * a.channels + c] * kLog2e : 0.f;
+  }
+  float steps = 0.f;
+  for (int t0 = first; t0 < end; t0 += kSelectTile) {
+    const int count = min(kSelectTile, end - t0);
+    for (int idx = tid; idx < count * CH; idx += kSelectThreads) {
+      const int tok = idx / CH, ch = idx % CH;
+      float d = 0.f, dx = 0.f;
+      if (c0 + ch < a.channels) {
+        d = softplus_f(a.dt.at(t0 + tok, c0 + ch) + a.dt_bias[c0 + ch]);
+        dx = d * a.x[(size_t)(t0 + tok) * a.x_stride + c0 + ch];
+      }
+      d_s[tok][ch] = d;
+      dx_s[tok][ch] = dx;
+    }
+    for (int idx = tid; idx < count * NP; idx += kSelectThreads) {
+      const int tok = idx / NP, n = idx % NP;
+      const bool live = n < a.states;
+      b_s[tok][n] = live ? a.B.at(t0 + tok, n) : 0.f;
+      if (MODE != kSelectLocal) c_s[tok][n] = live ? a.C.at(t0 + tok, n) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 4
+    for (int tok = 0; tok < count; ++tok) {
+      const float d = d_s[tok][local], dx = dx_s[tok][local];
+      float y = 0.f;
+#pragma unroll
+      for (int q = 0; q < PER / 4; ++q) {
+        const float4 b = *reinterpret_cast<const float4*>(&b_s[tok][part * PER + 4 * q]);
+        const float bb[4] = {b.x, b.y, b.z, b.w};
+        float cc[4] = {0.f, 0.f, 0.f, 0.f};
+        if (MODE != kSelectLocal) {
+          const float4 v = *reinterpret_cast<const float4*>(&c_s[tok][part * PER + 4 * q]);
+          cc[0] = v.x; cc[1] = v.y; cc[2] = v.z; cc[3] = v.w;
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          float& s = S[4 * q + i];
+          s = exp2_unit(d * rate[4 * q + i]) * s + dx * bb[i];
+          if (MODE != kSelectLocal) y += s * cc[i];
+        }
+      }
+      if (MODE == kSelectLocal) {
+        steps += d;
+      } else {
+#pragma unroll
+        for (int offset = PER_WARP; offset < 32; offset <<= 1) y += __shfl_xor_sync(0xffffffffu, y, offset);
+        if (part == 0) d_s[tok][local] = y;  // (the channel's other threads have read the step: they took part in the sum)
+      }
+    }
+    __syncthreads();
+    if (MODE != kSelectLocal) {
+      for (int idx = tid; idx < count * CH; idx += kSelectThreads) {  // (the same thread fills this place with the next tile)
+        const int tok = idx / CH, ch = idx % CH;
+        if (c0 + ch >= a.channels) continue;
+        const size_t t = t0 + tok;
+        const float y = d_s[tok][ch] + a.skip[c0 + ch] * a.x[t * a.x_stride + c0 + ch];
+        out[t * a.out_stride + c0 + ch] = from_float<T>(y * silu_f(a.gate.at(t, c0 + ch)));
+      }
+    }
+  }
+  if (!valid) return;
+  if (MODE == kSelectFinish) {
+    if (!last) return;
+    held = a.state + (size_t)a.seq_seat[row] * plane;
+  }
+  if (MODE == kSelectLocal && part == 0) a.tile_steps[(size_t)blockIdx.y * a.channels + c] = steps;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int n = part * PER + i;
+    if (n < a.states) held[(size_t)n * a.channels + c] = S[i];
+  }
+}
+
+// The chain over the tiles of each request, a thread per (state, channel).
+__global__ void __launch_bounds__(256) selective_chain_kernel(SelectArgs a) {
+  const size_t plane = (size_t)a.states * a.channels;
+  const size_t at = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (at >= plane) return;
+  const int c = (int)(at % a.channels);
+  const float rate = a.rates[at] * kLog2e;
+  float S = 0.f;
+  int row = -1;
+#pragma unroll 4
+  for (int tile = 0; tile < a.num_tiles; ++tile) {
+    const int mine = a.token_seq[a.tiles[2 * tile]];
+    const float left = a.tile_state[tile * plane + at];  // (of a request's last tile: not made, and not used)
+    const float keep = exp2_unit(rate * a.tile_steps[(size_t)tile * a.channels + c]);
+    if (mine != row) S = a.state[(size_t)a.seq_seat[mine] * plane + at];
+    row = mine;
+    a.tile_state[tile * plane + at] = S;
+    S = keep * S + left;
+  }
+}
+
+template <typename T, int PER, int LANES>
+static cudaError_t launch_select(const SelectArgs& a, T* out, int rows, bool tiled, cudaStream_t stream) {
+  const unsigned blocks = (unsigned)((a.channels + kSelectThreads / LANES - 1) / (kSelectThreads / LANES));
+  if (rows > 0) selective_scan_kernel<T, PER, LANES, kSelectWalk><<<dim3(blocks, rows), kSelectThreads, 0, stream>>>(a, out);
+  if (tiled) {
+    const dim3 grid(blocks, a.num_tiles);
+    selective_scan_kernel<T, PER, LANES, kSelectLocal><<<grid, kSelectThreads, 0, stream>>>(a, out);
+    const size_t plane = (size_t)a.states * a.channels;
+    selective_chain_kernel<<<(unsigned)((plane + 255) / 256), 256, 0, stream>>>(a);
+    selective_scan_kernel<T, PER, LANES, kSelectFinish><<<grid, kSelectThreads, 0, stream>>>(a, out);
+  }
+  return cudaGetLastError();
+}
+
+// Threads per channel: few where many tokens are walked (fewer loads and sums per token), more in steps of single tokens.
+template <typename T>
+static cudaError_t dispatch_select(const SelectArgs& a, T* out, int rows, bool tiled, int lanes, cudaStream_t stream) {
+  if (a.states <= 16) {
+    if (lanes == 1) return launch_select<T, 16, 1>(a, out, rows, tiled, stream);
+    if (lanes == 4) return launch_select<T, 4, 4>(a, out, rows, tiled, stream);
+    return launch_select<T, 8, 2>(a, out, rows, tiled, stream);
+  }
+  if (a.states <= 32) {
+    if (lanes >= 4) return launch_select<T, 8, 4>(a, out, rows, tiled, stream);
+    return launch_select<T, 16, 2>(a, out, rows, tiled, stream);
+  }
+  if (a.states <= 64) return launch_select<T, 16, 4>(a, out, rows, tiled, stream);
+  if (a.states <= 128) return launch_select<T, 16, 8>(a, out, rows, tiled, stream);
+  return launch_select<T, 16, 16>(a, out, rows, tiled, stream);
+}
+
+// ---------------------------------------------------------------------------
+// Delta rule with a decay w and a removal rate a per key channel.  Per head, with the unit key u = k / |k| (1e-6 under
+// the root), S [key, value]:
+//   S <- diag(w) S - (a * u) (u^T S) + k v^T   (the old S on the right);   o = S^T r
+// Element by element, with g = (k^T S) / (|k|^2 + 1e-6) per column:  S_i <- w_i S_i + k_i (v - a_i g), and the read-out
+// is taken from the state before the write:  o = sum_i r_i w_i S_i + v (r . k) - g (sum_i r_i a_i k_i), so both sums over
+// the state run side by side.
+//
+// Two kernels.  The first is parallel over tokens and leaves, per token and head, the rows k, w, a, r * w and v and the
+// numbers 1 / (|k|^2 + 1e-6), r . k and sum r a k.  The second walks the tokens: the columns of S (one per value
+// element) never meet, so COLS of them belong to a group of LANES threads that share their key channels (lane l holds
+// channels 4 l + 4 LANES q + e), a block of 64 threads owns 64 / LANES groups of one head of one request.  Tiles of
+// tokens come into shared memory by cp.async a tile ahead of the walk.
+// State layout: [seat, head, value element, key channel].
+// ---------------------------------------------------------------------------
+constexpr int kDeltaThreads = 64;
+constexpr float kDecayFactor = 0.6065306597126334f;  // exp(-1/2)
+
+struct DeltaArgs {
+  Sliced proj, decay;  // proj: [r | k | v | rate]
+  const float *decay_bias, *rate_bias;
+  float *rows, *numbers;  // [tokens, heads, 5, dim]; [tokens, heads, 4]
+  float* state;
+  float* out;
+  const int *seq_bounds, *seq_seat;
+  int tokens, heads, dim;
+};
+
+__global__ void __launch_bounds__(128) channel_delta_prepare_kernel(DeltaArgs a) {
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int n = a.heads * a.dim;
+  for (int head = blockIdx.y * 4 + warp; head < a.heads; head += gridDim.y * 4) {
+    float* rows = a.rows + ((size_t)t * a.heads + head) * 5 * a.dim;
+    float kk = 0.f, rk = 0.f, rak = 0.f;
+    for (int i = lane; i < a.dim; i += 32) {
+      const int col = head * a.dim + i;
+      const float r = a.proj.at(t, col), k = a.proj.at(t, n + col), v = a.proj.at(t, 2 * n + col);
+      const float rate = sigmoid_f(a.proj.at(t, 3 * n + col) + a.rate_bias[col]);
+      const float w = expf(-kDecayFactor * sigmoid_f(a.decay.at(t, col) + a.decay_bias[col]));
+      rows[i] = k;
+      rows[a.dim + i] = w;
+      rows[2 * a.dim + i] = rate;
+      rows[3 * a.dim + i] = r * w;
+      rows[4 * a.dim + i] = v;
+      kk += k * k;
+      rk += r * k;
+      rak += r * rate * k;
+    }
+    kk = warp_sum(kk);
+    rk = warp_sum(rk);
+    rak = warp_sum(rak);
+    if (lane == 0)
+      *reinterpret_cast<float4*>(a.numbers + ((size_t)t * a.heads + head) * 4) = make_float4(1.f / (kk + 1e-6f), rk, rak, 0.f);
+  }
+}
+
+template <int KD, int TILE, int CB>
+struct DeltaStage {
+  float rows[4][TILE][KD];  // k, w, a, r * w; zeros beyond dim
+  float v[TILE][CB];
+  float numbers[TILE][4];
+};
+
+template <int KD, int LANES, int COLS, int TILE, bool VEC>
+__global__ void __launch_bounds__(kDeltaThreads) channel_delta_kernel(DeltaArgs a) {
+  constexpr int PER = KD / LANES, CB = kDeltaThreads / LANES * COLS;
+  static_assert(PER >= 4 && PER % 4 == 0, "a thread holds whole float4s of its columns");
+  extern __shared__ __align__(16) unsigned char delta_smem[];
+  using Stage = DeltaStage<KD, TILE, CB>;
+  Stage* stages = reinterpret_cast<Stage*>(delta_smem);  // two
+  const int row = blockIdx.x, head = blockIdx.y;
+  const int tid = threadIdx.x, sub = tid % LANES, group = tid / LANES;
+  const int j0 = blockIdx.z * CB + group * COLS;
+  const int first = a.seq_bounds[row], end = a.seq_bounds[row + 1];
+  if (end <= first) return;
+
+  auto stage_tile = [&](int tile, Stage& st) {
+    const int count = min(TILE, end - tile);
+    const float* src = a.rows + ((size_t)tile * a.heads + head) * 5 * a.dim;
+    const size_t token_stride = (size_t)a.heads * 5 * a.dim;
+    if (VEC) {
+      for (int idx = tid; idx < count * 4 * (KD / 4); idx += kDeltaThreads) {
+        const int i = (idx % (KD / 4)) * 4, which = (idx / (KD / 4)) % 4, tok = idx / KD;
+        const bool live = i < a.dim;
+        cp_async_f4(&st.rows[which][tok][i], src + tok * token_stride + (size_t)which * a.dim + (live ? i : 0), live);
+      }
+    } else {
+      for (int idx = tid; idx < count * 4 * KD; idx += kDeltaThreads) {
+        const int i = idx % KD, which = (idx / KD) % 4, tok = idx / (4 * KD);
+        const bool live = i < a.dim;
+        cp_async_f1(&st.rows[which][tok][i], src + tok * token_stride + (size_t)which * a.dim + (live ? i : 0), live);
+      }
+    }
+    for (int idx = tid; idx < count * CB; idx += kDeltaThreads) {
+      const int tok = idx / CB, cj = blockIdx.z * CB + idx % CB;
+      const bool live = cj < a.dim;
+      cp_async_f1(&st.v[tok][idx % CB], src + tok * token_stride + 4 * (size_t)a.dim + (live ? cj : 0), live);
+    }
+    if (tid < count) cp_async_f4(st.numbers[tid], a.numbers + ((size_t)(tile + tid) * a.heads + head) * 4, true);
+    cp_async_commit();
+  };
+
+  stage_tile(first, stages[0]);
+  float* held = a.state + ((size_t)a.seq_seat[row] * a.heads + head) * a.dim * a.dim;
+  float S[COLS][PER];
+#pragma unroll
+  for (int col = 0; col < COLS; ++col)
+#pragma unroll
+    for (int q = 0; q < PER / 4; ++q) {
+      const int i = 4 * sub + 4 * LANES * q;
+      const bool live = j0 + col < a.dim;
+      if (VEC) {
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (live && i < a.dim) s = *reinterpret_cast<const float4*>(held + (size_t)(j0 + col) * a.dim + i);
+        S[col][4 * q] = s.x; S[col][4 * q + 1] = s.y; S[col][4 * q + 2] = s.z; S[col][4 * q + 3] = s.w;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[col][4 * q + e] = (live && i + e < a.dim) ? held[(size_t)(j0 + col) * a.dim + i + e] : 0.f;
+      }
+    }
+
+  int buffer = 0;
+  for (int tile = first; tile < end; tile += TILE, buffer ^= 1) {
+    const int count = min(TILE, end - tile);
+    const bool more = tile + TILE < end;
+    if (more) stage_tile(tile + TILE, stages[buffer ^ 1]);  // its last readers passed the barrier below
+    if (more) cp_async_wait<1>(); else cp_async_wait<0>();
+    __syncthreads();
+    const Stage& st = stages[buffer];
+#pragma unroll 2
+    for (int tok = 0; tok < count; ++tok) {
+      const float4 numbers = *reinterpret_cast<const float4*>(st.numbers[tok]);
+      float k[PER], rw[PER];
+#pragma unroll
+      for (int q = 0; q < PER / 4; ++q) {
+        const float4 kv = *reinterpret_cast<const float4*>(&st.rows[0][tok][4 * sub + 4 * LANES * q]);
+        const float4 rv = *reinterpret_cast<const float4*>(&st.rows[3][tok][4 * sub + 4 * LANES * q]);
+        k[4 * q] = kv.x; k[4 * q + 1] = kv.y; k[4 * q + 2] = kv.z; k[4 * q + 3] = kv.w;
+        rw[4 * q] = rv.x; rw[4 * q + 1] = rv.y; rw[4 * q + 2] = rv.z; rw[4 * q + 3] = rv.w;
+      }
+      float sum_k[COLS], sum_r[COLS];
+#pragma unroll
+      for (int col = 0; col < COLS; ++col) {
+        float dk[2] = {0.f, 0.f}, dr[2] = {0.f, 0.f};
+#pragma unroll
+        for (int e = 0; e < PER; ++e) {
+          dk[e & 1] += k[e] * S[col][e];
+          dr[e & 1] += rw[e] * S[col][e];
+        }
+        sum_k[col] = dk[0] + dk[1];
+        sum_r[col] = dr[0] + dr[1];
+      }
+#pragma unroll
+      for (int offset = 1; offset < LANES; offset <<= 1)
+#pragma unroll
+        for (int col = 0; col < COLS; ++col) {
+          sum_k[col] += __shfl_xor_sync(0xffffffffu, sum_k[col], offset);
+          sum_r[col] += __shfl_xor_sync(0xffffffffu, sum_r[col], offset);
+        }
+      float g[COLS], v[COLS];
+#pragma unroll
+      for (int col = 0; col < COLS; ++col) {
+        g[col] = numbers.x * sum_k[col];
+        v[col] = st.v[tok][group * COLS + col];
+        if (sub == col && j0 + col < a.dim)
+          a.out[((size_t)(tile + tok) * a.heads + head) * a.dim + j0 + col] = sum_r[col] + v[col] * numbers.y - g[col] * numbers.z;
+      }
+#pragma unroll
+      for (int q = 0; q < PER / 4; ++q) {
+        const float4 wv = *reinterpret_cast<const float4*>(&st.rows[1][tok][4 * sub + 4 * LANES * q]);
+        const float4 av = *reinterpret_cast<const float4*>(&st.rows[2][tok][4 * sub + 4 * LANES * q]);
+        const float w[4] = {wv.x, wv.y, wv.z, wv.w}, rate[4] = {av.x, av.y, av.z, av.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int col = 0; col < COLS; ++col)
+            S[col][4 * q + e] = w[e] * S[col][4 * q + e] + k[4 * q + e] * (v[col] - rate[e] * g[col]);
+      }
+    }
+    __syncthreads();  // everyone is done with this stage before the copies of the tile after next land in it
+  }
+#pragma unroll
+  for (int col = 0; col < COLS; ++col) {
+    if (j0 + col >= a.dim) continue;
+#pragma unroll
+    for (int q = 0; q < PER / 4; ++q)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = 4 * sub + 4 * LANES * q + e;
+        if (i < a.dim) held[(size_t)(j0 + col) * a.dim + i] = S[col][4 * q + e];
+      }
+  }
+}
+
+template <int KD, int LANES, int COLS>
+static cudaError_t launch_delta(const DeltaArgs& a, int num_seqs, bool vec, cudaStream_t stream) {
+  constexpr int TILE = KD >= 128 ? 8 : 16;
+  constexpr int CB = kDeltaThreads / LANES * COLS;
+  const dim3 grid(num_seqs, a.heads, (a.dim + CB - 1) / CB);
+  const size_t shared = 2 * sizeof(DeltaStage<KD, TILE, CB>);
+  auto run = [&](auto kernel) {
+    if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+    kernel<<<grid, kDeltaThreads, shared, stream>>>(a);
+  };
+  if (vec) run(channel_delta_kernel<KD, LANES, COLS, TILE, true>);
+  else run(channel_delta_kernel<KD, LANES, COLS, TILE, false>);
+  return cudaGetLastError();
+}
+
+// shape = 16 * lanes + columns of a thread; sizes a head has no room for fall back to the smallest.
+template <int KD>
+static cudaError_t dispatch_delta(const DeltaArgs& a, int num_seqs, bool vec, int lanes, int cols, cudaStream_t stream) {
+  if constexpr (KD >= 128) {
+    if (lanes == 32 && cols == 1) return launch_delta<KD, 32, 1>(a, num_seqs, vec, stream);
+    if (lanes == 32 && cols == 2) return launch_delta<KD, 32, 2>(a, num_seqs, vec, stream);
+    if (lanes == 32) return launch_delta<KD, 32, 4>(a, num_seqs, vec, stream);
+  }
+  if constexpr (KD >= 64) {
+    if (lanes >= 16 && cols == 1) return launch_delta<KD, 16, 1>(a, num_seqs, vec, stream);
+    if (lanes >= 16) return launch_delta<KD, 16, 2>(a, num_seqs, vec, stream);
+  }
+  if (cols >= 2) return launch_delta<KD, 8, 2>(a, num_seqs, vec, stream);
+  return launch_delta<KD, 8, 1>(a, num_seqs, vec, stream);
+}
+
+}  // namespace distie
+
+using namespace distie;
+
+// Floats of scratch for a step whose multi-token entries fill `num_tiles` tiles (0 tiles: none).
+extern "C" long long distie_selective_scan_scratch_floats(int num_tiles, int states, int channels) {
+  return (long long)num_tiles * channels * (states + 1);
+}
+
+// x [tokens, channels]; dt, gate [tokens, channels]; B, C [tokens, states], views of one projection (the same slices).
+// Rows first_row .. first_row + rows - 1 of the batch are walked token by token; with num_tiles > 0 the tiles in `tiles`
+// (int32 pairs: first token, length) take the three-launch form, with `scratch` from the function above.
+extern "C" int distie_selective_scan(const float* x, int x_stride, const float* dt, int dt_stride, int dt_splits,
+                                     long long dt_split_stride, const float* b, const float* c, int bc_stride,
+                                     int bc_splits, long long bc_split_stride, const float* gate, int gate_stride,
+                                     int gate_splits, long long gate_split_stride, const float* rates, const float* skip,
+                                     const float* dt_bias, float* state, void* out, int out_stride, const int* seq_bounds,
+                                     const int* seq_seat, const int* token_seq, const int* tiles, int num_tiles,
+                                     float* scratch, int first_row, int rows, int channels, int states, int lanes,
+                                     int dtype, cudaStream_t stream) {
+  if (rows <= 0 && num_tiles <= 0) return 0;
+  if (channels < 1 || states < 1 || dt_splits < 1 || bc_splits < 1 || gate_splits < 1 || rows < 0 || first_row < 0 || num_tiles < 0 ||
+      rows > 65535 || num_tiles > 65535 || (num_tiles > 0 && (!tiles || !scratch || !token_seq)))
+    return DISTIE_ERR_ARG;
+  if (states > 256) return DISTIE_ERR_UNSUPPORTED;
+  SelectArgs a;
+  a.x = x; a.x_stride = x_stride;
+  a.dt = Sliced{dt, dt_stride, dt_splits, dt_split_stride};
+  a.B = Sliced{b, bc_stride, bc_splits, bc_split_stride};
+  a.C = Sliced{c, bc_stride, bc_splits, bc_split_stride};
+  a.gate = Sliced{gate, gate_stride, gate_splits, gate_split_stride};
+  a.rates = rates; a.skip = skip; a.dt_bias = dt_bias; a.state = state; a.out_stride = out_stride;
+  a.seq_bounds = seq_bounds; a.seq_seat = seq_seat; a.token_seq = token_seq; a.tiles = tiles;
+  a.channels = channels; a.states = states; a.first_row = first_row; a.num_tiles = num_tiles;
+  a.tile_state = scratch;
+  a.tile_steps = scratch ? scratch + (size_t)num_tiles * states * channels : nullptr;
+  cudaError_t err;
+  if (dtype == DISTIE_BF16) err = dispatch_select(a, (__nv_bfloat16*)out, rows, num_tiles > 0, lanes, stream);
+  else if (dtype == DISTIE_F32) err = dispatch_select(a, (float*)out, rows, num_tiles > 0, lanes, stream);
+  else return DISTIE_ERR_UNSUPPORTED;
+  return err == cudaSuccess ? 0 : (int)err;
+}
+
+// Floats of scratch of the delta rule below.
+extern "C" long long distie_channel_delta_scratch_floats(int tokens, int heads, int dim) {
+  return (long long)tokens * heads * (5LL * dim + 4);
+}
+
+// proj [tokens, 4 heads dim (+ more)] = [r | k | v | rate], decay [tokens, heads dim] (each a matrix or slices); out
+// [tokens, heads dim]; scratch 16-byte aligned.  lanes: threads that share a column (8, 16, 32), cols: columns of a thread.
+extern "C" int distie_channel_delta(const float* proj, int proj_stride, int proj_splits, long long proj_split_stride,
+                                    const float* decay, int decay_stride, int decay_splits, long long decay_split_stride,
+                                    const float* decay_bias, const float* rate_bias, float* state, float* out,
+                                    float* scratch, const int* seq_bounds, const int* seq_seat, int tokens, int num_seqs,
+                                    int heads, int dim, int lanes, int cols, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (heads < 1 || heads > 65535 || dim < 1 || num_seqs < 1 || proj_splits < 1 || decay_splits < 1 || !scratch || !state ||
+      ((uintptr_t)scratch & 15))
+    return DISTIE_ERR_ARG;
+  if (dim > 256) return DISTIE_ERR_UNSUPPORTED;
+  DeltaArgs a;
+  a.proj = Sliced{proj, proj_stride, proj_splits, proj_split_stride};
+  a.decay = Sliced{decay, decay_stride, decay_splits, decay_split_stride};
+  a.decay_bias = decay_bias; a.rate_bias = rate_bias;
+  a.numbers = scratch;  // first: its rows of four floats stay aligned whatever dim is
+  a.rows = scratch + (size_t)tokens * heads * 4;
+  a.state = state; a.out = out; a.seq_bounds = seq_bounds; a.seq_seat = seq_seat;
+  a.tokens = tokens; a.heads = heads; a.dim = dim;
+  channel_delta_prepare_kernel<<<dim3(tokens, tokens < 512 ? (heads + 3) / 4 : 1), 128, 0, stream>>>(a);
+  DISTIE_LAUNCH_CHECK();
+  const bool vec = dim % 4 == 0 && ((uintptr_t)state & 15) == 0;
+  cudaError_t err;
+  if (dim <= 32) err = dispatch_delta<32>(a, num_seqs, vec, lanes, cols, stream);
+  else if (dim <= 64) err = dispatch_delta<64>(a, num_seqs, vec, lanes, cols, stream);
+  else if (dim <= 128) err = dispatch_delta<128>(a, num_seqs, vec, lanes, cols, stream);
+  else err = dispatch_delta<256>(a, num_seqs, vec, lanes, cols, stream);
+  return err == cudaSuccess ? 0 : (int)err;
+}

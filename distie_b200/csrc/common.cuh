@@ -63,6 +63,24 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int window, i
 // A cap on a score: cap * tanh(s / cap) with cap > 0; cap <= 0 leaves the score as it is.
 __device__ __forceinline__ float cap_score(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 
+// Activations of ungated hidden layers, by code: 1 the square of ReLU; 2 the exact GELU, z (1 + erf(z / sqrt 2)) / 2;
+// 3 xIELU with factors a and b: a z^2 + z / 2 right of zero, b (exp(z) - 1 - z) + z / 2 left of it.
+#define DISTIE_ACT_RELU2 1
+#define DISTIE_ACT_GELU 2
+#define DISTIE_ACT_XIELU 3
+struct HiddenAct {
+  int kind;
+  float a, b;
+};
+__device__ __forceinline__ float hidden_act(float z, HiddenAct act) {
+  if (act.kind == DISTIE_ACT_RELU2) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  }
+  if (act.kind == DISTIE_ACT_GELU) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+  return z > 0.f ? act.a * z * z + 0.5f * z : act.b * (expm1f(z) - z) + 0.5f * z;
+}
+
 // A sink in a softmax: one more term exp(sink) in the denominator that has no value.  Given the running maximum `m`
 // and sum `l` over the keys (sum of exp(s - m)), returns the factor the mix (sum of exp(s - m) v) is multiplied by:
 // 1 / (l + exp(sink - m)), evaluated around the larger of m and sink so that neither exponential overflows.

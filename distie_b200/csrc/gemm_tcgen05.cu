@@ -33,6 +33,7 @@ constexpr int kGemmWideThreads = 320;  // the tile kernels: producer, MMA issuer
 constexpr int GEMM_EPI_BF16 = 0;
 constexpr int GEMM_EPI_F32 = 1;
 constexpr int GEMM_EPI_SWIGLU = 2;
+constexpr int GEMM_EPI_ACT = 4;  // bfloat16 behind an activation (HiddenAct)
 constexpr int GEMM_EPI_QKV = 3;  // bias, rotation and the write of q, k and v (store_qkv_rope); tiles of 256 columns
 
 template <int BN, int STAGES>
@@ -92,7 +93,8 @@ constexpr int kEpilogueStageBytes = 32 * 32 * 4;  // per epilogue warp
 template <int BN, int EPI>
 __device__ __forceinline__ void store_accumulator(uint32_t lane_base, int row0, int lane, int n0,
                                                   void* __restrict__ out, int ldo, int M, int N, int inter, int part,
-                                                  unsigned char* stage, float limit = 0.f) {
+                                                  unsigned char* stage, float limit = 0.f,
+                                                  HiddenAct act = HiddenAct{0, 0.f, 0.f}) {
   const int rows_valid = M - row0;
   if (EPI == GEMM_EPI_SWIGLU) {
     constexpr int HALF = BN / 2;
@@ -129,7 +131,10 @@ __device__ __forceinline__ void store_accumulator(uint32_t lane_base, int row0, 
       uint32_t(&acc)[32] = whole[i];
       float v[32];
 #pragma unroll
-      for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(acc[j]);
+      for (int j = 0; j < 32; ++j) {
+        v[j] = __uint_as_float(acc[j]);
+        if (EPI == GEMM_EPI_ACT) v[j] = hidden_act(v[j], act);
+      }
       const int col = n0 + c0;
       if (rows_valid > 0 && col < N) {
         if (EPI == GEMM_EPI_F32) {
@@ -175,6 +180,7 @@ struct QkvEpilogue {
   __nv_bfloat16* k_cache;
   __nv_bfloat16* v_cache;
   int num_heads, num_kv_heads, head_dim, page_size;
+  HiddenAct act;         // GEMM_EPI_ACT only: the activation of the plain epilogue
 };
 
 // The epilogue of the q/k/v projection of prompt portions: bias, rotation of q and k (pairs (j, j + head_dim / 2),
@@ -412,7 +418,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         if (qkv.head_dim == 128) store_qkv_rope<128>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
         else store_qkv_rope<64>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
       } else {
-        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage);
+        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage, 0.f,
+                                   qkv.act);
       }
       // This warp has read its part of the accumulator: hand the buffer back to the MMA issuer.
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -436,7 +443,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 // each), and a list made on the device names the row tiles: (group, first row, rows <= 128) for tile
 // 0 .. *num_m_tiles - 1 (at most `max_m_tiles`).  A tile's box of 128 rows of A may reach into the next group's
 // rows: those rows of the accumulator are not stored.  EPI is GEMM_EPI_SWIGLU (B of a group is [2 inter, K],
-// out[row, inter] bfloat16) or GEMM_EPI_F32 (out[row, N] float32).  Every role skips the tiles past the list's end
+// out[row, inter] bfloat16), GEMM_EPI_ACT (out[row, N] bfloat16 behind an activation) or GEMM_EPI_F32 (out[row, N] float32).  Every role skips the tiles past the list's end
 // alike, so the rings stay in step.  Launched the ordinary way: the list comes from the kernel before this one.
 // ---------------------------------------------------------------------------------------------------------------
 struct GroupedTiles {
@@ -452,7 +459,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(kGemmWideThreads, 1)
 gemm_tcgen05_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                             void* __restrict__ out, int ldo, int N, int K, int inter, int num_tiles,
-                            const GroupedTiles tiles, float limit, int* __restrict__ error) {
+                            const GroupedTiles tiles, float limit, HiddenAct act, int* __restrict__ error) {
   extern __shared__ unsigned char raw[];
   auto& sm = *reinterpret_cast<GemmShared<BN, STAGES>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
   constexpr uint32_t TMEM_COLS = 512;
@@ -553,7 +560,7 @@ gemm_tcgen05_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __g
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t lane_base = tmem + buffer * ACC_STRIDE + ((uint32_t)(quadrant * 32) << 16);
       // (rows of the box past the group's own are not stored: the output ends at row m0 + rows for this tile)
-      store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, m0 + rows, N, inter, part, epilogue_stage, limit);
+      store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, m0 + rows, N, inter, part, epilogue_stage, limit, act);
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
       if (lane == 0) mbar_arrive(&sm.accum_empty[buffer]);
@@ -739,7 +746,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
         if (qkv.head_dim == 128) store_qkv_rope<128>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
         else store_qkv_rope<64>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
       } else {
-        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage);
+        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage, 0.f,
+                                   qkv.act);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
@@ -781,6 +789,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
 constexpr int SKINNY_EPI_SLICE = 0;
 constexpr int SKINNY_EPI_STORE = 1;
 constexpr int SKINNY_EPI_SWIGLU = 2;
+constexpr int SKINNY_EPI_ACT = 3;  // EPI_STORE without a bias and with an activation (HiddenAct)
 
 template <int BN, int STAGES>
 struct SkinnyShared {
@@ -798,7 +807,7 @@ template <int BN, int STAGES, int EPI, typename OutT>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tcgen05_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                            const float* __restrict__ bias, OutT* __restrict__ out, int ldo, int M, int N, int K,
-                           int inter, int* __restrict__ error) {
+                           int inter, HiddenAct act, int* __restrict__ error) {
   extern __shared__ unsigned char raw[];
   auto& sm = *reinterpret_cast<SkinnyShared<BN, STAGES>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
   constexpr uint32_t TMEM_COLS = BN < 32 ? 32 : BN;
@@ -944,7 +953,7 @@ gemm_tcgen05_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
         OutT* dst = out + (EPI == SKINNY_EPI_SLICE ? (size_t)split * M * ldo : 0) + row;
 #pragma unroll
         for (int j = 0; j < 16; ++j)
-          if (c0 + j < M) dst[(size_t)(c0 + j) * ldo] = from_float<OutT>(acc[j] + b);
+          if (c0 + j < M) dst[(size_t)(c0 + j) * ldo] = from_float<OutT>(EPI == SKINNY_EPI_ACT ? hidden_act(acc[j], act) : acc[j] + b);
       }
     }
   }
@@ -1053,17 +1062,31 @@ static int pick_tile_width(int M, int N, int tile_rows, int slots) {
 
 using namespace distie;
 
+extern "C" int distie_gemm_tcgen05_act(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
+                                       int epi, int tile_width, int kind, float a, float b, int sm_count, int* error,
+                                       cudaStream_t stream);
+
 // out = x[M, K] w[N, K]^T.  epi 0: bfloat16 [M, N]; 1: float32 [M, N]; 2: w is [2 * inter, K] and
 // out[M, inter] = silu(x Wg^T) * (x Wu^T) in bfloat16 (N = 2 * inter).  x and w are bfloat16 with row
 // strides ldx and K; K must be a multiple of 8 and the pointers 16-byte aligned.
 // `tile_width` 128, 192 or 256 picks the width of the output tiles; 0 leaves the choice to the kernel.
 extern "C" int distie_gemm_tcgen05(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
                                    int epi, int tile_width, int sm_count, int* error, cudaStream_t stream) {
+  return distie_gemm_tcgen05_act(x, ldx, w, out, ldo, M, N, K, epi, tile_width, 0, 0.f, 0.f, sm_count, error, stream);
+}
+
+// The same; epi 4: out[M, N] bfloat16 = act(x w^T) with the activation of code `kind` and its factors a and b.
+extern "C" int distie_gemm_tcgen05_act(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
+                                       int epi, int tile_width, int kind, float a, float b, int sm_count, int* error,
+                                       cudaStream_t stream) {
   if (M <= 0) return 0;
   if (N < 1 || K < 8 || (K & 7) || (ldx & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return DISTIE_ERR_UNSUPPORTED;
   if (epi == GEMM_EPI_SWIGLU && (N & 1)) return DISTIE_ERR_ARG;
+  if (epi == GEMM_EPI_ACT && (kind < DISTIE_ACT_RELU2 || kind > DISTIE_ACT_XIELU)) return DISTIE_ERR_ARG;
   if (sm_count < 1) sm_count = 148;
+  QkvEpilogue more = QkvEpilogue();
+  more.act = HiddenAct{kind, a, b};
   CUtensorMap map_a, map_b;
   int status = make_map(&map_a, x, M, K, ldx, kGemmBM);
   if (status != 0) return status;
@@ -1073,12 +1096,14 @@ extern "C" int distie_gemm_tcgen05(const void* x, int ldx, const void* w, void* 
       if ((status = make_map(&map_b, w, N, K, K, 128)) != 0) return status;
       return launch_gemm_pair<256, 6, 1, GEMM_EPI_SWIGLU>(map_a, map_b, out, ldo, M, N, K, N / 2, sm_count, error, stream);
     }
-    if (epi != GEMM_EPI_F32 && epi != GEMM_EPI_BF16) return DISTIE_ERR_ARG;
+    if (epi != GEMM_EPI_F32 && epi != GEMM_EPI_BF16 && epi != GEMM_EPI_ACT) return DISTIE_ERR_ARG;
     const int width = tile_width ? tile_width : pick_tile_width(M, N, 2 * kGemmBM, sm_count / 2);
     if (width != 128 && width != 192 && width != 256) return DISTIE_ERR_ARG;
     if ((status = make_map(&map_b, w, N, K, K, width / 2)) != 0) return status;
     // (stages: what fits beside the float32 epilogue's 32 KB of staging, where that is asked for)
 #define DISTIE_GEMM_PAIR(BNV, STAGESV, STAGES32)                                                                          \
+  if (epi == GEMM_EPI_ACT)                                                                                                \
+    return launch_gemm_pair<BNV, STAGESV, 1, GEMM_EPI_ACT>(map_a, map_b, out, ldo, M, N, K, 0, sm_count, error, stream, more); \
   return epi == GEMM_EPI_F32                                                                                             \
              ? launch_gemm_pair<BNV, STAGES32, 1, GEMM_EPI_F32>(map_a, map_b, out, ldo, M, N, K, 0, sm_count, error, stream) \
              : launch_gemm_pair<BNV, STAGESV, 1, GEMM_EPI_BF16>(map_a, map_b, out, ldo, M, N, K, 0, sm_count, error, stream)
@@ -1092,12 +1117,14 @@ extern "C" int distie_gemm_tcgen05(const void* x, int ldx, const void* w, void* 
     if (status != 0) return status;
     return launch_gemm<256, 4, GEMM_EPI_SWIGLU>(map_a, map_b, out, ldo, M, N, K, N / 2, sm_count, error, stream);
   }
-  if (epi != GEMM_EPI_F32 && epi != GEMM_EPI_BF16) return DISTIE_ERR_ARG;
+  if (epi != GEMM_EPI_F32 && epi != GEMM_EPI_BF16 && epi != GEMM_EPI_ACT) return DISTIE_ERR_ARG;
   const int width = tile_width ? tile_width : pick_tile_width(M, N, kGemmBM, sm_count);
   if (width != 128 && width != 192 && width != 256) return DISTIE_ERR_ARG;
   status = make_map(&map_b, w, N, K, K, width);
   if (status != 0) return status;
 #define DISTIE_GEMM(BNV, STAGESV, STAGES32)                                                                              \
+  if (epi == GEMM_EPI_ACT)                                                                                               \
+    return launch_gemm<BNV, STAGESV, GEMM_EPI_ACT>(map_a, map_b, out, ldo, M, N, K, 0, sm_count, error, stream, more);   \
   return epi == GEMM_EPI_F32                                                                                            \
              ? launch_gemm<BNV, STAGES32, GEMM_EPI_F32>(map_a, map_b, out, ldo, M, N, K, 0, sm_count, error, stream) \
              : launch_gemm<BNV, STAGESV, GEMM_EPI_BF16>(map_a, map_b, out, ldo, M, N, K, 0, sm_count, error, stream)
@@ -1110,11 +1137,13 @@ extern "C" int distie_gemm_tcgen05(const void* x, int ldx, const void* w, void* 
 // The grouped product (see gemm_tcgen05_grouped_kernel): a[rows_a, K] sorted by group, w[groups * w_rows, K]; the tile
 // list lives on the device.  epi 2: w_rows = 2 * inter and out[rows_a, inter] bfloat16 = silu(a Wg^T) * (a Wu^T), or with
 // limit > 0 its capped form g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit);
-// epi 1: w_rows = N and out[rows_a, N] float32.  K a multiple of 8, rows 16-byte aligned.
+// epi 1: w_rows = N and out[rows_a, N] float32; epi 4: w_rows = N and out[rows_a, N] bfloat16 = act(a w^T) with the activation
+// of code `kind` and its factors act_a and act_b.  K a multiple of 8, rows 16-byte aligned.
 extern "C" int distie_gemm_tcgen05_grouped(const void* a, int lda, int rows_a, const void* w, int groups, int w_rows,
-                                           void* out, int ldo, int N, int K, int epi, float limit, const int* num_m_tiles,
-                                           const int* tile_group, const int* tile_first, const int* tile_rows,
-                                           int max_m_tiles, int sm_count, int* error, cudaStream_t stream) {
+                                           void* out, int ldo, int N, int K, int epi, float limit, int kind, float act_a,
+                                           float act_b, const int* num_m_tiles, const int* tile_group, const int* tile_first,
+                                           const int* tile_rows, int max_m_tiles, int sm_count, int* error,
+                                           cudaStream_t stream) {
   if (rows_a <= 0 || max_m_tiles <= 0) return 0;
   if (N < 1 || K < 8 || (K & 7) || (lda & 7) || ((uintptr_t)a & 15) || ((uintptr_t)w & 15) || groups < 1 || w_rows < 1)
     return DISTIE_ERR_UNSUPPORTED;
@@ -1124,7 +1153,22 @@ extern "C" int distie_gemm_tcgen05_grouped(const void* a, int lda, int rows_a, c
   int status = make_map(&map_a, a, rows_a, K, lda, kGemmBM);
   if (status != 0) return status;
   const GroupedTiles tiles{num_m_tiles, tile_group, tile_first, tile_rows, max_m_tiles, w_rows};
-  if (epi == GEMM_EPI_SWIGLU) {
+  const HiddenAct act{kind, act_a, act_b};
+  if (epi == GEMM_EPI_ACT) {
+    if (w_rows != N || kind < DISTIE_ACT_RELU2 || kind > DISTIE_ACT_XIELU) return DISTIE_ERR_ARG;
+    if ((status = make_map(&map_b, w, groups * w_rows, K, K, 256)) != 0) return status;
+    const size_t shared = sizeof(GemmShared<256, 4>) + 1024;
+    static bool configured = false;
+    if (!configured) {
+      const cudaError_t err = cudaFuncSetAttribute(gemm_tcgen05_grouped_kernel<256, 4, GEMM_EPI_ACT>,
+                                                   cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+      if (err != cudaSuccess) return (int)err;
+      configured = true;
+    }
+    const int num_tiles = max_m_tiles * ((N + 255) / 256);
+    gemm_tcgen05_grouped_kernel<256, 4, GEMM_EPI_ACT><<<num_tiles < sm_count ? num_tiles : sm_count, kGemmWideThreads, shared,
+                                                        stream>>>(map_a, map_b, out, ldo, N, K, 0, num_tiles, tiles, 0.f, act, error);
+  } else if (epi == GEMM_EPI_SWIGLU) {
     if (w_rows != 2 * N) return DISTIE_ERR_ARG;  // N counts the output columns (inter)
     if ((status = make_map(&map_b, w, groups * w_rows, K, K, 128)) != 0) return status;
     const size_t shared = sizeof(GemmShared<256, 4>) + 1024;
@@ -1138,7 +1182,7 @@ extern "C" int distie_gemm_tcgen05_grouped(const void* a, int lda, int rows_a, c
     const int num_tiles = max_m_tiles * ((N + 127) / 128);
     gemm_tcgen05_grouped_kernel<256, 4, GEMM_EPI_SWIGLU><<<num_tiles < sm_count ? num_tiles : sm_count, kGemmWideThreads,
                                                            shared, stream>>>(map_a, map_b, out, ldo, 2 * N, K, N, num_tiles,
-                                                                             tiles, limit, error);
+                                                                             tiles, limit, act, error);
   } else if (epi == GEMM_EPI_F32) {
     if (w_rows != N) return DISTIE_ERR_ARG;
     if ((status = make_map(&map_b, w, groups * w_rows, K, K, 256)) != 0) return status;
@@ -1152,7 +1196,7 @@ extern "C" int distie_gemm_tcgen05_grouped(const void* a, int lda, int rows_a, c
     }
     const int num_tiles = max_m_tiles * ((N + 255) / 256);
     gemm_tcgen05_grouped_kernel<256, 4, GEMM_EPI_F32><<<num_tiles < sm_count ? num_tiles : sm_count, kGemmWideThreads, shared,
-                                                        stream>>>(map_a, map_b, out, ldo, N, K, 0, num_tiles, tiles, 0.f, error);
+                                                        stream>>>(map_a, map_b, out, ldo, N, K, 0, num_tiles, tiles, 0.f, act, error);
   } else {
     return DISTIE_ERR_ARG;
   }
@@ -1208,7 +1252,8 @@ static int skinny_splits(int tiles, int K, int sm_count) {
 
 template <int BN, int STAGES, int EPI, typename OutT>
 static int launch_skinny_tc(const CUtensorMap& map_w, const CUtensorMap& map_x, const float* bias, OutT* out, int ldo,
-                            int M, int N, int K, int inter, int tiles, int splits, int* error, cudaStream_t stream) {
+                            int M, int N, int K, int inter, int tiles, int splits, int* error, cudaStream_t stream,
+                            HiddenAct act) {
   const size_t shared = sizeof(SkinnyShared<BN, STAGES>) + 1024;
   static bool configured = false;
   if (!configured) {
@@ -1219,13 +1264,14 @@ static int launch_skinny_tc(const CUtensorMap& map_w, const CUtensorMap& map_x, 
   }
   const cudaError_t err =
       launch_dependent_family(16, gemm_tcgen05_skinny_kernel<BN, STAGES, EPI, OutT>, dim3(tiles, splits),
-                              dim3(kGemmThreads), shared, stream, map_w, map_x, bias, out, ldo, M, N, K, inter, error);
+                              dim3(kGemmThreads), shared, stream, map_w, map_x, bias, out, ldo, M, N, K, inter, act, error);
   return err == cudaSuccess ? 0 : (int)err;
 }
 
 template <int EPI, typename OutT>
 static int dispatch_skinny_tc(const CUtensorMap& map_w, const void* x, int ldx, const float* bias, OutT* out, int ldo,
-                              int M, int N, int K, int inter, int tiles, int splits, int* error, cudaStream_t stream) {
+                              int M, int N, int K, int inter, int tiles, int splits, int* error, cudaStream_t stream,
+                              HiddenAct act = HiddenAct{0, 0.f, 0.f}) {
   CUtensorMap map_x;
   int status;
   // A CTA whose share of K is four blocks long or less asks for a ring of four stages: the shared
@@ -1235,21 +1281,21 @@ static int dispatch_skinny_tc(const CUtensorMap& map_w, const void* x, int ldx, 
   if (M <= 16) {
     if ((status = make_map(&map_x, x, M, K, ldx, 16)) != 0) return status;
     if (brief)
-      return launch_skinny_tc<16, 4, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream);
+      return launch_skinny_tc<16, 4, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream, act);
     // The product that hands slices to a consumer runs on eight stages, the others on ten (measured:
     // a decode step is 1.3 % shorter than with ten for all, and longer again with seven).
     if (EPI == SKINNY_EPI_SLICE)
-      return launch_skinny_tc<16, 8, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream);
-    return launch_skinny_tc<16, 10, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream);
+      return launch_skinny_tc<16, 8, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream, act);
+    return launch_skinny_tc<16, 10, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream, act);
   }
   if (M <= 32) {
     if ((status = make_map(&map_x, x, M, K, ldx, 32)) != 0) return status;
     if (brief)
-      return launch_skinny_tc<32, 4, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream);
-    return launch_skinny_tc<32, 9, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream);
+      return launch_skinny_tc<32, 4, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream, act);
+    return launch_skinny_tc<32, 9, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream, act);
   }
   if ((status = make_map(&map_x, x, M, K, ldx, 64)) != 0) return status;
-  return launch_skinny_tc<64, 7, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream);
+  return launch_skinny_tc<64, 7, EPI, OutT>(map_w, map_x, bias, out, ldo, M, N, K, inter, tiles, splits, error, stream, act);
 }
 
 }  // namespace distie
@@ -1263,6 +1309,21 @@ extern "C" int distie_gemm_tcgen05_skinny_splits(int N, int K, int sm_count) {
 //   mode 0: out[splits, M, N] float32 slices (ldo = N); their sum is x w^T
 //   mode 1: out[M, N] bfloat16 (out_dtype 1) or float32 (0) = x w^T + bias
 //   mode 2: w is [2 * inter, K]; out[M, inter] bfloat16 = silu(x Wg^T) * (x Wu^T)
+//   mode 3 (the entry point below with an activation): out[M, N] bfloat16 = act(x w^T)
+extern "C" int distie_gemm_tcgen05_skinny_act(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
+                                              int kind, float a, float b, int sm_count, int* error, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (M > 64 || N < 1 || K < 8 || (K & 7) || (ldx & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
+    return DISTIE_ERR_UNSUPPORTED;
+  if (kind < DISTIE_ACT_RELU2 || kind > DISTIE_ACT_XIELU) return DISTIE_ERR_ARG;
+  (void)sm_count;
+  CUtensorMap map_w;
+  const int status = make_map(&map_w, w, N, K, K, kGemmBM);
+  if (status != 0) return status;
+  return dispatch_skinny_tc<SKINNY_EPI_ACT, __nv_bfloat16>(map_w, x, ldx, nullptr, (__nv_bfloat16*)out, ldo, M, N, K, 0,
+                                                           (N + kGemmBM - 1) / kGemmBM, 1, error, stream, HiddenAct{kind, a, b});
+}
+
 extern "C" int distie_gemm_tcgen05_skinny(const void* x, int ldx, const void* w, const float* bias, void* out, int ldo,
                                           int M, int N, int K, int mode, int out_dtype, int sm_count, int* error,
                                           cudaStream_t stream) {

@@ -9,7 +9,7 @@
 //   latent_attention  (kernels below) causal softmax over the request's rows with a sink in the denominator.
 //   latent_gate       [heads, T, vdim] -> [T, heads * vdim] times sigmoid(gate[t, head]).
 //   glu_act           float32 [T, 2 ff] (gate columns, then up columns) -> SwiGLU or its capped form, optionally
-//                     times sigmoid of a per-row logit; float32 [T, ff] -> squared ReLU.
+//                     times sigmoid of a per-row logit; float32 [T, ff] -> squared ReLU, GELU or xIELU.
 //
 // Arithmetic is float32 everywhere (norm statistics, angles, scores, softmax, the mix); T (float or bfloat16) is
 // the type of what is stored.  Nothing reads host-side batch data.
@@ -53,10 +53,12 @@ latent_kv_write_kernel(const float* __restrict__ proj, int row_stride, int slice
     if (c < q_rank) sq_q += v * v;
     else if (c < q_rank + kv_rank) sq_kv += v * v;
   }
-  sq_q = block_sum(sq_q, scratch);
-  const float inv_q = 1.f / sqrtf(sq_q / (float)q_rank + eps);
-  for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
-    q_out[(size_t)t * q_out_stride + c] = from_float<T>(row_s[c] * inv_q * q_norm[c]);
+  if (q_rank > 0) {
+    sq_q = block_sum(sq_q, scratch);
+    const float inv_q = 1.f / sqrtf(sq_q / (float)q_rank + eps);
+    for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
+      q_out[(size_t)t * q_out_stride + c] = from_float<T>(row_s[c] * inv_q * q_norm[c]);
+  }
   if (!write) return;
   sq_kv = block_sum(sq_kv, scratch);
   const float inv_kv = 1.f / sqrtf(sq_kv / (float)kv_rank + eps);
@@ -146,11 +148,11 @@ __device__ __forceinline__ float glu_value(float g, float u, float limit) {
   return g * sigmoid_f(g) * u;
 }
 
-// kind 0: gated (x is [T, 2 ff]); kind 1: squared ReLU (x is [T, ff]).
+// kind 0: gated (x is [T, 2 ff]); other kinds: the activation of that code (x is [T, ff]).
 template <typename T>
 __global__ void __launch_bounds__(256)
 glu_act_kernel(const float* __restrict__ x, int row_stride, int slices, long long slice_stride, int tokens, int ff,
-               int kind, float limit, const float* __restrict__ row_gate, int gate_stride, int gate_slices,
+               int kind, float limit, float act_a, float act_b, const float* __restrict__ row_gate, int gate_stride, int gate_slices,
                long long gate_slice_stride, T* __restrict__ out, int out_stride) {
   const int t = blockIdx.y;
   const float* src = x + (size_t)t * row_stride;
@@ -158,9 +160,8 @@ glu_act_kernel(const float* __restrict__ x, int row_stride, int slices, long lon
   if (row_gate) row_scale = sigmoid_f(sum_slices(row_gate + (size_t)t * gate_stride, gate_slices, gate_slice_stride));
   for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < ff; c += gridDim.x * blockDim.x) {
     float v;
-    if (kind == 1) {
-      const float z = fmaxf(sum_slices(src + c, slices, slice_stride), 0.f);
-      v = z * z;
+    if (kind > 0) {
+      v = hidden_act(sum_slices(src + c, slices, slice_stride), HiddenAct{kind, act_a, act_b});
     } else {
       v = glu_value(sum_slices(src + c, slices, slice_stride), sum_slices(src + ff + c, slices, slice_stride), limit);
     }
@@ -406,7 +407,7 @@ extern "C" int distie_latent_kv_write(const float* proj, int row_stride, int sli
                                       void* k_cache, int page_size, int num_pages, int write, int tokens, int dtype,
                                       int* error, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (q_rank < 1 || slices < 1 || (rotary_dim & 1) || rotary_dim < 0 || rotary_dim > rot_dim ||
+  if (q_rank < 0 || (q_rank > 0 && (!q_norm || !q_out)) || (q_rank == 0 && !write) || slices < 1 || (rotary_dim & 1) || rotary_dim < 0 || rotary_dim > rot_dim ||
       (write && (kv_rank < 1 || rot_dim < 0 || page_size < 1 || table_width < 1 || !k_cache || !kv_norm)) ||
       (write && rotary_dim > 0 && !inv_freq))
     return DISTIE_ERR_ARG;
@@ -515,17 +516,17 @@ extern "C" int distie_latent_gate(const void* y, int tokens, int heads, int vdim
 }
 
 extern "C" int distie_glu_act(const float* x, int row_stride, int slices, long long slice_stride, int tokens, int ff,
-                              int kind, float limit, const float* row_gate, int gate_stride, int gate_slices,
-                              long long gate_slice_stride, void* out, int out_stride, int dtype, cudaStream_t stream) {
+                              int kind, float limit, float act_a, float act_b, const float* row_gate, int gate_stride,
+                              int gate_slices, long long gate_slice_stride, void* out, int out_stride, int dtype, cudaStream_t stream) {
   if (tokens <= 0 || ff <= 0) return 0;
-  if (slices < 1 || kind < 0 || kind > 1 || (row_gate && gate_slices < 1) || tokens > 65535 * 32) return DISTIE_ERR_ARG;
+  if (slices < 1 || kind < 0 || kind > DISTIE_ACT_XIELU || (row_gate && gate_slices < 1) || tokens > 65535 * 32) return DISTIE_ERR_ARG;
   const dim3 grid((ff + 255) / 256 > 64 ? 64 : (ff + 255) / 256, tokens);
   if (dtype == DISTIE_BF16)
-    glu_act_kernel<<<grid, 256, 0, stream>>>(x, row_stride, slices, slice_stride, tokens, ff, kind, limit, row_gate,
-                                             gate_stride, gate_slices, gate_slice_stride, (__nv_bfloat16*)out, out_stride);
+    glu_act_kernel<<<grid, 256, 0, stream>>>(x, row_stride, slices, slice_stride, tokens, ff, kind, limit, act_a, act_b,
+                                             row_gate, gate_stride, gate_slices, gate_slice_stride, (__nv_bfloat16*)out, out_stride);
   else if (dtype == DISTIE_F32)
-    glu_act_kernel<<<grid, 256, 0, stream>>>(x, row_stride, slices, slice_stride, tokens, ff, kind, limit, row_gate,
-                                             gate_stride, gate_slices, gate_slice_stride, (float*)out, out_stride);
+    glu_act_kernel<<<grid, 256, 0, stream>>>(x, row_stride, slices, slice_stride, tokens, ff, kind, limit, act_a, act_b,
+                                             row_gate, gate_stride, gate_slices, gate_slice_stride, (float*)out, out_stride);
   else
     return DISTIE_ERR_UNSUPPORTED;
   DISTIE_LAUNCH_CHECK();

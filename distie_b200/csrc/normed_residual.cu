@@ -5,6 +5,8 @@
 //  * norm_add_rmsnorm: d = sum_j scale_j * term_j (float32); residual += d * rsqrt(mean(d^2) + eps_d) * w_d
 //    (or += d when there is no w_d), written back; out = residual * rsqrt(mean(residual^2) + eps) * w, cast
 //    once at the store.  One block per row; with a list of rows only those are made and the residual stays.
+//  * average_add_rmsnorm: the same with an average over depth between the sum and the second norm: the sum is the
+//    layer's own result X, kept as the next of the states so far, and the residual becomes a weighted sum of them all.
 //  * qk_rope_norm_write: from the float32 projection [q | k] (a matrix or the slices of a split product) plus
 //    bias: the key as projected is stored as the value; q and k are rotated over the first `rotary_dim`
 //    elements of each head (angles pos * inv_freq in float32), then each head is divided by its root mean
@@ -120,6 +122,122 @@ norm_add_rmsnorm_vec_kernel(ResidualTerms terms, const float* __restrict__ delta
     if (c < hidden) {
       const float4 w = *reinterpret_cast<const float4*>(weight + c);
       store4(out_row + c, make_float4(r[p].x * unit * w.x, r[p].y * unit * w.y, r[p].z * unit * w.z, r[p].w * unit * w.w));
+    }
+  }
+}
+
+// A layer's end in a decoder that averages over depth.  X = residual + (normed) sum of the terms; history[count] = X
+// (where count < slots); residual = sum_(j < count) mix[j] * history[j] + mix[count] * X; out = its norm.  history is
+// [slots, rows, hidden].  With a list of rows only those are made, and residual and history stay as they are.
+struct DepthStates {
+  float* history;
+  size_t stride;  // floats from one state to the next
+  int count, slots;
+  const float* mix;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(512)
+average_add_rmsnorm_kernel(ResidualTerms terms, const float* __restrict__ delta_weight, float delta_eps,
+                           float* __restrict__ residual, DepthStates states, const float* __restrict__ weight, float eps,
+                           T* __restrict__ out, const int* __restrict__ rows_index, int hidden) {
+  extern __shared__ __align__(16) float row_s[];  // the summed terms, then the averaged residual
+  __shared__ float scratch[32];
+  const int i = blockIdx.x;
+  const size_t row = rows_index ? (size_t)rows_index[i] : (size_t)i;
+  float* res = residual + row * hidden;
+  float* past = states.history + row * hidden;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    float d = 0.f;
+    for (int j = 0; j < terms.count; ++j) d += terms.scale[j] * terms.ptr[j][row * hidden + c];
+    row_s[c] = d;
+    ss += d * d;
+  }
+  float factor = 1.f;
+  if (delta_weight) factor = rsqrtf(block_sum(ss, scratch) / (float)hidden + delta_eps);
+  ss = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    const float x = res[c] + (delta_weight ? row_s[c] * factor * delta_weight[c] : row_s[c]);
+    float r = 0.f;
+    for (int j = 0; j < states.count; ++j) r += states.mix[j] * past[(size_t)j * states.stride + c];
+    r += states.mix[states.count] * x;
+    row_s[c] = r;
+    if (!rows_index) {
+      if (states.count < states.slots) past[(size_t)states.count * states.stride + c] = x;
+      res[c] = r;
+    }
+    ss += r * r;
+  }
+  if (!out) return;
+  const float unit = rsqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+  T* out_row = out + (size_t)i * hidden;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) out_row[c] = from_float<T>(row_s[c] * unit * weight[c]);
+}
+
+// The same with four columns a thread and the row in registers (sizes and alignment as in norm_add_rmsnorm_vec_kernel).
+// The earlier states do not wait for the layer's own result: their sum is on its way while the terms are normed.
+template <typename T, int PIECES>
+__global__ void __launch_bounds__(512)
+average_add_rmsnorm_vec_kernel(ResidualTerms terms, const float* __restrict__ delta_weight, float delta_eps,
+                               float* __restrict__ residual, DepthStates states, const float* __restrict__ weight,
+                               float eps, T* __restrict__ out, const int* __restrict__ rows_index, int hidden) {
+  __shared__ float scratch[32];
+  const int i = blockIdx.x;
+  const size_t row = rows_index ? (size_t)rows_index[i] : (size_t)i;
+  float* res = residual + row * hidden;
+  float* past = states.history + row * hidden;
+  float4 d[PIECES], sum[PIECES];
+  float ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 4;
+    d[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+    sum[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < hidden) {
+      for (int j = 0; j < terms.count; ++j) {
+        const float4 v = *reinterpret_cast<const float4*>(terms.ptr[j] + row * hidden + c);
+        const float s = terms.scale[j];
+        d[p].x += s * v.x; d[p].y += s * v.y; d[p].z += s * v.z; d[p].w += s * v.w;
+      }
+#pragma unroll 8
+      for (int j = 0; j < states.count; ++j) {
+        const float4 v = *reinterpret_cast<const float4*>(past + (size_t)j * states.stride + c);
+        const float s = states.mix[j];
+        sum[p].x += s * v.x; sum[p].y += s * v.y; sum[p].z += s * v.z; sum[p].w += s * v.w;
+      }
+      ss += (d[p].x * d[p].x + d[p].y * d[p].y) + (d[p].z * d[p].z + d[p].w * d[p].w);
+    }
+  }
+  float factor = 1.f;
+  if (delta_weight) factor = rsqrtf(block_sum(ss, scratch) / (float)hidden + delta_eps);
+  const float last = states.mix[states.count];
+  ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 4;
+    if (c < hidden) {
+      float4 x = *reinterpret_cast<const float4*>(res + c), w = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (delta_weight) w = *reinterpret_cast<const float4*>(delta_weight + c);
+      x.x += d[p].x * factor * w.x; x.y += d[p].y * factor * w.y;
+      x.z += d[p].z * factor * w.z; x.w += d[p].w * factor * w.w;
+      sum[p].x += last * x.x; sum[p].y += last * x.y; sum[p].z += last * x.z; sum[p].w += last * x.w;
+      if (!rows_index) {
+        if (states.count < states.slots) *reinterpret_cast<float4*>(past + (size_t)states.count * states.stride + c) = x;
+        *reinterpret_cast<float4*>(res + c) = sum[p];
+      }
+      ss += (sum[p].x * sum[p].x + sum[p].y * sum[p].y) + (sum[p].z * sum[p].z + sum[p].w * sum[p].w);
+    }
+  }
+  if (!out) return;
+  const float unit = rsqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+  T* out_row = out + (size_t)i * hidden;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * 4;
+    if (c < hidden) {
+      const float4 w = *reinterpret_cast<const float4*>(weight + c);
+      store4(out_row + c, make_float4(sum[p].x * unit * w.x, sum[p].y * unit * w.y, sum[p].z * unit * w.z, sum[p].w * unit * w.w));
     }
   }
 }
@@ -345,6 +463,56 @@ extern "C" int distie_norm_add_rmsnorm(const float* const* term_ptrs, const floa
   } else {
     return DISTIE_ERR_UNSUPPORTED;
   }
+  DISTIE_LAUNCH_CHECK();
+  return 0;
+}
+
+// As distie_norm_add_rmsnorm, with the average over depth of average_add_rmsnorm_kernel: history is [slots, rows of the
+// residual, hidden] (`history_stride` floats from one state to the next), mix [count + 1].
+extern "C" int distie_average_add_rmsnorm(const float* const* term_ptrs, const float* term_scales, int num_terms,
+                                          const float* delta_weight, float delta_eps, float* residual, float* history,
+                                          long long history_stride, int count, int slots, const float* mix,
+                                          const float* weight, float eps, void* out, const int* rows_index, int rows,
+                                          int hidden, int dtype, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (hidden < 1 || num_terms < 0 || num_terms > kResidualTerms || residual == nullptr || history == nullptr || mix == nullptr ||
+      count < 0 || count > slots || (out && !weight))
+    return DISTIE_ERR_ARG;
+  if (dtype != DISTIE_BF16 && dtype != DISTIE_F32) return DISTIE_ERR_UNSUPPORTED;
+  ResidualTerms terms;
+  terms.count = num_terms;
+  for (int j = 0; j < num_terms; ++j) { terms.ptr[j] = term_ptrs[j]; terms.scale[j] = term_scales[j]; }
+  const DepthStates states{history, (size_t)history_stride, count, slots, mix};
+  uintptr_t low_bits = (uintptr_t)residual | (uintptr_t)weight | (uintptr_t)delta_weight | (uintptr_t)out | (uintptr_t)history;
+  for (int j = 0; j < num_terms; ++j) low_bits |= (uintptr_t)term_ptrs[j];
+  if (hidden % 4 == 0 && hidden <= 4 * 4 * 512 && history_stride % 4 == 0 && (low_bits & 15) == 0) {
+    const int quads = hidden / 4;
+    int vec_threads = 32;
+    while (vec_threads < 512 && vec_threads < quads) vec_threads *= 2;
+    const int pieces = (quads + vec_threads - 1) / vec_threads;
+#define DISTIE_AVERAGE_VEC(T, PIECESV)                                                                                     \
+  average_add_rmsnorm_vec_kernel<T, PIECESV><<<rows, vec_threads, 0, stream>>>(terms, delta_weight, delta_eps, residual,   \
+                                                                               states, weight, eps, (T*)out, rows_index, hidden)
+    if (dtype == DISTIE_BF16) {
+      if (pieces == 1) DISTIE_AVERAGE_VEC(__nv_bfloat16, 1); else if (pieces == 2) DISTIE_AVERAGE_VEC(__nv_bfloat16, 2);
+      else DISTIE_AVERAGE_VEC(__nv_bfloat16, 4);
+    } else {
+      if (pieces == 1) DISTIE_AVERAGE_VEC(float, 1); else if (pieces == 2) DISTIE_AVERAGE_VEC(float, 2);
+      else DISTIE_AVERAGE_VEC(float, 4);
+    }
+#undef DISTIE_AVERAGE_VEC
+    DISTIE_LAUNCH_CHECK();
+    return 0;
+  }
+  const int threads = hidden >= 4096 ? 512 : (hidden >= 1024 ? 256 : 128);
+  const size_t shared = (size_t)hidden * sizeof(float);
+  if (shared > 200 * 1024) return DISTIE_ERR_UNSUPPORTED;
+  auto run = [&](auto kernel, auto typed) {
+    if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+    kernel<<<rows, threads, shared, stream>>>(terms, delta_weight, delta_eps, residual, states, weight, eps, typed, rows_index, hidden);
+  };
+  if (dtype == DISTIE_BF16) run(average_add_rmsnorm_kernel<__nv_bfloat16>, (__nv_bfloat16*)out);
+  else run(average_add_rmsnorm_kernel<float>, (float*)out);
   DISTIE_LAUNCH_CHECK();
   return 0;
 }

@@ -14,43 +14,9 @@
 // this step); `seq_seat[b]` is the request's slot in every state tensor.  Nothing here reads
 // host-side batch data, so captured decode steps replay these kernels for whatever seats they
 // are given.
-#include "common.cuh"
+#include "recurrent.cuh"
 
 namespace distie {
-
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f); }
-__device__ __forceinline__ float gate_f(int sigmoid, float z) { return sigmoid ? sigmoid_f(z) : silu_f(z); }
-
-// A float32 matrix that may still be the slices of a split product: `splits` matrices `split_stride` floats apart
-// whose sum it is (splits == 1: the matrix itself).  Loads add the slices up, in their order.
-struct Sliced {
-  const float* p;
-  int stride;  // of a row
-  int splits;
-  long long split_stride;
-  const float* bias = nullptr;  // per column, added to the sum of the slices (a projection's bias); null: none
-  __device__ __forceinline__ float at(size_t row, int col) const {
-    const float* q = p + row * stride + col;
-    float v = q[0];
-    for (int s = 1; s < splits; ++s) v += q[(size_t)s * split_stride];
-    return bias ? v + bias[col] : v;
-  }
-  __device__ __forceinline__ float4 at4(size_t row, int col) const {
-    const float* q = p + row * stride + col;
-    float4 v = *reinterpret_cast<const float4*>(q);
-    for (int s = 1; s < splits; ++s) {
-      const float4 w = *reinterpret_cast<const float4*>(q + (size_t)s * split_stride);
-      v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
-    }
-    if (bias) {
-      const float4 b = *reinterpret_cast<const float4*>(bias + col);
-      v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
-    }
-    return v;
-  }
-};
 
 // ---------------------------------------------------------------------------
 // residual += sum_j scale_j * term_j (float32, written back), then
@@ -235,7 +201,7 @@ __global__ void short_conv_kernel(Sliced x, const float* __restrict__ weight,
                                   const float* __restrict__ bias, float* __restrict__ state,
                                   const int* __restrict__ token_seq, const int* __restrict__ token_first,
                                   const int* __restrict__ seq_seat, int channels, int taps, int silu, int single,
-                                  float* __restrict__ out) {
+                                  float* __restrict__ out, __nv_bfloat16* __restrict__ typed) {
   const int t = blockIdx.y;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= channels) return;
@@ -258,7 +224,9 @@ __global__ void short_conv_kernel(Sliced x, const float* __restrict__ weight,
       *slot = v;
     }
   }
-  out[(size_t)t * channels + c] = silu ? silu_f(acc) : acc;
+  if (silu) acc = silu_f(acc);
+  out[(size_t)t * channels + c] = acc;
+  if (typed) typed[(size_t)t * channels + c] = __float2bfloat16_rn(acc);
 }
 
 // A step in which every request brings one token: the thread reads its channel's taps-1 held inputs at once,
@@ -266,7 +234,7 @@ __global__ void short_conv_kernel(Sliced x, const float* __restrict__ weight,
 __global__ void short_conv_single_kernel(Sliced x, const float* __restrict__ weight, const float* __restrict__ bias,
                                          float* __restrict__ state, const int* __restrict__ token_seq,
                                          const int* __restrict__ seq_seat, int channels, int taps, int silu,
-                                         float* __restrict__ out) {
+                                         float* __restrict__ out, __nv_bfloat16* __restrict__ typed) {
   const int t = blockIdx.y;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= channels) return;
@@ -282,7 +250,9 @@ __global__ void short_conv_single_kernel(Sliced x, const float* __restrict__ wei
 #pragma unroll
   for (int i = 0; i < kMaxTaps - 1; ++i)
     if (i < taps - 1) held[(size_t)i * channels] = i + 1 < taps - 1 ? old[i + 1] : now;
-  out[(size_t)t * channels + c] = silu ? silu_f(acc) : acc;
+  if (silu) acc = silu_f(acc);
+  out[(size_t)t * channels + c] = acc;
+  if (typed) typed[(size_t)t * channels + c] = __float2bfloat16_rn(acc);
 }
 
 // Where each request's tokens lie in the step: seq_bounds[b] .. seq_bounds[b + 1] - 1 are the tokens of batch row b
@@ -309,7 +279,7 @@ __global__ void short_conv_vec_kernel(Sliced x, const float* __restrict__ weight
                                       const float* __restrict__ bias, const float* __restrict__ state,
                                       const int* __restrict__ token_seq, const int* __restrict__ token_first,
                                       const int* __restrict__ seq_seat, int channels, int taps_runtime, int silu,
-                                      float* __restrict__ out) {
+                                      float* __restrict__ out, __nv_bfloat16* __restrict__ typed) {
   const int taps = TAPS > 0 ? TAPS : taps_runtime;
   const int t = blockIdx.y;
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -332,6 +302,7 @@ __global__ void short_conv_vec_kernel(Sliced x, const float* __restrict__ weight
   }
   if (silu) acc = make_float4(silu_f(acc.x), silu_f(acc.y), silu_f(acc.z), silu_f(acc.w));
   *reinterpret_cast<float4*>(out + (size_t)t * channels + c) = acc;
+  if (typed) store4(typed + (size_t)t * channels + c, acc);
 }
 
 // Four taps, four channels and a run of eight tokens a thread, the window of held inputs in registers: every input
@@ -341,7 +312,8 @@ constexpr int kConvRun = 8;
 __global__ void short_conv_run4_kernel(Sliced x, const float* __restrict__ weight, const float* __restrict__ bias,
                                        const float* __restrict__ state, const int* __restrict__ token_seq,
                                        const int* __restrict__ token_first, const int* __restrict__ seq_seat, int tokens,
-                                       int channels, int silu, float* __restrict__ out) {
+                                       int channels, int silu, float* __restrict__ out,
+                                       __nv_bfloat16* __restrict__ typed) {
   const int t0 = blockIdx.y * kConvRun;
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (c >= channels) return;
@@ -362,6 +334,7 @@ __global__ void short_conv_run4_kernel(Sliced x, const float* __restrict__ weigh
   auto finish = [&](int t, float4 acc) {
     if (silu) acc = make_float4(silu_f(acc.x), silu_f(acc.y), silu_f(acc.z), silu_f(acc.w));
     *reinterpret_cast<float4*>(out + (size_t)t * channels + c) = acc;
+    if (typed) store4(typed + (size_t)t * channels + c, acc);
   };
   auto mac = [](float4 acc, float4 wj, float4 v) {
     return make_float4(acc.x + wj.x * v.x, acc.y + wj.y * v.y, acc.z + wj.z * v.z, acc.w + wj.w * v.w);
@@ -488,18 +461,6 @@ __global__ void __launch_bounds__(128) recurrence_prepare_kernel(ScanArgs a) {
     if (lane == 0) a.kq[(size_t)t * a.groups + grp] = kq;
   }
 }
-
-__device__ __forceinline__ void cp_async_f4(float* dst, const float* src, bool live) {
-  const int bytes = live ? 16 : 0;  // zero-fills when not live
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_f1(float* dst, const float* src, bool live) {
-  const int bytes = live ? 4 : 0;
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // One stage of the ring: a tile of q, k (rows of KD floats, zero beyond key_dim), the block's columns of v, and
 // per token g, the factor of u and k . q.
@@ -755,8 +716,14 @@ gated_rmsnorm_vec_kernel(const float* __restrict__ x, int x_stride, Sliced gate,
 // ---------------------------------------------------------------------------
 // out[t, c] = act(x[t, c]) (* scale for c < scaled_columns), x a matrix or the slices of a split product.
 // ---------------------------------------------------------------------------
+constexpr int kActNone = 0, kActSilu = 1, kActTanh = 2;
+__device__ __forceinline__ float plain_act(float v, int kind) {
+  return kind == kActSilu ? silu_f(v) : (kind == kActTanh ? tanhf(v) : v);
+}
+
 // Four columns a thread: columns, scaled_columns and the strides multiples of 4, pointers 16-byte aligned.
-__global__ void activation_vec_kernel(Sliced x, float* __restrict__ out, int tokens, int columns, int silu, float scale,
+template <typename T>
+__global__ void activation_vec_kernel(Sliced x, T* __restrict__ out, int tokens, int columns, int kind, float scale,
                                       int scaled_columns) {
   const int quads = columns / 4;
   const size_t total = (size_t)tokens * quads;
@@ -764,22 +731,23 @@ __global__ void activation_vec_kernel(Sliced x, float* __restrict__ out, int tok
     const size_t t = idx / quads;
     const int c = (int)(idx % quads) * 4;
     float4 v = x.at4(t, c);
-    if (silu) v = make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w));
+    v = make_float4(plain_act(v.x, kind), plain_act(v.y, kind), plain_act(v.z, kind), plain_act(v.w, kind));
     if (c < scaled_columns) v = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
-    *reinterpret_cast<float4*>(out + t * columns + c) = v;
+    store4(out + t * columns + c, v);
   }
 }
 
-__global__ void activation_kernel(Sliced x, float* __restrict__ out, int tokens, int columns, int silu, float scale,
+template <typename T>
+__global__ void activation_kernel(Sliced x, T* __restrict__ out, int tokens, int columns, int kind, float scale,
                                   int scaled_columns) {
   const size_t total = (size_t)tokens * columns;
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
     const size_t t = idx / columns;
     const int c = (int)(idx % columns);
     float v = x.at(t, c);
-    if (silu) v = silu_f(v);
+    v = plain_act(v, kind);
     if (c < scaled_columns) v *= scale;
-    out[idx] = v;
+    out[idx] = from_float<T>(v);
   }
 }
 
@@ -1047,36 +1015,37 @@ extern "C" int distie_short_conv(const float* x_ptr, int x_stride, int splits, l
                                  const float* weight, const float* bias, float* state,
                                  const int* token_seq, const int* token_first, const int* seq_bounds,
                                  const int* seq_seat, int tokens, int num_seqs, int channels, int taps, int silu,
-                                 int single, float* out, const float* input_bias, cudaStream_t stream) {
+                                 int single, float* out, const float* input_bias, void* typed_out, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (channels < 1 || taps < 1 || num_seqs < 1) return DISTIE_ERR_ARG;
   if (taps > kMaxTaps) return DISTIE_ERR_UNSUPPORTED;
   if (taps > 1 && state == nullptr) return DISTIE_ERR_ARG;
   if (splits < 1) return DISTIE_ERR_ARG;
   const Sliced x{x_ptr, x_stride, splits, split_stride, input_bias};  // input_bias [channels]: added to every input of the step
+  __nv_bfloat16* typed = (__nv_bfloat16*)typed_out;  // the same values for a product that reads them; null: not asked for
   const int threads = 128;
   const bool vec = !single && channels % 4 == 0 && x_stride % 4 == 0 && split_stride % 4 == 0 &&
-                   (((uintptr_t)x_ptr | (uintptr_t)state | (uintptr_t)out | (uintptr_t)bias | (uintptr_t)input_bias) & 15) == 0;
+                   (((uintptr_t)x_ptr | (uintptr_t)state | (uintptr_t)out | (uintptr_t)bias | (uintptr_t)input_bias | (uintptr_t)typed) & 15) == 0;
   if (vec) {
     const dim3 grid((channels / 4 + threads - 1) / threads, tokens);
     if (taps == 4 && ((uintptr_t)weight & 15) == 0) {
       const dim3 grid_runs(grid.x, (tokens + kConvRun - 1) / kConvRun);
       short_conv_run4_kernel<<<grid_runs, threads, 0, stream>>>(x, weight, bias, state, token_seq, token_first, seq_seat,
-                                                                tokens, channels, silu, out);
+                                                                tokens, channels, silu, out, typed);
     } else if (taps == 4)
       short_conv_vec_kernel<4><<<grid, threads, 0, stream>>>(x, weight, bias, state, token_seq, token_first,
-                                                             seq_seat, channels, taps, silu, out);
+                                                             seq_seat, channels, taps, silu, out, typed);
     else
       short_conv_vec_kernel<0><<<grid, threads, 0, stream>>>(x, weight, bias, state, token_seq, token_first,
-                                                             seq_seat, channels, taps, silu, out);
+                                                             seq_seat, channels, taps, silu, out, typed);
   } else if (single && taps > 1) {
     const dim3 grid((channels + threads - 1) / threads, tokens);
     short_conv_single_kernel<<<grid, threads, 0, stream>>>(x, weight, bias, state, token_seq, seq_seat, channels, taps,
-                                                           silu, out);
+                                                           silu, out, typed);
   } else {
     const dim3 grid((channels + threads - 1) / threads, tokens);
     short_conv_kernel<<<grid, threads, 0, stream>>>(x, weight, bias, state, token_seq, token_first, seq_seat,
-                                                    channels, taps, silu, single, out);
+                                                    channels, taps, silu, single, out, typed);
   }
   DISTIE_LAUNCH_CHECK();
   if (taps > 1 && !single) {
@@ -1165,23 +1134,26 @@ extern "C" int distie_gated_rmsnorm(const float* x, int x_stride, const float* g
   return 0;
 }
 
-extern "C" int distie_activation(const float* x, int x_stride, int splits, long long split_stride, float* out, int tokens,
-                                 int columns, int silu, float scale, int scaled_columns, cudaStream_t stream) {
+// kind: 0 none, 1 silu, 2 tanh; dtype: the type of out.
+extern "C" int distie_activation(const float* x, int x_stride, int splits, long long split_stride, void* out, int tokens,
+                                 int columns, int kind, float scale, int scaled_columns, int dtype, cudaStream_t stream) {
   if (tokens <= 0 || columns <= 0) return 0;
-  if (splits < 1 || scaled_columns < 0 || scaled_columns > columns) return DISTIE_ERR_ARG;
+  if (splits < 1 || scaled_columns < 0 || scaled_columns > columns || kind < 0 || kind > kActTanh) return DISTIE_ERR_ARG;
+  if (dtype != DISTIE_BF16 && dtype != DISTIE_F32) return DISTIE_ERR_UNSUPPORTED;
   const size_t total = (size_t)tokens * columns;
-  if (columns % 4 == 0 && scaled_columns % 4 == 0 && x_stride % 4 == 0 && split_stride % 4 == 0 &&
-      (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
-    const size_t quads = total / 4;
-    const unsigned vec_blocks = (unsigned)((quads + 255) / 256 > 148 * 16 ? 148 * 16 : (quads + 255) / 256);
-    activation_vec_kernel<<<vec_blocks, 256, 0, stream>>>(Sliced{x, x_stride, splits, split_stride}, out, tokens, columns,
-                                                         silu, scale, scaled_columns);
-    DISTIE_LAUNCH_CHECK();
-    return 0;
-  }
-  const unsigned blocks = (unsigned)((total + 255) / 256 > 148 * 16 ? 148 * 16 : (total + 255) / 256);
-  activation_kernel<<<blocks, 256, 0, stream>>>(Sliced{x, x_stride, splits, split_stride}, out, tokens, columns, silu,
-                                               scale, scaled_columns);
+  const bool vec = columns % 4 == 0 && scaled_columns % 4 == 0 && x_stride % 4 == 0 && split_stride % 4 == 0 &&
+                   (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+  const size_t units = vec ? total / 4 : total;
+  const unsigned blocks = (unsigned)((units + 255) / 256 > 148 * 16 ? 148 * 16 : (units + 255) / 256);
+  const Sliced rows{x, x_stride, splits, split_stride};
+#define DISTIE_ACTIVATION(T)                                                                                            \
+  do {                                                                                                                  \
+    if (vec) activation_vec_kernel<T><<<blocks, 256, 0, stream>>>(rows, (T*)out, tokens, columns, kind, scale, scaled_columns); \
+    else activation_kernel<T><<<blocks, 256, 0, stream>>>(rows, (T*)out, tokens, columns, kind, scale, scaled_columns); \
+  } while (0)
+  if (dtype == DISTIE_BF16) DISTIE_ACTIVATION(__nv_bfloat16);
+  else DISTIE_ACTIVATION(float);
+#undef DISTIE_ACTIVATION
   DISTIE_LAUNCH_CHECK();
   return 0;
 }

@@ -1,12 +1,13 @@
-// Kernels of a routed feed-forward: every token goes through `top` of `experts` small SwiGLU layers.
+// Kernels of a routed feed-forward: every token goes through `top` of `experts` small layers (SwiGLU, or two matrices
+// with an activation between them).
 //
-//   route_top     logits = x W_router^T in float32, scores = sigmoid(logits), the `top` largest per token
-//                 (ties to the lower index) with their scores.  One block per token.
+//   route_top     logits = x W_router^T (+ bias) in float32, scores = sigmoid(logits), the `top` largest per token
+//                 (ties to the lower index) with their scores; or the softmax over all or over the chosen logits.
 //   route_plan    (token, choice) pairs sorted by expert: for every slot of the sorted order the token it reads,
 //                 the weight of the pair and the row of the output it writes; the list of row tiles (expert,
 //                 first slot, rows) that the grouped products walk.  One block.
 //   grouped products over the sorted slots, a tile of rows of one expert per block:
-//                 hidden = silu(z Wg_e^T) * (z Wu_e^T) with z = weight * x[token] (or x[token]);
+//                 hidden = silu(z Wg_e^T) * (z Wu_e^T) with z = weight * x[token] (or x[token]), or act(z Wu_e^T);
 //                 out[choice, token, :] = hidden Wd_e^T (times the weight when it was not on the input).
 //
 // Nothing reads host-side batch data: counts, offsets and tiles stay on the device, so a captured decode step
@@ -32,6 +33,11 @@ __device__ __forceinline__ float routed_glu(float g, float u, float limit) {
   return routed_silu(g) * u;
 }
 
+// What a grouped product does: 0 the float32 rows of the output (down); 1 the gated hidden layer of stacked gate and up
+// rows; 2 the hidden layer of up rows alone with the activation of HiddenAct.
+constexpr int kGroupedDown = 0, kGroupedGated = 1, kGroupedAct = 2;
+
+constexpr int kScoreSigmoid = 0, kScoreSoftmax = 1, kScoreChosen = 2;  // 2: the softmax over the chosen logits alone
 constexpr int kRouteThreads = 256;
 constexpr int kMaxTop = 32;
 
@@ -42,9 +48,10 @@ constexpr int kMaxTop = 32;
 // index; the weights are the scores times `weight_scale`.  `plain` holds the scores the weights are taken from: `mine`
 // itself, or a second array when the choice runs on scores with a correction added (which may lie anywhere, so what
 // is taken or not eligible is marked with -infinity).  `normalise`: the chosen scores are divided by their sum + 1e-20.
+// `of_chosen`: the scores are logits and the weights the softmax over the chosen ones (the first chosen is the largest).
 __device__ __forceinline__ void route_choose(float* mine, float* group_s, int experts, int top, int count, int keep,
                                              float weight_scale, int* __restrict__ ids, float* __restrict__ weights,
-                                             int lane, const float* plain = nullptr, int normalise = 0) {
+                                             int lane, const float* plain = nullptr, int normalise = 0, int of_chosen = 0) {
   if (plain == nullptr) plain = mine;
   if (count > 1 && keep < count) {
     const int size = experts / count;
@@ -78,7 +85,7 @@ __device__ __forceinline__ void route_choose(float* mine, float* group_s, int ex
       if (group_s[e / size] != -3.f) mine[e] = -INFINITY;
     __syncwarp();
   }
-  float total = 0.f;
+  float total = 0.f, largest = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;  // a score taken or not eligible is -infinity
     int at = experts;
@@ -94,14 +101,19 @@ __device__ __forceinline__ void route_choose(float* mine, float* group_s, int ex
     }
     if (lane == 0 && at < experts) {
       ids[j] = at;
-      weights[j] = plain[at] * weight_scale;
-      total += plain[at];
+      float score = plain[at];
+      if (of_chosen) {
+        if (j == 0) largest = score;
+        score = expf(score - largest);
+      }
+      weights[j] = score * weight_scale;
+      total += score;
       mine[at] = -INFINITY;
     }
     __syncwarp();
   }
-  if (normalise && lane == 0) {
-    const float inv = 1.f / (total + 1e-20f);
+  if ((normalise || of_chosen) && lane == 0) {
+    const float inv = 1.f / (of_chosen ? total : total + 1e-20f);
     for (int j = 0; j < top; ++j) weights[j] *= inv;
   }
 }
@@ -111,7 +123,7 @@ __device__ __forceinline__ void route_choose(float* mine, float* group_s, int ex
 // the row itself becomes score + correction.  Returns where the plain scores lie.
 __device__ __forceinline__ const float* route_scores(float* mine, float* plain_s, int experts, int softmax,
                                                      const float* __restrict__ correction, int lane) {
-  if (softmax) {
+  if (softmax == kScoreSoftmax) {
     float top = -INFINITY;
     for (int e = lane; e < experts; e += 32) top = fmaxf(top, mine[e]);
 #pragma unroll
@@ -143,7 +155,7 @@ __global__ void __launch_bounds__(kRouteThreads)
 route_top_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ router, int tokens, int hidden, int experts,
                  int top, int* __restrict__ ids, float* __restrict__ weights, int group_count, int group_keep,
                  float weight_scale, int extra, float* __restrict__ extra_out, int softmax,
-                 const float* __restrict__ correction, int normalise) {
+                 const float* __restrict__ correction, int normalise, const float* __restrict__ logit_bias) {
   extern __shared__ __align__(16) float route_s[];
   float* x_s = route_s;
   float* scores_s = route_s + (size_t)TOK * hidden;  // per token: experts scores, group_count floats, experts plain scores
@@ -194,7 +206,8 @@ route_top_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ ro
     for (int r = 0; r < TOK; ++r) {
       const float z = warp_sum(dot[r]);
       if (lane == 0) {
-        if (e < experts) scores_s[r * score_row + e] = softmax ? z : routed_sigmoid(z);
+        const float zb = (logit_bias && e < experts) ? z + logit_bias[e] : z;
+        if (e < experts) scores_s[r * score_row + e] = softmax ? zb : routed_sigmoid(zb);
         else if (r < live) extra_out[(size_t)(t0 + r) * extra + e - experts] = z;
       }
     }
@@ -205,7 +218,7 @@ route_top_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ ro
     const size_t t = t0 + r;
     const float* plain = route_scores(mine, mine + experts + group_count, experts, softmax, correction, lane);
     route_choose(mine, mine + experts, experts, top, group_count, group_keep, weight_scale, ids + t * top, weights + t * top, lane,
-                 plain, normalise);
+                 plain, normalise, softmax == kScoreChosen);
   }
 }
 
@@ -213,20 +226,20 @@ route_top_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ ro
 __global__ void __launch_bounds__(kRouteThreads)
 route_pick_kernel(const float* __restrict__ logits, int logit_stride, int tokens, int experts, int top,
                   int* __restrict__ ids, float* __restrict__ weights, int group_count, int group_keep, float weight_scale,
-                  int softmax, const float* __restrict__ correction, int normalise) {
+                  int softmax, const float* __restrict__ correction, int normalise, const float* __restrict__ logit_bias) {
   extern __shared__ float pick_s[];  // per warp: a row of scores, group_count floats, a row of plain scores
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * (kRouteThreads / 32) + warp;
   if (t >= tokens) return;
   float* mine = pick_s + (size_t)warp * (2 * experts + group_count);
   for (int e = lane; e < experts; e += 32) {
-    const float z = logits[(size_t)t * logit_stride + e];
+    const float z = logits[(size_t)t * logit_stride + e] + (logit_bias ? logit_bias[e] : 0.f);
     mine[e] = softmax ? z : routed_sigmoid(z);
   }
   __syncwarp();
   const float* plain = route_scores(mine, mine + experts + group_count, experts, softmax, correction, lane);
   route_choose(mine, mine + experts, experts, top, group_count, group_keep, weight_scale, ids + (size_t)t * top,
-               weights + (size_t)t * top, lane, plain, normalise);
+               weights + (size_t)t * top, lane, plain, normalise, softmax == kScoreChosen);
 }
 
 // plan layout (int32): [0] number of tiles; [1 .. 1 + experts] offsets of the experts' slots; then
@@ -309,15 +322,17 @@ route_plan_kernel(const int* __restrict__ ids, const float* __restrict__ weights
 constexpr int kTileM = 32, kTileN = 64, kTileK = 16, kGroupedThreads = 256;
 
 // C[slot, n] = sum_k A[row(slot), k] * W[e][n, k] for the slots of one tile of one expert.
-//   SWIGLU: W is [experts, 2 N, K]; C = silu(A Wg^T) * (A Wu^T), stored as T in `out` [pairs, N] by slot.
-//   else:   W is [experts, N, K]; C stored as float32 in `out32` at row dest[slot] (times scale[slot] with scale_out).
+//   gated:  W is [experts, 2 N, K]; C = silu(A Wg^T) * (A Wu^T), stored as T in `out` [pairs, N] by slot.
+//   act:    W is [experts, N, K]; act(C) stored as T in `out` [pairs, N] by slot.
+//   down:   W is [experts, N, K]; C stored as float32 in `out32` at row dest[slot] (times scale[slot] with scale_out).
 // `gather`: A's row of a slot is source[slot] and is multiplied by scale[slot] when scale_in is set; otherwise the
 // slot's own row.
-template <typename T, bool SWIGLU>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(kGroupedThreads)
 grouped_product_kernel(const T* __restrict__ a, int a_stride, const T* __restrict__ w, int* __restrict__ plan_base,
                        int pairs, int experts, T* __restrict__ out, float* __restrict__ out32, int N, int K, int gather,
-                       int scale_in, int scale_out, float limit) {
+                       int scale_in, int scale_out, float limit, HiddenAct act) {
+  constexpr bool SWIGLU = MODE == kGroupedGated;
   const RoutePlan plan = plan_views(plan_base, pairs, experts, kTileM);
   const int tile = blockIdx.x;
   if (tile >= *plan.num_tiles) return;
@@ -383,6 +398,8 @@ grouped_product_kernel(const T* __restrict__ a, int a_stride, const T* __restric
       if (n >= N) continue;
       if (SWIGLU) {
         out[(size_t)slot * N + n] = from_float<T>(routed_glu(acc[r][c], acc_up[r][c], limit));
+      } else if (MODE == kGroupedAct) {
+        out[(size_t)slot * N + n] = from_float<T>(hidden_act(acc[r][c], act));
       } else {
         const float v = scale_out ? acc[r][c] * scale_s[local] : acc[r][c];
         out32[(size_t)plan.dest[slot] * N + n] = v;
@@ -397,12 +414,14 @@ grouped_product_kernel(const T* __restrict__ a, int a_stride, const T* __restric
 // 4 (rows) x 2 (columns) over a 64 x 64 tile (x 2 for gate and up).
 constexpr int kMmaM = 64, kMmaN = 64, kMmaK = 32, kMmaThreads = 256, kMmaPad = 8;
 
-template <bool SWIGLU>
+template <int MODE>
 __global__ void __launch_bounds__(kMmaThreads)
 grouped_product_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const __nv_bfloat16* __restrict__ w,
                            int* __restrict__ plan_base, int pairs, int experts, __nv_bfloat16* __restrict__ out,
-                           float* __restrict__ out32, int N, int K, int gather, int scale_in, int scale_out, float limit) {
+                           float* __restrict__ out32, int N, int K, int gather, int scale_in, int scale_out, float limit,
+                           HiddenAct act) {
   using namespace nvcuda;
+  constexpr bool SWIGLU = MODE == kGroupedGated;
   const RoutePlan plan = plan_views(plan_base, pairs, experts, kMmaM);
   const int tile = blockIdx.x;
   if (tile >= *plan.num_tiles) return;
@@ -487,6 +506,7 @@ grouped_product_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, co
         const int slot = first + local;
         const float v = c_s[warp][r][c];
         if (SWIGLU) out[(size_t)slot * N + n] = __float2bfloat16_rn(v);
+        else if (MODE == kGroupedAct) out[(size_t)slot * N + n] = __float2bfloat16_rn(hidden_act(v, act));
         else out32[(size_t)plan.dest[slot] * N + n] = scale_out ? v * scale_s[local] : v;
       }
     }
@@ -569,11 +589,12 @@ __global__ void routed_identity_kernel(const T* __restrict__ x, int x_stride, co
 constexpr int kRowsR = 8, kRowsWarps = 8;
 
 
-template <typename T, bool SWIGLU, int VEC>
+template <typename T, int MODE, int VEC>
 __global__ void __launch_bounds__(kRowsWarps * 32, 3)
 grouped_rows_kernel(int rounds, const T* __restrict__ a, int a_stride, const T* __restrict__ w, int* __restrict__ plan_base, int pairs,
                     int experts, T* __restrict__ out, float* __restrict__ out32, int N, int K, int gather, int scale_in,
-                    int scale_out, float limit) {
+                    int scale_out, float limit, HiddenAct act) {
+  constexpr bool SWIGLU = MODE == kGroupedGated;
   extern __shared__ __align__(16) unsigned char rows_raw[];
   T* a_s = reinterpret_cast<T*>(rows_raw);  // [kRowsR][K]
   __shared__ int src_s[kRowsR];
@@ -658,6 +679,9 @@ grouped_rows_kernel(int rounds, const T* __restrict__ a, int a_stride, const T* 
       const int slot = first + lane;
       if (SWIGLU) {
         out[(size_t)slot * N + n] = from_float<T>(routed_glu(v0, v1, limit));
+      } else if (MODE == kGroupedAct) {
+        out[(size_t)slot * N + n] = from_float<T>(hidden_act(v0, act));
+        if (second) out[(size_t)slot * N + n + 1] = from_float<T>(hidden_act(v1, act));
       } else {
         const float s = scale_out ? scale_s[lane] : 1.f;
         float* dst = out32 + (size_t)plan.dest[slot] * N + n;
@@ -668,9 +692,11 @@ grouped_rows_kernel(int rounds, const T* __restrict__ a, int a_stride, const T* 
   }
 }
 
-template <typename T, bool SWIGLU>
+template <typename T, int MODE>
 static int launch_grouped_rows(const T* a, int a_stride, const T* w, int* plan, int pairs, int experts, T* out, float* out32,
-                               int N, int K, int gather, int scale_in, int scale_out, float limit, unsigned max_tiles, cudaStream_t stream) {
+                               int N, int K, int gather, int scale_in, int scale_out, float limit, HiddenAct act, unsigned max_tiles,
+                               cudaStream_t stream) {
+  constexpr bool SWIGLU = MODE == kGroupedGated;
   constexpr int WIDE = sizeof(T) == 2 ? 8 : 4;
   const bool vec = K % WIDE == 0 && a_stride % WIDE == 0 && (((uintptr_t)a | (uintptr_t)w) & 15) == 0;
   const size_t shared = (size_t)kRowsR * K * sizeof(T);
@@ -681,10 +707,10 @@ static int launch_grouped_rows(const T* a, int a_stride, const T* w, int* plan, 
   auto run = [&](auto kernel) {
     if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     kernel<<<grid, kRowsWarps * 32, shared, stream>>>(rounds, a, a_stride, w, plan, pairs, experts, out, out32, N, K, gather, scale_in,
-                                                     scale_out, limit);
+                                                     scale_out, limit, act);
   };
-  if (vec) run(grouped_rows_kernel<T, SWIGLU, WIDE>);
-  else run(grouped_rows_kernel<T, SWIGLU, 1>);
+  if (vec) run(grouped_rows_kernel<T, MODE, WIDE>);
+  else run(grouped_rows_kernel<T, MODE, 1>);
   DISTIE_LAUNCH_CHECK();
   return 0;
 }
@@ -697,7 +723,7 @@ using namespace distie;
 extern "C" int distie_route_top(const void* x, int x_stride, const void* router, int tokens, int hidden, int experts,
                                 int top, int* ids, float* weights, int group_count, int group_keep, float weight_scale,
                                 int extra, float* extra_out, int softmax, const float* correction, int normalise,
-                                int dtype, cudaStream_t stream) {
+                                const float* logit_bias, int dtype, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (correction != nullptr && group_count > 1 && group_keep < group_count) return DISTIE_ERR_ARG;
   if (hidden < 1 || experts < 1 || top < 1 || top > experts || top > kMaxTop || experts > 8192 || group_count < 1 ||
@@ -714,7 +740,7 @@ extern "C" int distie_route_top(const void* x, int x_stride, const void* router,
   auto run = [&](auto kernel, auto xp, auto rp) {
     if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     kernel<<<blocks, kRouteThreads, shared, stream>>>(xp, x_stride, rp, tokens, hidden, experts, top, ids, weights, group_count,
-                                                      group_keep, weight_scale, extra, extra_out, softmax, correction, normalise);
+                                                      group_keep, weight_scale, extra, extra_out, softmax, correction, normalise, logit_bias);
   };
 #define DISTIE_ROUTE(T, VECV)                                                                             \
   do {                                                                                                    \
@@ -760,6 +786,58 @@ extern "C" int distie_routed_identity(const void* x, int x_stride, const int* id
   return 0;
 }
 
+// Both grouped products of every tile, HIDDEN: kGroupedGated (`up` is [experts, 2 ff, hidden]: gate rows, then up rows) or
+// kGroupedAct (`up` is [experts, ff, hidden]).
+template <int HIDDEN>
+static int run_experts(const void* x, int x_stride, const void* up, const void* down, int* plan, void* mid, float* out, int pairs,
+                       int experts, int hidden, int ff, int in, float limit, HiddenAct act, int tile, int dtype,
+                       cudaStream_t stream) {
+  typedef __nv_bfloat16 B16;
+  const unsigned max_tiles = (unsigned)((pairs + tile - 1) / tile + experts);
+  const HiddenAct none{0, 0.f, 0.f};
+  if (tile == kRowsR) {
+    int status;
+    if (dtype == DISTIE_BF16) {
+      status = launch_grouped_rows<B16, HIDDEN>((const B16*)x, x_stride, (const B16*)up, plan, pairs, experts, (B16*)mid, nullptr,
+                                                ff, hidden, 1, in, 0, limit, act, max_tiles, stream);
+      if (status != 0) return status;
+      return launch_grouped_rows<B16, kGroupedDown>((const B16*)mid, ff, (const B16*)down, plan, pairs, experts, nullptr, out,
+                                                    hidden, ff, 0, 0, 1 - in, 0.f, none, max_tiles, stream);
+    }
+    status = launch_grouped_rows<float, HIDDEN>((const float*)x, x_stride, (const float*)up, plan, pairs, experts, (float*)mid,
+                                                nullptr, ff, hidden, 1, in, 0, limit, act, max_tiles, stream);
+    if (status != 0) return status;
+    return launch_grouped_rows<float, kGroupedDown>((const float*)mid, ff, (const float*)down, plan, pairs, experts, nullptr, out,
+                                                    hidden, ff, 0, 0, 1 - in, 0.f, none, max_tiles, stream);
+  }
+  if (tile == kMmaM) {
+    const dim3 up_grid(max_tiles, (ff + kMmaN - 1) / kMmaN), down_grid(max_tiles, (hidden + kMmaN - 1) / kMmaN);
+    grouped_product_mma_kernel<HIDDEN><<<up_grid, kMmaThreads, 0, stream>>>(
+        (const B16*)x, x_stride, (const B16*)up, plan, pairs, experts, (B16*)mid, nullptr, ff, hidden, 1, in, 0, limit, act);
+    DISTIE_LAUNCH_CHECK();
+    grouped_product_mma_kernel<kGroupedDown><<<down_grid, kMmaThreads, 0, stream>>>(
+        (const B16*)mid, ff, (const B16*)down, plan, pairs, experts, nullptr, out, hidden, ff, 0, 0, 1 - in, 0.f, none);
+    DISTIE_LAUNCH_CHECK();
+    return 0;
+  }
+  const dim3 up_grid(max_tiles, (ff + kTileN - 1) / kTileN), down_grid(max_tiles, (hidden + kTileN - 1) / kTileN);
+  if (dtype == DISTIE_BF16) {
+    grouped_product_kernel<B16, HIDDEN><<<up_grid, kGroupedThreads, 0, stream>>>(
+        (const B16*)x, x_stride, (const B16*)up, plan, pairs, experts, (B16*)mid, nullptr, ff, hidden, 1, in, 0, limit, act);
+    DISTIE_LAUNCH_CHECK();
+    grouped_product_kernel<B16, kGroupedDown><<<down_grid, kGroupedThreads, 0, stream>>>(
+        (const B16*)mid, ff, (const B16*)down, plan, pairs, experts, nullptr, out, hidden, ff, 0, 0, 1 - in, 0.f, none);
+  } else {
+    grouped_product_kernel<float, HIDDEN><<<up_grid, kGroupedThreads, 0, stream>>>(
+        (const float*)x, x_stride, (const float*)up, plan, pairs, experts, (float*)mid, nullptr, ff, hidden, 1, in, 0, limit, act);
+    DISTIE_LAUNCH_CHECK();
+    grouped_product_kernel<float, kGroupedDown><<<down_grid, kGroupedThreads, 0, stream>>>(
+        (const float*)mid, ff, (const float*)down, plan, pairs, experts, nullptr, out, hidden, ff, 0, 0, 1 - in, 0.f, none);
+  }
+  DISTIE_LAUNCH_CHECK();
+  return 0;
+}
+
 // x [tokens, hidden]; gate_up [experts, 2 ff, hidden]; down [experts, hidden, ff]; ids, weights [tokens, top];
 // ids experts .. experts + identity - 1 stand for experts that return their input (weight on the output only).
 // plan: distie_route_plan_words int32; mid [tokens * top, ff] of the type; out [top, tokens, hidden] float32.
@@ -774,9 +852,8 @@ extern "C" int distie_routed_swiglu(const void* x, int x_stride, const int* ids,
   if (dtype != DISTIE_BF16 && dtype != DISTIE_F32) return DISTIE_ERR_UNSUPPORTED;
   const int pairs = tokens * top;
   const int tile = distie_routed_tile(dtype, hidden, ff, pairs, experts);
-  const bool mma = tile == kMmaM && x_stride % 8 == 0 &&
-                   (((uintptr_t)x | (uintptr_t)gate_up | (uintptr_t)down | (uintptr_t)mid) & 15) == 0;
-  if (tile == kMmaM && !mma) return DISTIE_ERR_UNSUPPORTED;
+  if (tile == kMmaM && (x_stride % 8 != 0 || (((uintptr_t)x | (uintptr_t)gate_up | (uintptr_t)down | (uintptr_t)mid) & 15) != 0))
+    return DISTIE_ERR_UNSUPPORTED;
   route_plan_kernel<<<1, 1024, 2 * (size_t)experts * sizeof(int), stream>>>(ids, weights, tokens, top, experts, tile, plan,
                                                                            error, identity);
   DISTIE_LAUNCH_CHECK();
@@ -784,54 +861,28 @@ extern "C" int distie_routed_swiglu(const void* x, int x_stride, const int* ids,
     const int status = distie_routed_identity(x, x_stride, ids, weights, tokens, top, experts, out, hidden, dtype, stream);
     if (status != 0) return status;
   }
-  const unsigned max_tiles = (unsigned)((pairs + tile - 1) / tile + experts);
-  const int in = weight_on_input ? 1 : 0;
-  if (tile == kRowsR) {
-    int status;
-    if (dtype == DISTIE_BF16) {
-      status = launch_grouped_rows<__nv_bfloat16, true>((const __nv_bfloat16*)x, x_stride, (const __nv_bfloat16*)gate_up, plan,
-                                                        pairs, experts, (__nv_bfloat16*)mid, nullptr, ff, hidden, 1, in, 0,
-                                                        limit, max_tiles, stream);
-      if (status != 0) return status;
-      return launch_grouped_rows<__nv_bfloat16, false>((const __nv_bfloat16*)mid, ff, (const __nv_bfloat16*)down, plan, pairs,
-                                                       experts, nullptr, out, hidden, ff, 0, 0, 1 - in, 0.f, max_tiles, stream);
-    }
-    status = launch_grouped_rows<float, true>((const float*)x, x_stride, (const float*)gate_up, plan, pairs, experts,
-                                              (float*)mid, nullptr, ff, hidden, 1, in, 0, limit, max_tiles, stream);
-    if (status != 0) return status;
-    return launch_grouped_rows<float, false>((const float*)mid, ff, (const float*)down, plan, pairs, experts, nullptr, out,
-                                             hidden, ff, 0, 0, 1 - in, 0.f, max_tiles, stream);
-  }
-  if (mma) {
-    const dim3 up_grid(max_tiles, (ff + kMmaN - 1) / kMmaN), down_grid(max_tiles, (hidden + kMmaN - 1) / kMmaN);
-    grouped_product_mma_kernel<true><<<up_grid, kMmaThreads, 0, stream>>>(
-        (const __nv_bfloat16*)x, x_stride, (const __nv_bfloat16*)gate_up, plan, pairs, experts, (__nv_bfloat16*)mid,
-        nullptr, ff, hidden, 1, in, 0, limit);
-    DISTIE_LAUNCH_CHECK();
-    grouped_product_mma_kernel<false><<<down_grid, kMmaThreads, 0, stream>>>(
-        (const __nv_bfloat16*)mid, ff, (const __nv_bfloat16*)down, plan, pairs, experts, nullptr, out, hidden, ff, 0, 0,
-        1 - in, 0.f);
-    DISTIE_LAUNCH_CHECK();
-    return 0;
-  }
-  const dim3 up_grid(max_tiles, (ff + kTileN - 1) / kTileN), down_grid(max_tiles, (hidden + kTileN - 1) / kTileN);
-  if (dtype == DISTIE_BF16) {
-    grouped_product_kernel<__nv_bfloat16, true><<<up_grid, kGroupedThreads, 0, stream>>>(
-        (const __nv_bfloat16*)x, x_stride, (const __nv_bfloat16*)gate_up, plan, pairs, experts, (__nv_bfloat16*)mid,
-        nullptr, ff, hidden, 1, in, 0, limit);
-    DISTIE_LAUNCH_CHECK();
-    grouped_product_kernel<__nv_bfloat16, false><<<down_grid, kGroupedThreads, 0, stream>>>(
-        (const __nv_bfloat16*)mid, ff, (const __nv_bfloat16*)down, plan, pairs, experts, nullptr, out, hidden, ff, 0, 0,
-        1 - in, 0.f);
-  } else {
-    grouped_product_kernel<float, true><<<up_grid, kGroupedThreads, 0, stream>>>(
-        (const float*)x, x_stride, (const float*)gate_up, plan, pairs, experts, (float*)mid, nullptr, ff, hidden, 1, in, 0, limit);
-    DISTIE_LAUNCH_CHECK();
-    grouped_product_kernel<float, false><<<down_grid, kGroupedThreads, 0, stream>>>(
-        (const float*)mid, ff, (const float*)down, plan, pairs, experts, nullptr, out, hidden, ff, 0, 0, 1 - in, 0.f);
-  }
+  return run_experts<kGroupedGated>(x, x_stride, gate_up, down, plan, mid, out, pairs, experts, hidden, ff,
+                                    weight_on_input ? 1 : 0, limit, HiddenAct{0, 0.f, 0.f}, tile, dtype, stream);
+}
+
+// The same for experts of two matrices: up [experts, ff, hidden], the activation of code `kind` with factors a and b
+// between them, the pair's weight on the expert's output.
+extern "C" int distie_routed_act(const void* x, int x_stride, const int* ids, const float* weights, const void* up,
+                                 const void* down, int* plan, void* mid, float* out, int tokens, int top, int experts,
+                                 int hidden, int ff, int kind, float a, float b, int dtype, int* error, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (top < 1 || experts < 1 || hidden < 1 || ff < 1 || experts > 4096 || kind < DISTIE_ACT_RELU2 || kind > DISTIE_ACT_XIELU)
+    return DISTIE_ERR_ARG;
+  if (dtype != DISTIE_BF16 && dtype != DISTIE_F32) return DISTIE_ERR_UNSUPPORTED;
+  const int pairs = tokens * top;
+  const int tile = distie_routed_tile(dtype, hidden, ff, pairs, experts);
+  if (tile == kMmaM && (x_stride % 8 != 0 || (((uintptr_t)x | (uintptr_t)up | (uintptr_t)down | (uintptr_t)mid) & 15) != 0))
+    return DISTIE_ERR_UNSUPPORTED;
+  route_plan_kernel<<<1, 1024, 2 * (size_t)experts * sizeof(int), stream>>>(ids, weights, tokens, top, experts, tile, plan,
+                                                                           error, 0);
   DISTIE_LAUNCH_CHECK();
-  return 0;
+  return run_experts<kGroupedAct>(x, x_stride, up, down, plan, mid, out, pairs, experts, hidden, ff, 0, 0.f, HiddenAct{kind, a, b},
+                                  tile, dtype, stream);
 }
 
 // The plan alone (see route_plan_kernel), for callers that run the grouped products themselves; `tile` rows a tile.
@@ -871,7 +922,7 @@ extern "C" int distie_routed_scatter(const float* y, int* plan, int pairs, int e
 // ids and weights from float32 logits [tokens, experts] (row stride logit_stride): see route_pick_kernel.
 extern "C" int distie_route_pick(const float* logits, int logit_stride, int tokens, int experts, int top, int* ids,
                                  float* weights, int group_count, int group_keep, float weight_scale, int softmax,
-                                 const float* correction, int normalise, cudaStream_t stream) {
+                                 const float* correction, int normalise, const float* logit_bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (correction != nullptr && group_count > 1 && group_keep < group_count) return DISTIE_ERR_ARG;
   if (experts < 1 || top < 1 || top > experts || top > kMaxTop || experts > 4096 || group_count < 1 ||
@@ -882,7 +933,8 @@ extern "C" int distie_route_pick(const float* logits, int logit_stride, int toke
   if (shared > 48 * 1024) cudaFuncSetAttribute(route_pick_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
   route_pick_kernel<<<(tokens + warps - 1) / warps, kRouteThreads, shared, stream>>>(logits, logit_stride, tokens, experts,
                                                                                     top, ids, weights, group_count, group_keep,
-                                                                                    weight_scale, softmax, correction, normalise);
+                                                                                    weight_scale, softmax, correction, normalise,
+                                                                                    logit_bias);
   DISTIE_LAUNCH_CHECK();
   return 0;
 }

@@ -20,7 +20,7 @@ import torch
 import ctypes
 
 from . import library
-from .interface import KernelSet, StepTensors, Terms
+from .interface import KernelSet, Normed, StepTensors, Terms
 from .library import KernelError, check, function
 
 _CODE = {torch.float32: 0, torch.bfloat16: 1}
@@ -31,6 +31,9 @@ _CLUSTER_SPLITS = 8             # splits of a decode attention that one cluster 
 _TENSOR_CORE_ROWS = 128         # from here on the tcgen05 kernel's 128-row tiles are full; in between: the library
 _MAX_TERMS = 24                 # terms of a pending sum that the layer-norm kernel adds up itself
 _RULES = {"delta": 0, "ssd": 1, "gated": 2}
+_ACTS = {"relu2": 1, "gelu": 2, "xielu": 3}
+_SCORINGS = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
+_PLAIN_ACTS = {"none": 0, "silu": 1, "tanh": 2}
 _GROUPED_TENSOR_CORE_PAIRS = 512  # (token, expert) pairs from which the routed products run on the tcgen05 tile kernel
 
 _ERROR_TEXT = {
@@ -564,22 +567,26 @@ class DeviceKernels(KernelSet):
             made = step.derived["seq_index"] = (token_first, bounds)
         return made
 
-    def short_conv(self, x, weight, bias, state, step, activation="silu", input_bias=None):
+    def short_conv(self, x, weight, bias, state, step, activation="silu", input_bias=None, typed=False):
         sliced = self._sliced(x, "short_conv")
         channels, taps = weight.shape
         out = torch.empty((step.num_tokens, channels), dtype=torch.float32, device=x.device)
         single = step.num_decode_tokens == step.num_tokens  # one token per request: the kernel moves the state on itself
         token_first, seq_bounds = self._seq_index(step)
+        narrow = torch.empty_like(out, dtype=self.dtype) if typed and self.dtype != torch.float32 else None
         check(
             function("distie_short_conv")(
                 *sliced, weight.data_ptr(), bias.data_ptr() if bias is not None else None,
                 state.data_ptr() if state is not None else None, step.token_seq.data_ptr(), token_first.data_ptr(),
                 seq_bounds.data_ptr(), step.seq_seat.data_ptr(), step.num_tokens, step.num_seqs, channels, taps, int(activation == "silu"), int(single), out.data_ptr(),
-                input_bias.data_ptr() if input_bias is not None else None, self._stream(),
+                input_bias.data_ptr() if input_bias is not None else None, narrow.data_ptr() if narrow is not None else None,
+                self._stream(),
             ),
             "short_conv",
         )
         self._ran("short_conv", 2 if taps > 1 and not single else 1)
+        if typed:
+            return out, out if narrow is None else narrow
         return out
 
     def linear_recurrence(self, rule, q, k, v, decay, write, state, step, heads, groups, key_dim, value_dim,
@@ -624,6 +631,58 @@ class DeviceKernels(KernelSet):
         )
         self._ran("gated_rmsnorm")
 
+    # -- recurrences whose decay varies by channel ------------------------------------------------------------------
+    def selective_scan(self, x, dt, B, C, gate, rates, skip, dt_bias, state, step, out) -> None:
+        self._rows32(x, "selective_scan x")
+        b_at, c_at = self._sliced(B, "selective_scan B"), self._sliced(C, "selective_scan C")
+        if b_at[1:] != c_at[1:]:
+            raise KernelError("selective_scan: B and C are views of one projection")
+        if not rates.is_contiguous() or not state.is_contiguous():
+            raise KernelError("selective_scan: contiguous rates and state are expected")
+        states, channels = rates.shape
+        # A long portion is cut into the step's tiles of 128 tokens where its channels alone would not fill the machine.
+        portions = step.num_seqs - step.num_decode_tokens
+        tiled = portions > 0 and step.num_q_tiles >= portions + 3 and portions * channels < 1024 * self.sm_count
+        tiles = step.num_q_tiles if tiled else 0
+        rows = step.num_decode_tokens if tiled else step.num_seqs
+        scratch = None
+        if tiled:
+            floats = function("distie_selective_scan_scratch_floats")(tiles, states, channels)
+            scratch = torch.empty(floats, dtype=torch.float32, device=x.device)
+        lanes = 4 if step.num_decode_tokens == step.num_tokens else 2
+        check(
+            function("distie_selective_scan")(
+                x.data_ptr(), x.stride(0), *self._sliced(dt, "selective_scan dt"), b_at[0], c_at[0], *b_at[1:],
+                *self._sliced(gate, "selective_scan gate"), rates.data_ptr(), skip.data_ptr(), dt_bias.data_ptr(),
+                state.data_ptr(), out.data_ptr(), out.stride(0), self._seq_index(step)[1].data_ptr(), step.seq_seat.data_ptr(),
+                step.token_seq.data_ptr(), step.q_tiles.data_ptr() if tiled else None, tiles,
+                scratch.data_ptr() if tiled else None, 0, rows, channels, states, lanes, _CODE[out.dtype], self._stream(),
+            ),
+            "selective_scan",
+        )
+        self._ran("selective_scan", (3 if tiled else 0) + (1 if rows else 0))
+        if tiled:
+            self._ran("selective_scan_tiled", 0)
+
+    def channel_delta(self, proj, decay, decay_bias, rate_bias, state, step, heads, dim):
+        if not state.is_contiguous():
+            raise KernelError("channel_delta: a contiguous state is expected")
+        tokens = step.num_tokens
+        out = torch.empty((tokens, heads * dim), dtype=torch.float32, device=proj.device)
+        floats = function("distie_channel_delta_scratch_floats")(tokens, heads, dim)
+        scratch = torch.empty(floats, dtype=torch.float32, device=proj.device)
+        lanes, cols = (16, 1) if step.num_decode_tokens < tokens else (8, 1)
+        check(
+            function("distie_channel_delta")(
+                *self._sliced(proj, "channel_delta"), *self._sliced(decay, "channel_delta decay"), decay_bias.data_ptr(),
+                rate_bias.data_ptr(), state.data_ptr(), out.data_ptr(), scratch.data_ptr(), self._seq_index(step)[1].data_ptr(),
+                step.seq_seat.data_ptr(), tokens, step.num_seqs, heads, dim, lanes, cols, self._stream(),
+            ),
+            "channel_delta",
+        )
+        self._ran("channel_delta", 2)
+        return out
+
     # -- norms around a sublayer, keys as values, memories with exponential gates, routed feed-forwards -------------
     def norm_add_rmsnorm(self, delta, delta_weight, delta_eps, residual, weight, eps, out, rows_index=None) -> None:
         pairs = [] if delta is None else Terms.of(delta).flat()
@@ -644,6 +703,33 @@ class DeviceKernels(KernelSet):
             "norm_add_rmsnorm",
         )
         self._ran("norm_add_rmsnorm")
+
+    def average_add_rmsnorm(self, ahead, residual, weight, eps, out, rows_index=None) -> None:
+        value, delta_weight, delta_eps = ahead.value, None, 0.0
+        if isinstance(value, Normed):
+            value, delta_weight, delta_eps = value.value, value.weight, value.eps
+        pairs = [] if value is None else Terms.of(value).flat()
+        if len(pairs) > _MAX_TERMS:  # more terms than the kernel takes: the tail is summed here, in float32
+            tail = Terms(pairs[_MAX_TERMS - 1 :]).total()
+            pairs = pairs[: _MAX_TERMS - 1] + [(tail, 1.0)]
+        pairs = [(t if t.is_contiguous() else t.contiguous(), s) for t, s in pairs]
+        pointers = (ctypes.c_void_p * max(1, len(pairs)))(*[t.data_ptr() for t, _ in pairs])
+        scales = (ctypes.c_float * max(1, len(pairs)))(*[s for _, s in pairs])
+        history = ahead.history
+        if not history[0].is_contiguous() or ahead.weights.numel() != ahead.count + 1:
+            raise KernelError("average_add_rmsnorm: contiguous states and a weight for each of them are expected")
+        check(
+            function("distie_average_add_rmsnorm")(
+                pointers, scales, len(pairs), delta_weight.data_ptr() if delta_weight is not None else None, float(delta_eps),
+                residual.data_ptr(), history.data_ptr(), history.stride(0), ahead.count, history.shape[0],
+                ahead.weights.data_ptr(), weight.data_ptr() if weight is not None else None, float(eps),
+                out.data_ptr() if out is not None else None, rows_index.data_ptr() if rows_index is not None else None,
+                out.shape[0] if out is not None else residual.shape[0], residual.shape[1],
+                _CODE[out.dtype] if out is not None else self.code, self._stream(),
+            ),
+            "average_add_rmsnorm",
+        )
+        self._ran("average_add_rmsnorm")
 
     def qk_rope_norm_write(self, qk, bias, step, kv, rotary, num_heads, num_kv_heads, head_dim, norm_eps, q_out) -> None:
         write = kv is not None
@@ -691,13 +777,14 @@ class DeviceKernels(KernelSet):
         )
         self._ran("qkv_norm_write")
 
-    def activation(self, x, kind="silu", scale=1.0, scaled_columns=0):
-        if kind not in ("silu", "none"):
-            raise KernelError(f"activation {kind!r}: 'silu' or 'none'")
-        out = torch.empty((x.shape[-2], x.shape[-1]), dtype=torch.float32, device=x.device)
+    def activation(self, x, kind="silu", scale=1.0, scaled_columns=0, out_dtype=None):
+        if kind not in _PLAIN_ACTS:
+            raise KernelError(f"activation {kind!r}: one of {', '.join(_PLAIN_ACTS)}")
+        out = torch.empty((x.shape[-2], x.shape[-1]), dtype=out_dtype or torch.float32, device=x.device)
         check(
             function("distie_activation")(*self._sliced(x, "activation"), out.data_ptr(), out.shape[0], out.shape[1],
-                                          int(kind == "silu"), float(scale), int(scaled_columns), self._stream()),
+                                          _PLAIN_ACTS[kind], float(scale), int(scaled_columns), _CODE[out.dtype],
+                                          self._stream()),
             "activation",
         )
         self._ran("activation")
@@ -735,10 +822,13 @@ class DeviceKernels(KernelSet):
         return out
 
     def route_top(self, x, router, top, scoring="sigmoid", groups=None, weight_scale=1.0, extra_rows=0, correction=None,
-                  normalise=False):
-        if scoring not in ("sigmoid", "softmax"):
-            raise KernelError(f"route_top: scoring {scoring!r} is not built; 'sigmoid' and 'softmax' are")
-        softmax, norm = int(scoring == "softmax"), int(bool(normalise))
+                  normalise=False, logit_bias=None):
+        if scoring not in _SCORINGS:
+            raise KernelError(f"route_top: scoring {scoring!r} is not built; {', '.join(_SCORINGS)} are")
+        if scoring == "softmax_chosen" and (correction is not None or groups is not None):
+            raise KernelError("route_top: a softmax over the chosen logits goes with neither a correction nor groups")
+        softmax, norm = _SCORINGS[scoring], int(bool(normalise))
+        bias_ptr = logit_bias.data_ptr() if logit_bias is not None else None
         correction_ptr = correction.data_ptr() if correction is not None else None
         library.load_unit("routed")
         if x.dtype != router.dtype:
@@ -757,7 +847,7 @@ class DeviceKernels(KernelSet):
             self._gemm_tcgen05(x, router, logits, 1)
             check(function("distie_route_pick")(logits.data_ptr(), logits.stride(0), tokens, experts, top, ids.data_ptr(),
                                                 weights.data_ptr(), count, keep, float(weight_scale), softmax, correction_ptr,
-                                                norm, self._stream()),
+                                                norm, bias_ptr, self._stream()),
                   "route_pick")
             self._ran("route_top")
             return (ids, weights, logits[:, experts:]) if extra else (ids, weights)
@@ -765,7 +855,7 @@ class DeviceKernels(KernelSet):
         check(
             function("distie_route_top")(x.data_ptr(), x.stride(0), router.data_ptr(), tokens, x.shape[1], experts, top,
                                          ids.data_ptr(), weights.data_ptr(), count, keep, float(weight_scale), extra,
-                                         extra_out.data_ptr() if extra else None, softmax, correction_ptr, norm,
+                                         extra_out.data_ptr() if extra else None, softmax, correction_ptr, norm, bias_ptr,
                                          _CODE[x.dtype], self._stream()),
             "route_top",
         )
@@ -789,7 +879,7 @@ class DeviceKernels(KernelSet):
             # rows that are no multiples of 16 bytes: the float32 form of the grouped products takes any size
             x, gate_up, down, code = x.float(), gate_up.float(), down.float(), 0
         if code == 1 and self.dtype == torch.bfloat16 and tokens * top >= _GROUPED_TENSOR_CORE_PAIRS:
-            return self._routed_swiglu_tcgen05(x, ids, weights, gate_up, down, scale_input, limit, identity)
+            return self._routed_tcgen05(x, ids, weights, gate_up, down, scale_input, limit, identity)
         tile = function("distie_routed_tile")(code, hidden, ff, tokens * top, experts)
         words = function("distie_route_plan_words")(tokens * top, experts, tile)
         plan = torch.empty(words, dtype=torch.int32, device=x.device)
@@ -806,11 +896,12 @@ class DeviceKernels(KernelSet):
         self._ran("routed_swiglu", 3)
         return out
 
-    def _routed_swiglu_tcgen05(self, x, ids, weights, gate_up, down, scale_input, limit=None, identity=0):
+    def _routed_tcgen05(self, x, ids, weights, up, down, scale_input, limit=None, identity=0, act=None):
         """Prompt portions in bfloat16: the rows sorted by expert (and scaled by their weights) are gathered once, and
-        both products run on the tcgen05 tile kernel over a list of row tiles that stays on the device."""
+        both products run on the tcgen05 tile kernel over a list of row tiles that stays on the device.  ``up`` holds gate
+        and up rows of gated experts, or with ``act`` (code, a, b) the up rows of experts with that activation."""
         tokens, top = ids.shape
-        experts, hidden, ff = gate_up.shape[0], x.shape[1], down.shape[2]
+        experts, hidden, ff = up.shape[0], x.shape[1], down.shape[2]
         pairs, tile = tokens * top, 128
         max_tiles = (pairs + tile - 1) // tile + experts
         words = function("distie_route_plan_words")(pairs, experts, tile)
@@ -825,12 +916,12 @@ class DeviceKernels(KernelSet):
                                                int(bool(scale_input)), 1, stream), "routed_gather")
         mid = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
         check(function("distie_gemm_tcgen05_grouped")(
-            gathered.data_ptr(), hidden, pairs, gate_up.data_ptr(), experts, 2 * ff, mid.data_ptr(), ff, ff, hidden, 2,
-            float(limit) if limit is not None else 0.0, base,
+            gathered.data_ptr(), hidden, pairs, up.data_ptr(), experts, up.shape[1], mid.data_ptr(), ff, ff, hidden,
+            2 if act is None else 4, float(limit) if limit is not None else 0.0, *(act or (0, 0.0, 0.0)), base,
             tile_expert, tile_first, tile_rows, max_tiles, self.sm_count, error, stream), "gemm_tcgen05_grouped")
         sorted_out = torch.empty((pairs, hidden), dtype=torch.float32, device=x.device)
         check(function("distie_gemm_tcgen05_grouped")(
-            mid.data_ptr(), ff, pairs, down.data_ptr(), experts, hidden, sorted_out.data_ptr(), hidden, hidden, ff, 1, 0.0, base,
+            mid.data_ptr(), ff, pairs, down.data_ptr(), experts, hidden, sorted_out.data_ptr(), hidden, hidden, ff, 1, 0.0, 0, 0.0, 0.0, base,
             tile_expert, tile_first, tile_rows, max_tiles, self.sm_count, error, stream), "gemm_tcgen05_grouped")
         out = torch.empty((top, tokens, hidden), dtype=torch.float32, device=x.device)
         if identity:
@@ -838,19 +929,53 @@ class DeviceKernels(KernelSet):
                                                      experts, out.data_ptr(), hidden, _CODE[x.dtype], stream), "routed_identity")
         check(function("distie_routed_scatter")(sorted_out.data_ptr(), base, pairs, experts, tile, out.data_ptr(), hidden,
                                                 int(not scale_input), stream), "routed_scatter")
-        self._ran("routed_swiglu", 5)
+        self._ran("routed_swiglu" if act is None else "routed_act", 5)
         self._ran("gemm_tcgen05_grouped", 0)
         return out
 
+    def routed_act(self, x, ids, weights, up, down, kind="gelu", numbers=None):
+        if kind not in _ACTS:
+            raise KernelError(f"routed_act: activation {kind!r} is not built; {', '.join(_ACTS)} are")
+        a, b = numbers or (0.0, 0.0)
+        if up.dtype != down.dtype:
+            raise KernelError("routed_act: the experts' matrices are of one type")
+        if up.dtype != x.dtype:
+            x = x.to(up.dtype)
+        if x.stride(1) != 1 or not up.is_contiguous() or not down.is_contiguous():
+            raise KernelError("routed_act: contiguous expert matrices and rows with unit column stride are expected")
+        tokens, top = ids.shape
+        experts, hidden, ff = up.shape[0], x.shape[1], down.shape[2]
+        code = _CODE[x.dtype]
+        if code == 1 and (x.stride(0) % 8 or hidden % 8 or ff % 8):
+            # rows that are no multiples of 16 bytes: the float32 form of the grouped products takes any size
+            x, up, down, code = x.float(), up.float(), down.float(), 0
+        if code == 1 and self.dtype == torch.bfloat16 and tokens * top >= _GROUPED_TENSOR_CORE_PAIRS:
+            return self._routed_tcgen05(x, ids, weights, up, down, False, act=(_ACTS[kind], float(a), float(b)))
+        tile = function("distie_routed_tile")(code, hidden, ff, tokens * top, experts)
+        words = function("distie_route_plan_words")(tokens * top, experts, tile)
+        plan = torch.empty(words, dtype=torch.int32, device=x.device)
+        mid = torch.empty((tokens * top, ff), dtype=x.dtype, device=x.device)
+        out = torch.empty((top, tokens, hidden), dtype=torch.float32, device=x.device)
+        check(
+            function("distie_routed_act")(
+                x.data_ptr(), x.stride(0), ids.data_ptr(), weights.data_ptr(), up.data_ptr(), down.data_ptr(), plan.data_ptr(),
+                mid.data_ptr(), out.data_ptr(), tokens, top, experts, hidden, ff, _ACTS[kind], float(a), float(b), code,
+                self.error_flag.data_ptr(), self._stream(),
+            ),
+            "routed_act",
+        )
+        self._ran("routed_act", 3)
+        return out
+
     # -- gated and squared-ReLU hidden layers on float32 accumulators; attention through a latent ------------------
-    def _glu_act(self, x32, ff: int, kind: int, limit, row_gate):
+    def _glu_act(self, x32, ff: int, kind: int, limit, row_gate, numbers=None):
         library.load_unit("latent")
         tokens = x32.shape[-2]
         out = torch.empty((tokens, ff), dtype=self.dtype, device=x32.device)
         gate = self._sliced(row_gate, "glu_act") if row_gate is not None else (None, 0, 1, 0)
         check(
             function("distie_glu_act")(*self._sliced(x32, "glu_act"), tokens, ff, kind, float(limit) if limit is not None else 0.0,
-                                       *gate, out.data_ptr(), out.stride(0), self.code, self._stream()),
+                                       *(float(n) for n in numbers or (0.0, 0.0)), *gate, out.data_ptr(), out.stride(0), self.code, self._stream()),
             "glu_act",
         )
         self._ran("glu_act")
@@ -865,29 +990,44 @@ class DeviceKernels(KernelSet):
             raise KernelError("linear_glu: the row gate is one logit per row")
         return self._glu_act(self.linear_split(x, weight), weight.shape[0] // 2, 0, limit, row_gate)
 
-    def linear_act(self, x, weight, kind="relu2"):
-        if kind != "relu2":
-            raise KernelError(f"linear_act: activation {kind!r} is not built; 'relu2' is")
-        return self._glu_act(self.linear_split(x, weight), weight.shape[0], 1, None, None)
+    def linear_act(self, x, weight, kind="relu2", numbers=None):
+        if kind not in _ACTS:
+            raise KernelError(f"linear_act: activation {kind!r} is not built; {', '.join(_ACTS)} are")
+        a, b = (float(n) for n in numbers or (0.0, 0.0))
+        if self._skinny(x, weight) or self._tensor_core(x, weight):  # the activation in the product's epilogue
+            out = torch.empty((x.shape[0], weight.shape[0]), dtype=self.dtype, device=x.device)
+            head = (x.data_ptr(), x.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0), x.shape[0], weight.shape[0],
+                    weight.shape[1])
+            tail = (_ACTS[kind], a, b, self.sm_count, self.error_flag.data_ptr(), self._stream())
+            if self._skinny(x, weight):
+                check(function("distie_gemm_tcgen05_skinny_act")(*head, *tail), "gemm_tcgen05_skinny_act")
+                self._ran("gemm_tcgen05_skinny")
+            else:
+                check(function("distie_gemm_tcgen05_act")(*head, 4, 0, *tail), "gemm_tcgen05_act")
+                self._ran("gemm_tcgen05")
+            return out
+        return self._glu_act(self.linear_split(x, weight), weight.shape[0], _ACTS[kind], None, None, numbers)
 
     def latent_kv_write(self, proj, step, kv, rotary, q_rank, q_norm, kv_rank, kv_norm, rot_dim, eps, q_latent_out) -> None:
         library.load_unit("latent")
         write = kv is not None
-        if write and (kv.k.dtype != q_latent_out.dtype or kv.k.shape[-1] != kv_rank + rot_dim or kv.k.shape[-3] != 1
+        dtype = q_latent_out.dtype if q_latent_out is not None else self.dtype
+        if write and (kv.k.dtype != dtype or kv.k.shape[-1] != kv_rank + rot_dim or kv.k.shape[-3] != 1
                       or not kv.k.is_contiguous()):
             raise KernelError("latent_kv_write: the cache holds one contiguous row [kv_rank + rot_dim] per token, of q's type")
         table = kv.block_table if write else step.seq_seat
         turned = rotary.rotary_dim if rotary is not None else 0
         check(
             function("distie_latent_kv_write")(
-                *self._sliced(proj, "latent_kv_write"), q_rank, q_norm.data_ptr(), kv_rank,
-                kv_norm.data_ptr() if write else None, rot_dim, float(eps), q_latent_out.data_ptr(), q_latent_out.stride(0),
+                *self._sliced(proj, "latent_kv_write"), q_rank, q_norm.data_ptr() if q_rank else None, kv_rank,
+                kv_norm.data_ptr() if write else None, rot_dim, float(eps), q_latent_out.data_ptr() if q_rank else None,
+                q_latent_out.stride(0) if q_rank else 0,
                 step.positions.data_ptr(), step.token_seq.data_ptr(), step.seq_seat.data_ptr(), table.data_ptr(),
                 table.shape[-1] if write else 1, rotary.inv_freq.data_ptr() if rotary is not None else None,
                 float(rotary.factor) if rotary is not None else 1.0, turned,
                 int(rotary.interleaved) if rotary is not None else 0, kv.k.data_ptr() if write else None,
                 kv.page_size if write else 1, kv.num_pages if write else 1, int(write), step.num_tokens,
-                _CODE[q_latent_out.dtype], self.error_flag.data_ptr(), self._stream(),
+                _CODE[dtype], self.error_flag.data_ptr(), self._stream(),
             ),
             "latent_kv_write",
         )

@@ -116,6 +116,29 @@ class Normed:
     eps: float
 
 
+@dataclass
+class Averaged:
+    """A layer's end in a decoder that averages over depth.  ``value`` (a :class:`Normed`, :class:`Terms`, a tensor or
+    None) is still to be added to the residual, which gives the layer's own result ``X``; ``X`` is then kept as
+    ``history[count]`` (when there is room: the last one is read by nobody) and the residual becomes
+    ``sum_(j < count) weights[j] * history[j] + weights[count] * X``.  ``history [slots, T, hidden]`` is float32, like
+    ``weights [count + 1]``.  The norm kernel that follows does all of it beside its own norm."""
+
+    value: object
+    history: torch.Tensor
+    count: int
+    weights: torch.Tensor
+
+    def close(self, state: torch.Tensor) -> torch.Tensor:
+        """The average, given the layer's own result (plain tensor operations)."""
+        if self.count < self.history.shape[0]:
+            self.history[self.count].copy_(state)
+        out = self.weights[self.count] * state
+        for j in range(self.count):
+            out = out + self.weights[j] * self.history[j]
+        return out
+
+
 @dataclass(frozen=True)
 class RotaryTable:
     """What the fused rotation kernel needs of a rotary position encoding."""
@@ -231,6 +254,12 @@ class KernelSet(ABC):
         residual stays as it is.  ``out`` None: only the residual is moved on."""
         raise NotImplementedError
 
+    def average_add_rmsnorm(self, ahead: Averaged, residual, weight, eps: float, out, rows_index=None) -> None:
+        """What :class:`Averaged` describes, then ``out = cast(residual * rsqrt(mean(residual^2) + eps) * weight)`` of
+        the averaged residual (kept), all float32 up to the one cast.  With ``rows_index`` only those rows are made and
+        residual and history stay as they are.  ``out`` None: only residual and history are moved on."""
+        raise NotImplementedError
+
     def qk_rope_norm_write(self, qk, bias, step: StepTensors, kv: KvSlot | None, rotary: RotaryTable | None,
                            num_heads: int, num_kv_heads: int, head_dim: int, norm_eps: float | None, q_out) -> None:
         """For layers whose values are their keys: ``qk`` is the projection ``[T, (heads + kv_heads) * head_dim]``
@@ -240,9 +269,10 @@ class KernelSet(ABC):
         its page (if ``kv``) and q to ``q_out [T, heads * head_dim]`` in the set's dtype.  All arithmetic float32."""
         raise NotImplementedError
 
-    def activation(self, x, kind: str = "silu", scale: float = 1.0, scaled_columns: int = 0):
-        """A float32 matrix ``[T, n]`` out of ``x`` (float32, any row stride, or slices): ``act(x)`` with ``kind``
-        ``"silu"`` or ``"none"``, the first ``scaled_columns`` columns also times ``scale``."""
+    def activation(self, x, kind: str = "silu", scale: float = 1.0, scaled_columns: int = 0, out_dtype=None):
+        """A matrix ``[T, n]`` (float32, or of ``out_dtype``) out of ``x`` (float32, any row stride, or slices):
+        ``act(x)`` with ``kind`` ``"silu"``, ``"tanh"`` or ``"none"``, the first ``scaled_columns`` columns also times
+        ``scale``."""
         raise NotImplementedError
 
     def exp_gate_scan(self, log_in, log_forget, in_bias, forget_bias, cap: float, state, step: StepTensors):
@@ -262,7 +292,8 @@ class KernelSet(ABC):
         raise NotImplementedError
 
     def route_top(self, x, router, top: int, scoring: str = "sigmoid", groups: tuple[int, int] | None = None,
-                  weight_scale: float = 1.0, extra_rows: int = 0, correction=None, normalise: bool = False):
+                  weight_scale: float = 1.0, extra_rows: int = 0, correction=None, normalise: bool = False,
+                  logit_bias=None):
         """The ``top`` experts of every token: logits ``x @ router.T`` (``router [experts, hidden]``) accumulated in
         float32 -> ``(ids [T, top] int32, weights [T, top] float32)``, ``weights`` the chosen experts' scores
         (``sigmoid(logit)``, not renormalised) times ``weight_scale``, the largest first, ties to the lower index.
@@ -275,7 +306,9 @@ class KernelSet(ABC):
 
         ``scoring="softmax"``: the scores are a softmax over all experts' logits.  ``correction [experts]``
         (float32) is added to the scores for the choice only; the weights are the plain scores.  ``normalise``:
-        the chosen scores are divided by their sum (+ 1e-20) before ``weight_scale``."""
+        the chosen scores are divided by their sum (+ 1e-20) before ``weight_scale``.
+        ``scoring="softmax_chosen"``: the choice is made on the logits and the weights are the softmax over the chosen
+        logits alone.  ``logit_bias [experts]`` (float32) is part of the logits."""
         raise NotImplementedError
 
     def routed_swiglu(self, x, ids, weights, gate_up, down, scale_input: bool = True, limit: float | None = None,
@@ -297,9 +330,17 @@ class KernelSet(ABC):
         ``sigmoid(row_gate[t])``.  Returns ``[T, rows / 2]`` in the set's dtype."""
         raise NotImplementedError
 
-    def linear_act(self, x, weight, kind: str = "relu2"):
+    def linear_act(self, x, weight, kind: str = "relu2", numbers: tuple[float, float] | None = None):
         """``act(x @ weight.T)`` in the set's dtype, the activation applied to the float32 accumulators:
-        ``"relu2"`` is ``max(z, 0)^2``."""
+        ``"relu2"`` is ``max(z, 0)^2``; ``"gelu"`` is ``z (1 + erf(z / sqrt 2)) / 2``; ``"xielu"`` with ``numbers = (a,
+        b)`` is ``a z^2 + z / 2`` right of zero and ``b (exp(z) - 1 - z) + z / 2`` left of it."""
+        raise NotImplementedError
+
+    def routed_act(self, x, ids, weights, up, down, kind: str = "gelu", numbers: tuple[float, float] | None = None):
+        """Every token through its chosen experts of two matrices: ``up [experts, ff, hidden]``, ``down [experts,
+        hidden, ff]``; pair (t, j) with expert e computes ``weights[t, j] * down_e act(up_e x[t])`` (``kind`` and
+        ``numbers`` as in :meth:`linear_act`).  Returns float32 slices ``[top, T, hidden]`` whose sum over the first
+        axis is the routed output."""
         raise NotImplementedError
 
     # -- attention through a latent: one shared key/value row per token, queries folded into the latent's space ------
@@ -310,7 +351,8 @@ class KernelSet(ABC):
         ``q_latent_out [T, q_rank]`` in the set's dtype.  With ``kv`` the next ``kv_rank`` columns, normed the same
         way with ``kv_norm``, and the last ``rot_dim`` columns, rotated by ``rotary`` at the token's position and not
         normed, are stored side by side as the token's one row ``[kv_rank + rot_dim]`` of ``kv.k``.  All float32
-        up to the stores.  Without ``kv`` the projection has the query columns only."""
+        up to the stores.  Without ``kv`` the projection has the query columns only.  ``q_rank`` 0 (with ``q_norm`` and
+        ``q_latent_out`` None): there is no query latent and the projection starts with the ``kv_rank`` columns."""
         raise NotImplementedError
 
     def latent_queries(self, q, up_keys, step: StepTensors, rotary: RotaryTable | None, num_heads: int, dim: int,
@@ -356,13 +398,39 @@ class KernelSet(ABC):
         With ``num_heads`` the number of columns (``d = 1``) the gate is element by element."""
         raise NotImplementedError
 
-    def short_conv(self, x, weight, bias, state, step: StepTensors, activation: str = "silu", input_bias=None):
+    def short_conv(self, x, weight, bias, state, step: StepTensors, activation: str = "silu", input_bias=None, typed: bool = False):
         """Causal convolution over time, per channel and per request: ``x [T, C]`` float32 (any row stride; or slices),
         ``weight [C, taps]`` whose last column multiplies the current token, ``state [seats, taps - 1, C]`` the
         request's last inputs (oldest first; zeros at a request's start), which the call moves on by the
         step's tokens.  Returns float32 ``[T, C]`` after the activation (``"silu"`` or ``"none"``).  ``input_bias [C]``
         (float32) is added to every input of the step before anything else (the state holds the sums; before a
-        request's start the inputs are zeros, not the bias)."""
+        request's start the inputs are zeros, not the bias).  ``typed``: returns a pair, the same values
+        in the set's dtype as the second, for a product that reads them."""
+        raise NotImplementedError
+
+    # -- recurrences whose decay varies by channel ------------------------------------------------------------------
+    def selective_scan(self, x, dt, B, C, gate, rates, skip, dt_bias, state, step: StepTensors, out) -> None:
+        """A diagonal state per channel and request, moved on token by token in float32: with ``d =
+        softplus(dt[t, c] + dt_bias[c])``
+
+        ``S[n, c] <- exp(d rates[n, c]) S[n, c] + d x[t, c] B[t, n]``;
+        ``out[t, c] = (sum_n S[n, c] C[t, n] + skip[c] x[t, c]) * silu(gate[t, c])`` in the set's dtype.
+
+        ``x [T, channels]``, ``dt, gate [T, channels]`` and ``B, C [T, states]`` float32 (any row stride; ``dt``, ``B``,
+        ``C`` and ``gate`` or slices; ``B`` and ``C`` are views of one projection), ``rates [states, channels]`` the
+        (negative) rates of decay, ``state [seats, states, channels]`` float32, read and written through each token's
+        seat."""
+        raise NotImplementedError
+
+    def channel_delta(self, proj, decay, decay_bias, rate_bias, state, step: StepTensors, heads: int, dim: int):
+        """A matrix state ``S [dim, dim]`` per head and request with a decay and a removal rate per key channel:
+
+        ``S <- diag(w) S - (a * u) (u^T S) + k v^T`` (the old S on the right), ``o = S^T r``, ``u = k / sqrt(sum(k^2) +
+        1e-6)``, ``w = exp(-exp(-1/2) sigmoid(decay + decay_bias))``, ``a = sigmoid(rate + rate_bias)``.
+
+        ``proj [T, 4 * heads * dim (+ more)]`` float32 (or slices) holds ``[r | k | v | rate]``, each head by head;
+        ``decay [T, heads * dim]`` float32 (or slices); the biases ``[heads * dim]``; ``state [seats, heads, dim, dim]``
+        float32 (S transposed: value element, then key channel).  Returns float32 ``[T, heads * dim]``."""
         raise NotImplementedError
 
     def linear_recurrence(self, rule: str, q, k, v, decay, write, state, step: StepTensors, heads: int, groups: int,

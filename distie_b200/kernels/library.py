@@ -37,6 +37,7 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
         "base", [P, I, I, L, P, P, I, P, P, P, P, I, P, F, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, F, F, I, P, P]
     ),
     "distie_norm_add_rmsnorm": ("base", [P, P, I, P, F, P, P, F, P, P, I, I, I, P]),
+    "distie_average_add_rmsnorm": ("base", [P, P, I, P, F, P, P, L, I, I, P, P, F, P, P, I, I, I, P]),
     "distie_qk_rope_norm_write": (
         "base", [P, I, I, L, P, P, I, P, P, P, P, I, P, F, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P]
     ),
@@ -60,23 +61,30 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     "distie_kv_write": ("state", [P, I, P, I, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, P, P]),
     "distie_head_gate": ("state", [P, P, I, I, L, I, I, I, I, P]),
     "distie_seq_index": ("state", [P, I, I, P, P, P]),
-    "distie_short_conv": ("state", [P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P, P, P]),
+    "distie_short_conv": ("state", [P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P, P, P, P]),
     "distie_linear_recurrence": (
         "state", [I, P, I, P, I, P, I, P, I, P, I, I, L, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, P]
     ),
-    "distie_activation": ("state", [P, I, I, L, P, I, I, I, F, I, P]),
+    "distie_activation": ("state", [P, I, I, L, P, I, I, I, F, I, I, P]),
+    "distie_selective_scan": (
+        "state", [P, I, P, I, I, L, P, P, I, I, L, P, I, I, L, P, P, P, P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, P]
+    ),
+    "distie_selective_scan_scratch_floats": ("state", [I, I, I]),
+    "distie_channel_delta": ("state", [P, I, I, L, P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P]),
+    "distie_channel_delta_scratch_floats": ("state", [I, I, I]),
     "distie_exp_gate_scan": ("state", [P, P, I, I, L, P, P, F, P, P, P, I, I, I, P, P, P, P]),
     "distie_stabilized_readout": ("state", [P, I, P, P, I, I, I, P]),
-    "distie_route_top": ("routed", [P, I, P, I, I, I, I, P, P, I, I, F, I, P, I, P, I, I, P]),
-    "distie_route_pick": ("routed", [P, I, I, I, I, P, P, I, I, F, I, P, I, P]),
+    "distie_route_top": ("routed", [P, I, P, I, I, I, I, P, P, I, I, F, I, P, I, P, I, P, I, P]),
+    "distie_route_pick": ("routed", [P, I, I, I, I, P, P, I, I, F, I, P, I, P, P]),
     "distie_routed_identity": ("routed", [P, I, P, P, I, I, I, P, I, I, P]),
     "distie_routed_tile": ("routed", [I, I, I, I, I]),
     "distie_route_plan_words": ("routed", [I, I, I]),
     "distie_route_plan": ("routed", [P, P, I, I, I, I, P, P, I, P]),
     "distie_routed_gather": ("routed", [P, I, P, I, I, I, P, I, I, I, P]),
     "distie_routed_scatter": ("routed", [P, P, I, I, I, P, I, I, P]),
-    "distie_gemm_tcgen05_grouped": ("bf16", [P, I, I, P, I, I, P, I, I, I, I, F, P, P, P, P, I, I, P, P]),
+    "distie_gemm_tcgen05_grouped": ("bf16", [P, I, I, P, I, I, P, I, I, I, I, F, I, F, F, P, P, P, P, I, I, P, P]),
     "distie_routed_swiglu": ("routed", [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P]),
+    "distie_routed_act": ("routed", [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, P, P]),
     "distie_latent_kv_write": (
         "latent", [P, I, I, L, I, P, I, P, I, F, P, I, P, P, P, P, I, P, F, I, I, P, I, I, I, I, I, P, P]
     ),
@@ -87,15 +95,18 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     "distie_latent_merge": ("latent", [P, P, I, I, I, I, P, I, I, I, P]),
     "distie_latent_attention_tiles": ("latent", [P, P, P, I, I, I, I, P, I, P, P, P, P, I, P, I, I, F, P, P, P]),
     "distie_latent_gate": ("latent", [P, I, I, I, P, I, I, L, P, I, I, P]),
-    "distie_glu_act": ("latent", [P, I, I, L, I, I, I, F, P, I, I, L, P, I, I, P]),
+    "distie_glu_act": ("latent", [P, I, I, L, I, I, I, F, F, F, P, I, I, L, P, I, I, P]),
     "distie_gated_rmsnorm": ("state", [P, I, P, I, I, L, P, I, P, I, I, I, I, F, I, I, P]),
     "distie_gemm_tcgen05": ("bf16", [P, I, P, P, I, I, I, I, I, I, I, P, P]),
+    "distie_gemm_tcgen05_act": ("bf16", [P, I, P, P, I, I, I, I, I, I, I, F, F, I, P, P]),
     "distie_gemm_tcgen05_qkv": ("bf16", [P, I, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, P, P]),
     "distie_gemm_tcgen05_skinny_splits": ("bf16", [I, I, I]),
+    "distie_gemm_tcgen05_skinny_act": ("bf16", [P, I, P, P, I, I, I, I, I, F, F, I, P, P]),
     "distie_gemm_tcgen05_skinny": ("bf16", [P, I, P, P, P, I, I, I, I, I, I, I, P, P]),
 }
 _RESULT = {"distie_attention_decode_scratch_floats": c_longlong, "distie_route_plan_words": c_longlong,
-           "distie_latent_attention_scratch_floats": c_longlong}
+           "distie_latent_attention_scratch_floats": c_longlong, "distie_selective_scan_scratch_floats": c_longlong,
+           "distie_channel_delta_scratch_floats": c_longlong}
 
 _libraries: dict[str, ctypes.CDLL] = {}
 _functions: dict[str, object] = {}

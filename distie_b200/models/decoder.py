@@ -17,6 +17,7 @@ import torch
 from ..config.model_spec import ModelSpec
 from ..kernels.interface import KernelSet, KvSlot, StepTensors
 from ..parts.base import BLOCKS, MIXERS, NORMS, BuildContext, CacheNeed, LayerRun, ResidualStream, StateNeed, TensorSpec, build_part
+from ..parts.depth import DepthAverage
 from ..parts.linear import Linear
 
 
@@ -27,6 +28,7 @@ def model_tensor_specs(spec: ModelSpec) -> list[TensorSpec]:
         specs += NORMS.get(spec.embedding_norm.kind).tensor_specs(spec.embedding_norm, spec.hidden_size)
     for layer in spec.layers:
         specs += BLOCKS.get(layer.block).tensor_specs(layer, spec.hidden_size)
+    specs += DepthAverage.tensor_specs(spec)
     specs += NORMS.get(spec.final_norm.kind).tensor_specs(spec.final_norm, spec.hidden_size)
     if spec.head_name is not None:
         specs.append(TensorSpec(spec.head_name, (spec.vocab_size, spec.hidden_size), "table"))
@@ -65,6 +67,7 @@ class DecoderModel:
         self.embedding = weights.table(spec.embedding_name)
         self.embedding_norm = build_part(NORMS, spec.embedding_norm, ctx) if spec.embedding_norm is not None else None
         self.blocks = [BLOCKS.get(layer.block).build(layer, ctx) for layer in spec.layers]
+        self.average = DepthAverage.build(spec, ctx) if spec.depth_averaged else None
         self.final_norm = build_part(NORMS, spec.final_norm, ctx)
         head = self.embedding if spec.head_name is None else weights.table(spec.head_name)
         self.head = Linear(head, None, kernels)
@@ -90,6 +93,7 @@ class DecoderModel:
                         visit(value)
 
         visit(self.blocks)
+        visit(self.average)
         visit(self.final_norm)
         visit(self.embedding_norm)
         visit(self.head)
@@ -107,7 +111,9 @@ class DecoderModel:
             # first block's norm kernel does both norms in one pass.
             stream = ResidualStream(torch.zeros_like(residual), self.embedding_norm.pending(residual))
             residual = stream.residual
-        for call in self.spec.order:
+        if self.average is not None:
+            self.average.start(stream)
+        for index, call in enumerate(self.spec.order):
             run = LayerRun(
                 step=step,
                 seqs=seqs,
@@ -116,6 +122,8 @@ class DecoderModel:
                 writes_cache=call.writes_cache,
             )
             self.blocks[call.layer].forward(stream, run)
+            if self.average is not None:
+                self.average.after(index, stream)
         if logit_rows is None or logit_rows.numel() == 0:
             return None
         x = torch.empty((logit_rows.numel(), self.spec.hidden_size), dtype=k.dtype, device=k.device)

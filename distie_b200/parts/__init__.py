@@ -9,6 +9,7 @@ from .base import (
     Branches,
     BuildContext,
     CacheNeed,
+    FreeSize,
     LayerRun,
     ResidualStream,
     SeqSlice,
@@ -16,7 +17,7 @@ from .base import (
     TensorSpec,
     build_part,
 )
-from . import attention, block, hybrid, latent, memory, mlp, norm, position, recurrent, routed  # noqa: F401  (register the built-in kinds)
+from . import attention, block, channelwise, hybrid, latent, memory, mlp, norm, position, recurrent, routed  # noqa: F401  (register the built-in kinds)
 
 __all__ = [
     "BLOCKS",
@@ -27,6 +28,7 @@ __all__ = [
     "Branches",
     "BuildContext",
     "CacheNeed",
+    "FreeSize",
     "LayerRun",
     "ResidualStream",
     "SeqSlice",

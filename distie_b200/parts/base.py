@@ -32,10 +32,19 @@ from typing import Any, Callable, Sequence
 import torch
 
 from ..config.model_spec import PartSpec
-from ..kernels.interface import KernelSet, KvSlot, Normed, StepTensors, Terms
+from ..kernels.interface import Averaged, KernelSet, KvSlot, Normed, StepTensors, Terms
 
 
 # -- what parts declare --------------------------------------------------------
+@dataclass(frozen=True)
+class FreeSize:
+    """A size that no configuration gives: the checkpoint decides it.  Tensors whose shapes name the same ``key`` agree
+    on it; a model with random weights gets ``default``."""
+
+    key: str
+    default: int
+
+
 @dataclass(frozen=True)
 class TensorSpec:
     """A tensor a part reads from the checkpoint.  ``role`` decides conversion and random init:
@@ -45,11 +54,17 @@ class TensorSpec:
     ``bias``    vector added to a product (kept in float32 on the device)
     ``norm``    scale of a norm (float32 on the device; random mode writes ones)
     ``norm0``   scale of a norm that is stored around zero (the norm multiplies by 1 + it; random mode writes zeros)
+    ``average`` weights of a sum over states (float32 on the device; random mode favours the last of them)
     """
 
     name: str
-    shape: tuple[int, ...]
+    shape: tuple[int | FreeSize, ...]
     role: str = "matrix"
+
+    @property
+    def default_shape(self) -> tuple[int, ...]:
+        """The shape with the defaults of its free sizes."""
+        return tuple(n.default if isinstance(n, FreeSize) else n for n in self.shape)
 
 
 @dataclass(frozen=True)
@@ -137,6 +152,11 @@ class ResidualStream:
         self.pending = pending
 
     def settle(self) -> torch.Tensor:
+        if isinstance(self.pending, Averaged):  # a layer's end: its result joins the states, the residual becomes their average
+            ahead = self.pending
+            state = ResidualStream(self.residual.clone(), ahead.value).settle()
+            self.residual.copy_(ahead.close(state))
+            self.pending = None
         if isinstance(self.pending, Normed):  # a sublayer's output that joins the residual through a norm
             value = ResidualStream(torch.zeros_like(self.residual), self.pending.value).settle()
             unit = value * torch.rsqrt((value * value).mean(-1, keepdim=True) + self.pending.eps)

@@ -21,7 +21,10 @@ of one token and a portion of a prompt run the same ops.
 A layer with ``own_latent=False`` has no ``W_dkv``: it reads the rows that the owner of its cache slot stored
 (after that layer's norm and rotation), with its own ``W_uk``, ``W_uv``, queries, sink, gate and output.
 
-The projections that read ``h`` (``W_dq``, ``W_dkv``, ``W_g``) are one product against the row-stacked weight;
+Without a query latent (``q_rank`` None) the queries come straight from the input, ``q = W_q h``; the sink and the gate
+are options too.
+
+The projections that read ``h`` (``W_dq`` or ``W_q``, ``W_dkv``, ``W_g``) are one product against the row-stacked weight;
 both norms, the rotation of ``r`` and the store of the cache row are one op on its float32 accumulators.
 """
 
@@ -37,16 +40,17 @@ from .linear import fuse_rows
 @MIXERS.register("latent_attention")
 class LatentAttention:
     """params: ``num_heads``, ``head_dim`` (plain query/key dimensions per head), ``rot_dim``, ``value_dim``,
-    ``kv_rank``, ``q_rank``, ``scale``, ``eps`` (of the two latent norms), ``position`` (a PartSpec; its table
+    ``kv_rank``, ``q_rank`` (None: no query latent), ``scale``, ``eps`` (of the latent norms), ``position`` (a PartSpec; its table
     rotates the ``rot_dim`` part), ``sink`` (bool), ``gate`` (None or ``"head_sigmoid"``), ``own_latent`` (bool),
     ``names`` (what the tensors' names add to the prefix).
 
-    tensors: ``dq [q_rank, hidden]``, ``dq.norm [q_rank]``, ``uq [heads * (head_dim + rot_dim), q_rank]``,
+    tensors: ``dq [q_rank, hidden]``, ``dq.norm [q_rank]``, ``uq [heads * (head_dim + rot_dim), q_rank]`` (or, without a
+    query latent, ``q [heads * (head_dim + rot_dim), hidden]``),
     ``dkv [kv_rank + rot_dim, hidden]`` and ``dkv.norm [kv_rank]`` (with a latent of its own),
     ``uk [heads * head_dim, kv_rank]``, ``uv [heads * value_dim, kv_rank]``, ``sink [heads]``,
     ``g [heads, hidden]``, ``o [hidden, heads * value_dim]``."""
 
-    _NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk",
+    _NAMES = {"q": "q", "dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk",
               "uv": "uv", "sink": "sink", "g": "g", "o": "o"}
 
     def __init__(self, prm: dict, kernels, position, down, q_norm, kv_norm, up_q, up_keys, up_values, sink, out) -> None:
@@ -57,7 +61,7 @@ class LatentAttention:
         self.rot_dim = int(prm["rot_dim"])
         self.value_dim = int(prm["value_dim"])
         self.kv_rank = int(prm["kv_rank"])
-        self.q_rank = int(prm["q_rank"])
+        self.q_rank = int(prm["q_rank"]) if prm["q_rank"] is not None else None
         self.scale = float(prm["scale"])
         self.eps = float(prm["eps"])
         self.own_latent = bool(prm.get("own_latent", True))
@@ -73,7 +77,7 @@ class LatentAttention:
     @staticmethod
     def _check(prm) -> None:
         for key in ("num_heads", "head_dim", "value_dim", "kv_rank", "q_rank"):
-            if int(prm[key]) < 1:
+            if (key != "q_rank" or prm[key] is not None) and int(prm[key]) < 1:
                 raise ValueError(f"{key} must be >= 1, got {prm[key]}")
         if int(prm["rot_dim"]) < 0:
             raise ValueError(f"rot_dim must be >= 0, got {prm['rot_dim']}")
@@ -88,12 +92,15 @@ class LatentAttention:
         cls._check(spec.params)
         prm = spec.params
         heads, dim, rot, vdim = int(prm["num_heads"]), int(prm["head_dim"]), int(prm["rot_dim"]), int(prm["value_dim"])
-        rank, q_rank = int(prm["kv_rank"]), int(prm["q_rank"])
-        specs = [
-            TensorSpec(cls._name(spec, "dq"), (q_rank, hidden_size)),
-            TensorSpec(cls._name(spec, "dq_norm"), (q_rank,), "norm"),
-            TensorSpec(cls._name(spec, "uq"), (heads * (dim + rot), q_rank)),
-        ]
+        rank, q_rank = int(prm["kv_rank"]), prm["q_rank"]
+        if q_rank is None:
+            specs = [TensorSpec(cls._name(spec, "q"), (heads * (dim + rot), hidden_size))]
+        else:
+            specs = [
+                TensorSpec(cls._name(spec, "dq"), (int(q_rank), hidden_size)),
+                TensorSpec(cls._name(spec, "dq_norm"), (int(q_rank),), "norm"),
+                TensorSpec(cls._name(spec, "uq"), (heads * (dim + rot), int(q_rank))),
+            ]
         if prm.get("own_latent", True):
             specs += [TensorSpec(cls._name(spec, "dkv"), (rank + rot, hidden_size)),
                       TensorSpec(cls._name(spec, "dkv_norm"), (rank,), "norm")]
@@ -122,8 +129,9 @@ class LatentAttention:
         prm, w = spec.params, ctx.weights
         heads, dim, vdim, rank = int(prm["num_heads"]), int(prm["head_dim"]), int(prm["value_dim"]), int(prm["kv_rank"])
         own = bool(prm.get("own_latent", True))
-        # Everything that reads the mixer's input, row-stacked: query latent, (key/value latent, key part), gates.
-        stacked = [w.matrix(cls._name(spec, "dq"))]
+        # Everything that reads the mixer's input, row-stacked: queries or their latent, (key/value latent, key part), gates.
+        direct = prm["q_rank"] is None
+        stacked = [w.matrix(cls._name(spec, "q" if direct else "dq"))]
         if own:
             stacked.append(w.matrix(cls._name(spec, "dkv")))
         if prm.get("gate"):
@@ -133,8 +141,8 @@ class LatentAttention:
         up_values = w.matrix(cls._name(spec, "uv")).reshape(heads, vdim, rank).transpose(1, 2).contiguous()  # [h, rank, vdim]
         return cls(
             dict(prm), ctx.kernels, position, fuse_rows(stacked),
-            w.vector(cls._name(spec, "dq_norm")), w.vector(cls._name(spec, "dkv_norm")) if own else None,
-            w.matrix(cls._name(spec, "uq")), up_keys, up_values,
+            None if direct else w.vector(cls._name(spec, "dq_norm")), w.vector(cls._name(spec, "dkv_norm")) if own else None,
+            None if direct else w.matrix(cls._name(spec, "uq")), up_keys, up_values,
             w.vector(cls._name(spec, "sink")) if prm.get("sink") else None, w.matrix(cls._name(spec, "o")),
         )
 
@@ -147,11 +155,18 @@ class LatentAttention:
         k = self.kernels
         tokens = x.shape[0]
         table = self.position.rotary_table()
-        proj = k.linear_split(x, self.down)  # float32 [S, T, q_rank (+ kv_rank + rot_dim) (+ heads)]
-        q_latent = torch.empty((tokens, self.q_rank), dtype=x.dtype, device=x.device)
-        k.latent_kv_write(proj, run.step, run.kv if self.own_latent else None, table, self.q_rank, self.q_norm,
-                          self.kv_rank, self.kv_norm, self.rot_dim, self.eps, q_latent)
-        q = k.linear(q_latent, self.up_q, None, torch.float32)
+        proj = k.linear_split(x, self.down)  # float32 [S, T, q_rank or all queries (+ kv_rank + rot_dim) (+ heads)]
+        if self.q_rank is None:
+            columns = self.num_heads * (self.head_dim + self.rot_dim)
+            q = proj[..., :columns]
+            if self.own_latent:
+                k.latent_kv_write(proj[..., columns:], run.step, run.kv, table, 0, None, self.kv_rank, self.kv_norm,
+                                  self.rot_dim, self.eps, None)
+        else:
+            q_latent = torch.empty((tokens, self.q_rank), dtype=x.dtype, device=x.device)
+            k.latent_kv_write(proj, run.step, run.kv if self.own_latent else None, table, self.q_rank, self.q_norm,
+                              self.kv_rank, self.kv_norm, self.rot_dim, self.eps, q_latent)
+            q = k.linear(q_latent, self.up_q, None, torch.float32)
         folded, rotated = k.latent_queries(q, self.up_keys, run.step, table, self.num_heads, self.head_dim, self.rot_dim)
         mixed = torch.empty((self.num_heads, tokens, self.kv_rank), dtype=x.dtype, device=x.device)
         k.latent_attention(folded, rotated, run.step, run.kv, self.num_heads, self.kv_rank, self.rot_dim, self.scale,

@@ -7,6 +7,8 @@ up are one product against the row-stacked weight ``[2 * inter, hidden]``.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..config.model_spec import PartSpec
@@ -54,39 +56,55 @@ class SwiGluFeedForward:
         return self.kernels.linear_split(self.kernels.linear_swiglu(x, self.gate_up.weight), self.down.weight)
 
 
+def _softplus(z: float) -> float:
+    return max(z, 0.0) + math.log1p(math.exp(-abs(z)))
+
+
 @FEED_FORWARDS.register("activated")
 class ActivatedFeedForward:
     """``down(act(up(x)))`` with the activation on the product's float32 accumulators.  params:
-    ``intermediate_size``, ``activation`` (``"relu2"``: the square of ReLU); optional ``names``: what the names of
-    the up and down matrices add to the prefix (default ``up_proj.weight``, ``down_proj.weight``)."""
+    ``intermediate_size``, ``activation`` (``"relu2"``: the square of ReLU; ``"gelu"``: the exact one; ``"xielu"``: a
+    parabola right of zero and an exponential left of it, see :meth:`KernelSet.linear_act`); optional ``names``: what
+    the names of the up and down matrices add to the prefix (default ``up_proj.weight``, ``down_proj.weight``);
+    ``numbers`` (xielu): what the name of its two learned numbers ``[p, q]`` adds to the prefix, whose factors are
+    ``softplus(p)`` and ``1/2 + softplus(q)``."""
 
     _NAMES = ("up_proj.weight", "down_proj.weight")
-    _ACTIVATIONS = ("relu2",)
+    _ACTIVATIONS = ("relu2", "gelu", "xielu")
 
-    def __init__(self, up: torch.Tensor, down: torch.Tensor, activation: str, kernels) -> None:
-        self.up, self.down, self.activation, self.kernels = up, down, activation, kernels
+    def __init__(self, up: torch.Tensor, down: torch.Tensor, activation: str, kernels, numbers=None) -> None:
+        self.up, self.down, self.activation, self.kernels, self.numbers = up, down, activation, kernels, numbers
 
     @classmethod
     def _check(cls, spec: PartSpec) -> None:
         if spec.params.get("activation") not in cls._ACTIVATIONS:
             raise ValueError(f"activation {spec.params.get('activation')!r}: one of {cls._ACTIVATIONS}")
+        if (spec.params["activation"] == "xielu") != bool(spec.params.get("numbers")):
+            raise ValueError("xielu, and no other activation, has two learned numbers")
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, hidden_size: int) -> list[TensorSpec]:
         cls._check(spec)
         p, inter = spec.prefix, int(spec.params["intermediate_size"])
         up, down = spec.params.get("names", cls._NAMES)
-        return [TensorSpec(p + up, (inter, hidden_size)), TensorSpec(p + down, (hidden_size, inter))]
+        specs = [TensorSpec(p + up, (inter, hidden_size)), TensorSpec(p + down, (hidden_size, inter))]
+        if spec.params.get("numbers"):
+            specs.append(TensorSpec(p + spec.params["numbers"], (2,), "bias"))
+        return specs
 
     @classmethod
     def build(cls, spec: PartSpec, ctx: BuildContext) -> "ActivatedFeedForward":
         cls._check(spec)
         p, w = spec.prefix, ctx.weights
         up, down = spec.params.get("names", cls._NAMES)
-        return cls(w.matrix(p + up), w.matrix(p + down), spec.params["activation"], ctx.kernels)
+        numbers = None
+        if spec.params.get("numbers"):
+            right, left = w.vector(p + spec.params["numbers"]).double().tolist()
+            numbers = (_softplus(right), 0.5 + _softplus(left))
+        return cls(w.matrix(p + up), w.matrix(p + down), spec.params["activation"], ctx.kernels, numbers)
 
     def forward(self, x: torch.Tensor, run: LayerRun) -> torch.Tensor:
-        return self.kernels.linear_split(self.kernels.linear_act(x, self.up, self.activation), self.down)
+        return self.kernels.linear_split(self.kernels.linear_act(x, self.up, self.activation, self.numbers), self.down)
 
 
 @FEED_FORWARDS.register("none")

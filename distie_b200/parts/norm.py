@@ -12,7 +12,7 @@ squared deviations, all in float32 up to the store.
 from __future__ import annotations
 
 from ..config.model_spec import PartSpec
-from ..kernels.interface import Normed, Terms
+from ..kernels.interface import Averaged, Normed, Terms
 from .base import NORMS, BuildContext, TensorSpec
 
 
@@ -20,8 +20,9 @@ from .base import NORMS, BuildContext, TensorSpec
 class RMSNorm:
     """params: ``eps``; optional ``name`` (what the tensor's name adds to the prefix, default ``"weight"``),
     ``offset`` (added to the stored scale; 0 when the checkpoint stores the scale itself) and ``exact`` (the norm
-    is float32 up to the one cast of its output, scale included; an offset implies it).
-    tensors: ``<prefix><name> [hidden]``."""
+    is float32 up to the one cast of its output, scale included; an offset implies it) and ``times`` (the name of a
+    second vector that multiplies the norm's output element by element, as a layer scale does; implies ``exact``).
+    tensors: ``<prefix><name> [hidden]``, ``<prefix><times> [hidden]``."""
 
     def __init__(self, weight, eps: float, kernels, exact: bool = False) -> None:
         self.weight = weight
@@ -32,7 +33,10 @@ class RMSNorm:
     @classmethod
     def tensor_specs(cls, spec: PartSpec, hidden_size: int) -> list[TensorSpec]:
         role = "norm0" if float(spec.params.get("offset", 0.0)) else "norm"
-        return [TensorSpec(spec.prefix + spec.params.get("name", "weight"), (hidden_size,), role)]
+        specs = [TensorSpec(spec.prefix + spec.params.get("name", "weight"), (hidden_size,), role)]
+        if spec.params.get("times"):
+            specs.append(TensorSpec(spec.prefix + spec.params["times"], (hidden_size,), "norm"))
+        return specs
 
     @classmethod
     def build(cls, spec: PartSpec, ctx: BuildContext) -> "RMSNorm":
@@ -40,7 +44,10 @@ class RMSNorm:
         offset = float(spec.params.get("offset", 0.0))
         if offset:
             weight = weight + offset  # float32: exact for a scale stored in 16 bits, up to float32 rounding
-        return cls(weight, spec.params["eps"], ctx.kernels, exact=bool(offset) or bool(spec.params.get("exact")))
+        times = spec.params.get("times")
+        if times:
+            weight = weight * ctx.weights.vector(spec.prefix + times)
+        return cls(weight, spec.params["eps"], ctx.kernels, exact=bool(offset) or bool(times) or bool(spec.params.get("exact")))
 
     def pending(self, value) -> Normed:
         """``value`` (a sublayer's output) as something the next norm adds to the residual through this norm."""
@@ -48,6 +55,9 @@ class RMSNorm:
 
     def apply(self, delta, residual, out, rows=None) -> None:
         """``residual += delta`` (if any), ``out = norm(residual)``; with ``rows`` only those rows, residual kept."""
+        if isinstance(delta, Averaged):
+            self._after_average(delta, residual, out, rows)
+            return
         if isinstance(delta, Normed):
             self.kernels.norm_add_rmsnorm(delta.value, delta.weight, delta.eps, residual, self.weight, self.eps, out, rows)
             return
@@ -57,6 +67,13 @@ class RMSNorm:
         if isinstance(delta, Terms):
             delta = delta.total()
         self.kernels.add_rmsnorm(delta, residual, self.weight, self.eps, out, rows)
+
+
+    def _after_average(self, ahead: Averaged, residual, out, rows) -> None:
+        """Behind a layer whose states are averaged over depth: average and norm in one kernel."""
+        if not self.exact:
+            raise ValueError("a norm behind a depth average is float32 up to one cast: set exact (or an offset)")
+        self.kernels.average_add_rmsnorm(ahead, residual, self.weight, self.eps, out, rows)
 
 
 @NORMS.register("layernorm")
@@ -86,4 +103,7 @@ class LayerNorm:
 
     def apply(self, delta, residual, out, rows=None) -> None:
         """``residual += delta`` (if any; a :class:`Terms` is summed in the kernel), ``out = norm(residual)``."""
+        if isinstance(delta, Averaged):  # the average moves the residual on by itself; the norm then reads it
+            self.kernels.average_add_rmsnorm(delta, residual, None, 0.0, None)
+            delta = None
         self.kernels.add_layernorm(delta, residual, self.weight, self.bias, self.eps, out, rows)

@@ -1,4 +1,4 @@
-"""Routed feed-forward: every token goes through a few of many small gated experts, and through a shared one.
+"""Routed feed-forwards: every token goes through a few of many small experts, and perhaps through a shared one.
 
 ``routed_swiglu``: router scores ``s = sigmoid(W_router h)`` from float32 logits; the ``top`` experts with the
 largest scores are chosen (ties to the lower index) and weighted by their scores as they are (times
@@ -14,6 +14,10 @@ softmax over all router outputs; ``correction`` names a vector (``[router output
 the choice only; ``normalise`` divides the chosen scores by their sum (+ 1e-20); with ``identity = n`` the router has
 ``n`` more outputs than there are experts, which stand for experts without tensors that return their input.  The output stays a sum still to be done
 (the routed slices and the shared expert's), which the norm kernel that follows adds up.
+
+``routed_activated``: experts of two matrices, ``down(act(up h))``, no shared one.  The router's float32 logits may have
+a bias; with ``scoring="softmax_chosen"`` the ``top`` largest logits choose and the weights, on the experts' outputs,
+are the softmax over the chosen logits alone.
 """
 
 from __future__ import annotations
@@ -151,3 +155,55 @@ class RoutedSwiGlu:
         # tokens, where each is a chain of short kernels, they run side by side.
         both = Branches.run([routed, shared], x.shape[0], x.device)
         return Terms.of(both[0]) + Terms.of(both[1])
+
+
+@FEED_FORWARDS.register("routed_activated")
+class RoutedActivated:
+    """params: ``experts``, ``top``, ``intermediate_size``, ``activation`` (``"gelu"`` or ``"relu2"``), optional ``scoring``
+    (``"softmax_chosen"``, default, ``"sigmoid"`` or ``"softmax"``) and ``router_bias`` (None, or the name of the vector
+    added to the logits).
+    tensors (prefix +): ``router [experts, hidden]``, ``<router_bias> [experts]``, ``e<j>.up [ff, hidden]``,
+    ``e<j>.down [hidden, ff]``."""
+
+    graph_safe = True
+
+    def __init__(self, router, router_bias, up, down, prm: dict, kernels) -> None:
+        self.router, self.router_bias, self.up, self.down, self.kernels = router, router_bias, up, down, kernels
+        self.top = int(prm["top"])
+        self.activation = prm["activation"]
+        self.scoring = prm.get("scoring", "softmax_chosen")
+
+    @staticmethod
+    def _check(prm) -> None:
+        experts, top = int(prm["experts"]), int(prm["top"])
+        if experts < 1 or not 1 <= top <= min(experts, 32):
+            raise ValueError(f"experts {experts}, top {top}: 1 <= top <= min(experts, 32)")
+        if prm["activation"] not in ("gelu", "relu2"):
+            raise ValueError(f"activation {prm['activation']!r}: 'gelu' or 'relu2'")
+        if prm.get("scoring", "softmax_chosen") not in ("softmax_chosen", "sigmoid", "softmax"):
+            raise ValueError(f"scoring {prm['scoring']!r}: 'softmax_chosen', 'sigmoid' or 'softmax'")
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, hidden_size: int) -> list[TensorSpec]:
+        cls._check(spec.params)
+        p, prm = spec.prefix, spec.params
+        experts, ff = int(prm["experts"]), int(prm["intermediate_size"])
+        specs = [TensorSpec(p + "router", (experts, hidden_size))]
+        if prm.get("router_bias"):
+            specs.append(TensorSpec(p + prm["router_bias"], (experts,), "bias"))
+        for e in range(experts):
+            specs += [TensorSpec(f"{p}e{e}.up", (ff, hidden_size)), TensorSpec(f"{p}e{e}.down", (hidden_size, ff))]
+        return specs
+
+    @classmethod
+    def build(cls, spec: PartSpec, ctx: BuildContext) -> "RoutedActivated":
+        cls._check(spec.params)
+        p, prm, w = spec.prefix, spec.params, ctx.weights
+        up, down = (torch.stack([w.matrix(f"{p}e{e}.{n}") for e in range(int(prm["experts"]))]).contiguous() for n in ("up", "down"))
+        bias = w.vector(p + prm["router_bias"]) if prm.get("router_bias") else None
+        return cls(w.matrix(p + "router"), bias, up, down, dict(prm), ctx.kernels)
+
+    def forward(self, x: torch.Tensor, run: LayerRun):
+        k = self.kernels
+        ids, weights = k.route_top(x, self.router, self.top, self.scoring, logit_bias=self.router_bias)
+        return Terms.of(k.routed_act(x, ids, weights, self.up, self.down, self.activation))

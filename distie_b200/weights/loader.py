@@ -17,7 +17,7 @@ Conversion on the way to the device:
   is a float32 checkpoint and is cast; in a checkpoint that stores matrices in
   16-bit, one stored in 32-bit was kept wide on purpose and stays so (its products
   then run in float32).  ``"keep"``: 32-bit tensors always stay; ``"cast"``: never.
-* ``bias`` / ``norm``: float32 (exact for bfloat16 inputs): stored in 32-bit they stay so.
+* ``bias`` / ``norm`` / ``average``: float32 (exact for bfloat16 inputs): stored in 32-bit they stay so.
 * integer tensors: int32.
 """
 
@@ -28,7 +28,7 @@ from typing import Iterable, Mapping
 
 import torch
 
-from ..parts.base import TensorSpec
+from ..parts.base import FreeSize, TensorSpec
 from .safetensors_io import ModelTensors
 
 
@@ -74,11 +74,20 @@ def check_checkpoint(
     missing = [name for name in wanted if name not in shapes]
     allowed = set(tolerated)
     unexpected = sorted(name for name in shapes if name not in wanted and name not in allowed)
-    wrong = [
-        (name, shapes[name], spec.shape)
-        for name, spec in wanted.items()
-        if name in shapes and tuple(shapes[name]) != tuple(spec.shape)
-    ]
+    # Sizes that the checkpoint decides: the first tensor that has one settles it for the others.
+    free: dict[str, int] = {}
+    wrong = []
+    for name, spec in wanted.items():
+        if name not in shapes:
+            continue
+        have = tuple(shapes[name])
+        if len(have) == len(spec.shape):
+            for n, size in zip(spec.shape, have):
+                if isinstance(n, FreeSize) and size >= 1:
+                    free.setdefault(n.key, size)
+        want = tuple(free.get(n.key, "n") if isinstance(n, FreeSize) else n for n in spec.shape)
+        if have != want:
+            wrong.append((name, have, want))
     wrong_kind = []
     if dtypes is not None:
         for name in wanted:
@@ -117,7 +126,7 @@ class WeightStore:
         raw = self._source.tensor(name)
         if not raw.dtype.is_floating_point:
             target = torch.int32
-        elif role in ("bias", "norm", "norm0"):
+        elif role in ("bias", "norm", "norm0", "average"):
             target = torch.float32
         elif self.dtype == torch.float32 or (self.keep_wide and raw.dtype in _WIDE):
             target = torch.float32

@@ -5,7 +5,7 @@ parts declare, under their checkpoint names, so that the ordinary loader reads t
 folder like any other.  Values come from one ``torch.Generator(seed)`` on the CPU,
 drawn in float32 in the declared order of the tensors and then cast: products'
 weights, tables and biases ``N(0, std)``, norm scales ``1 + N(0, norm_noise)`` (``N(0, norm_noise)`` for a
-scale that is stored around zero).
+scale that is stored around zero; one more is added to the last of the weights of a sum over states).
 ``std`` defaults to the configuration's ``initializer_range`` when it has one.
 """
 
@@ -29,11 +29,13 @@ def random_tensors(specs, seed: int, std: float, norm_noise: float, dtype: torch
         if spec.name in out:
             continue
         if spec.role in ("norm", "norm0"):
-            value = torch.ones(spec.shape) if spec.role == "norm" else torch.zeros(spec.shape)
+            value = torch.ones(spec.default_shape) if spec.role == "norm" else torch.zeros(spec.default_shape)
             if norm_noise:
-                value = value + torch.randn(spec.shape, generator=generator) * norm_noise
+                value = value + torch.randn(spec.default_shape, generator=generator) * norm_noise
         else:
-            value = torch.randn(spec.shape, generator=generator) * std
+            value = torch.randn(spec.default_shape, generator=generator) * std
+            if spec.role == "average":
+                value[-1] += 1.0
         out[spec.name] = value.to(dtype)
     return out
 
@@ -57,7 +59,7 @@ class RandomSource:
         return self._specs.keys()
 
     def shape(self, name):
-        return tuple(self._specs[name][0].shape)
+        return self._specs[name][0].default_shape
 
     def dtype(self, name):
         return self._dtype
@@ -66,11 +68,13 @@ class RandomSource:
         spec, index = self._specs[name]
         generator = torch.Generator(device=self.device).manual_seed(self.seed * 1_000_003 + index)
         if spec.role in ("norm", "norm0"):
-            value = (torch.ones if spec.role == "norm" else torch.zeros)(spec.shape, device=self.device)
+            value = (torch.ones if spec.role == "norm" else torch.zeros)(spec.default_shape, device=self.device)
             if self.norm_noise:
-                value += torch.randn(spec.shape, generator=generator, device=self.device) * self.norm_noise
+                value += torch.randn(spec.default_shape, generator=generator, device=self.device) * self.norm_noise
         else:
-            value = torch.randn(spec.shape, generator=generator, device=self.device) * self.std
+            value = torch.randn(spec.default_shape, generator=generator, device=self.device) * self.std
+            if spec.role == "average":
+                value[-1] += 1.0
         return value.to(self._dtype)
 
 

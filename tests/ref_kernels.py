@@ -9,6 +9,8 @@ without a GPU.  The product never imports this file.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from distie_b200.kernels.interface import KernelSet, KvSlot, Normed, RotaryTable, StepTensors, Terms
@@ -258,6 +260,23 @@ def norm_add_rmsnorm(delta, delta_weight, delta_eps, residual, weight, eps, dtyp
     return (summed if rows_index is None else residual), out
 
 
+def average_add_rmsnorm(ahead, residual, weight, eps, dtype, rows_index=None):
+    """Returns (averaged residual, layer's own result, normed or None)."""
+    value, state = ahead.value, residual
+    if isinstance(value, Normed):
+        state, _ = norm_add_rmsnorm(value.value, value.weight, value.eps, residual, torch.ones(residual.shape[1]), 1.0, torch.float32)
+    elif value is not None:
+        state = residual + flat_sum(value)
+    averaged = ahead.weights[ahead.count] * state
+    for j in range(ahead.count):
+        averaged = averaged + ahead.weights[j] * ahead.history[j]
+    source = averaged if rows_index is None else averaged[rows_index.long()]
+    out = None
+    if weight is not None:
+        out = (source * torch.rsqrt((source * source).mean(-1, keepdim=True) + eps) * weight.float()).to(dtype)
+    return averaged, state, out
+
+
 def qk_rope_norm_write(qk, bias, step: StepTensors, kv: KvSlot | None, rotary, num_heads, num_kv_heads, head_dim,
                        norm_eps, q_dtype):
     """Returns q [T, heads * head_dim]; stores k (rotated, normed) and v (the key as projected) in their pages."""
@@ -320,6 +339,8 @@ def activation(x, kind="silu", scale=1.0, scaled_columns=0):
     out = whole(x).clone()
     if kind == "silu":
         out = _silu(out)
+    elif kind == "tanh":
+        out = torch.tanh(out)
     if scaled_columns:
         out[:, :scaled_columns] *= scale
     return out
@@ -380,9 +401,14 @@ def glu(g, u, limit=None):
 
 
 def route_top(x, router, top, scoring="sigmoid", groups=None, weight_scale=1.0, extra_rows=0, correction=None,
-              normalise=False):
+              normalise=False, logit_bias=None):
     logits = x.float() @ router.float().T
     experts = router.shape[0] - int(extra_rows)
+    if logit_bias is not None:
+        logits[:, :experts] += logit_bias.float()
+    if scoring == "softmax_chosen":
+        values, ids = torch.sort(logits[:, :experts], dim=-1, descending=True, stable=True)
+        return ids[:, :top].to(torch.int32).contiguous(), torch.softmax(values[:, :top], -1).contiguous() * float(weight_scale)
     scores = torch.softmax(logits[:, :experts], -1) if scoring == "softmax" else torch.sigmoid(logits[:, :experts])
     if correction is not None or normalise:
         choice = scores + correction.float() if correction is not None else scores
@@ -434,11 +460,61 @@ def linear_glu(x, weight, dtype, limit=None, row_gate=None):
     return hidden.to(dtype)
 
 
-def linear_act(x, weight, dtype, kind="relu2"):
-    z = x.float() @ weight.float().T
-    if kind != "relu2":
-        raise ValueError(kind)
-    return (torch.relu(z) ** 2).to(dtype)
+def act(z, kind, numbers=None):
+    if kind == "relu2":
+        return torch.relu(z) ** 2
+    if kind == "gelu":
+        return torch.nn.functional.gelu(z)
+    if kind == "xielu":
+        left = numbers[1] * (torch.expm1(torch.clamp(z, max=0.0)) - z)
+        return torch.where(z > 0, numbers[0] * z * z, left) + 0.5 * z
+    raise ValueError(kind)
+
+
+def linear_act(x, weight, dtype, kind="relu2", numbers=None):
+    return act(x.float() @ weight.float().T, kind, numbers).to(dtype)
+
+
+def routed_act(x, ids, weights, up, down, kind="gelu", numbers=None):
+    tokens, top = ids.shape
+    out = torch.zeros((top, tokens, x.shape[1]), dtype=torch.float32, device=x.device)
+    for t in range(tokens):
+        for j in range(top):
+            e = int(ids[t, j])
+            hidden = act(up[e].float() @ x[t].float(), kind, numbers).to(x.dtype).float()
+            out[j, t] = (down[e].float() @ hidden) * weights[t, j].float()
+    return out
+
+
+# -- recurrences whose decay varies by channel ---------------------------------------------------------------------
+def selective_scan(x, dt, B, C, gate, rates, skip, dt_bias, state, step: StepTensors, dtype):
+    tokens = step.num_tokens
+    dt, B, C, gate = _softplus(whole(dt) + dt_bias.float()), whole(B), whole(C), whole(gate)
+    seats = token_seats(step)
+    out = torch.zeros((tokens, x.shape[1]), dtype=torch.float32, device=x.device)
+    for t in range(tokens):
+        seat = int(seats[t])
+        state[seat] = torch.exp(dt[t] * rates) * state[seat] + B[t][:, None] * (dt[t] * x[t])[None, :]
+        out[t] = C[t] @ state[seat] + skip * x[t]
+    return (out * _silu(gate)).to(dtype)
+
+
+def channel_delta(proj, decay, decay_bias, rate_bias, state, step: StepTensors, heads, dim):
+    tokens, n = step.num_tokens, heads * dim
+    proj = whole(proj)
+    r, k, v = (proj[:, i * n : (i + 1) * n].reshape(tokens, heads, dim) for i in range(3))
+    rate = torch.sigmoid(proj[:, 3 * n : 4 * n] + rate_bias.float()).reshape(tokens, heads, dim)
+    keep = torch.exp(-math.exp(-0.5) * torch.sigmoid(whole(decay) + decay_bias.float())).reshape(tokens, heads, dim)
+    seats = token_seats(step)
+    out = torch.zeros((tokens, heads, dim), dtype=torch.float32, device=proj.device)
+    for t in range(tokens):
+        S = state[int(seats[t])]  # [heads, value element, key channel]
+        u = k[t] / torch.sqrt((k[t] * k[t]).sum(-1, keepdim=True) + 1e-6)
+        seen = torch.einsum("hvk,hk->hv", S, u)
+        S = keep[t][:, None, :] * S - seen[:, :, None] * (rate[t] * u)[:, None, :] + v[t][:, :, None] * k[t][:, None, :]
+        state[int(seats[t])] = S
+        out[t] = torch.einsum("hvk,hk->hv", S, r[t])
+    return out.reshape(tokens, n)
 
 
 # -- attention through a latent ------------------------------------------------------------------------------------
@@ -450,7 +526,7 @@ def latent_kv_write(proj, step: StepTensors, kv, rotary, q_rank, q_norm, kv_rank
     """Returns the normed query latent ``[T, q_rank]``; stores the token's row in ``kv.k`` (if ``kv``)."""
     tokens = step.num_tokens
     proj = whole(proj)[:tokens]
-    q_latent = _unit_rms(proj[:, :q_rank], q_norm, eps).to(dtype)
+    q_latent = _unit_rms(proj[:, :q_rank], q_norm, eps).to(dtype) if q_rank else None
     if kv is not None:
         latent = _unit_rms(proj[:, q_rank : q_rank + kv_rank], kv_norm, eps)
         part = proj[:, q_rank + kv_rank : q_rank + kv_rank + rot_dim]
@@ -557,11 +633,21 @@ class RefKernels(KernelSet):
         if out is not None:
             out.copy_(normed)
 
+    def average_add_rmsnorm(self, ahead, residual, weight, eps, out, rows_index=None):
+        averaged, state, normed = average_add_rmsnorm(ahead, residual, weight, eps, out.dtype if out is not None else self.dtype,
+                                                      rows_index)
+        if rows_index is None:
+            if ahead.count < ahead.history.shape[0]:
+                ahead.history[ahead.count].copy_(state)
+            residual.copy_(averaged)
+        if out is not None:
+            out.copy_(normed)
+
     def qk_rope_norm_write(self, qk, bias, step, kv, rotary, num_heads, num_kv_heads, head_dim, norm_eps, q_out):
         q_out.copy_(qk_rope_norm_write(qk, bias, step, kv, rotary, num_heads, num_kv_heads, head_dim, norm_eps, q_out.dtype))
 
-    def activation(self, x, kind="silu", scale=1.0, scaled_columns=0):
-        return activation(x, kind, scale, scaled_columns)
+    def activation(self, x, kind="silu", scale=1.0, scaled_columns=0, out_dtype=None):
+        return activation(x, kind, scale, scaled_columns).to(out_dtype or torch.float32)
 
     def exp_gate_scan(self, log_in, log_forget, in_bias, forget_bias, cap, state, step):
         return exp_gate_scan(log_in, log_forget, in_bias, forget_bias, cap, state, step)
@@ -570,8 +656,8 @@ class RefKernels(KernelSet):
         return stabilized_readout(read, floor, heads, value_dim)
 
     def route_top(self, x, router, top, scoring="sigmoid", groups=None, weight_scale=1.0, extra_rows=0, correction=None,
-                  normalise=False):
-        return route_top(x, router, top, scoring, groups, weight_scale, extra_rows, correction, normalise)
+                  normalise=False, logit_bias=None):
+        return route_top(x, router, top, scoring, groups, weight_scale, extra_rows, correction, normalise, logit_bias)
 
     def routed_swiglu(self, x, ids, weights, gate_up, down, scale_input=True, limit=None, identity=0):
         return routed_swiglu(x, ids, weights, gate_up, down, scale_input, limit, identity)
@@ -579,11 +665,22 @@ class RefKernels(KernelSet):
     def linear_glu(self, x, weight, limit=None, row_gate=None):
         return linear_glu(x, weight, self.dtype, limit, row_gate)
 
-    def linear_act(self, x, weight, kind="relu2"):
-        return linear_act(x, weight, self.dtype, kind)
+    def linear_act(self, x, weight, kind="relu2", numbers=None):
+        return linear_act(x, weight, self.dtype, kind, numbers)
+
+    def routed_act(self, x, ids, weights, up, down, kind="gelu", numbers=None):
+        return routed_act(x, ids, weights, up, down, kind, numbers)
+
+    def selective_scan(self, x, dt, B, C, gate, rates, skip, dt_bias, state, step, out):
+        out.copy_(selective_scan(x, dt, B, C, gate, rates, skip, dt_bias, state, step, out.dtype))
+
+    def channel_delta(self, proj, decay, decay_bias, rate_bias, state, step, heads, dim):
+        return channel_delta(proj, decay, decay_bias, rate_bias, state, step, heads, dim)
 
     def latent_kv_write(self, proj, step, kv, rotary, q_rank, q_norm, kv_rank, kv_norm, rot_dim, eps, q_latent_out):
-        q_latent_out.copy_(latent_kv_write(proj, step, kv, rotary, q_rank, q_norm, kv_rank, kv_norm, rot_dim, eps, self.dtype))
+        q_latent = latent_kv_write(proj, step, kv, rotary, q_rank, q_norm, kv_rank, kv_norm, rot_dim, eps, self.dtype)
+        if q_latent_out is not None:
+            q_latent_out.copy_(q_latent)
 
     def latent_queries(self, q, up_keys, step, rotary, num_heads, dim, rot_dim):
         return latent_queries(q, up_keys, step, rotary, num_heads, dim, rot_dim, self.dtype)
@@ -606,8 +703,9 @@ class RefKernels(KernelSet):
     def head_gate(self, x, logits, num_heads):
         x.copy_(head_gate(x, logits, num_heads))
 
-    def short_conv(self, x, weight, bias, state, step, activation="silu", input_bias=None):
-        return short_conv(x, weight, bias, state, step, activation, input_bias)
+    def short_conv(self, x, weight, bias, state, step, activation="silu", input_bias=None, typed=False):
+        out = short_conv(x, weight, bias, state, step, activation, input_bias)
+        return (out, out.to(self.dtype)) if typed else out
 
     def linear_recurrence(self, rule, q, k, v, decay, write, state, step, heads, groups, key_dim, value_dim,
                           decay_rate=None, decay_bias=None, skip=None, unit_column=False):
