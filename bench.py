@@ -298,6 +298,24 @@ def zuzunex_config(size: dict, layers: int) -> dict:
             "logit_scale": 1.0, "layers": [pattern[i % 4] for i in range(layers)]}
 
 
+def mekusun_config(size: dict, layers: int) -> dict:
+    """The Mekusun design at a Qwen2.5 layer's width and heads: a selective scan over twice the width (16 states a
+    channel, steps of rank width / 16, four taps), attention through a latent of 512 (heads of 128 plain and 64 rotated
+    dimensions, values of 128), a delta rule with heads of 128; one layer in four has the dense xIELU feed-forward of
+    the dense width, the others 16 experts of a quarter of it, four of them a token (the same active part)."""
+    width, heads = size["width"], size["heads"]
+    dense = {"kind": "dense", "ff": size["ff"]}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 4}, "expert": {"ff": size["ff"] // 4}}
+    latent = {"type": "latent_attention", "mlp": moe, "mixer": {
+        "heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+        "rot": {"base": 1e6, "dims": 64}}}
+    scan = {"type": "mamba1", "mlp": moe, "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}}
+    delta = {"type": "general_delta", "mlp": dense, "mixer": {"heads": heads, "dim": 128}}
+    pattern = [delta, scan, latent, latent]
+    return {"architecture": "Mekusun", "vocab": COMPARE_VOCAB, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "layers": [pattern[i % 4] for i in range(layers)]}
+
+
 def qwen2_config(size: dict, layers: int) -> dict:
     return {"architectures": ["Qwen2ForCausalLM"], "vocab_size": COMPARE_VOCAB, "hidden_size": size["width"],
             "intermediate_size": size["ff"], "num_hidden_layers": layers, "num_attention_heads": size["heads"],
@@ -306,9 +324,10 @@ def qwen2_config(size: dict, layers: int) -> dict:
 
 
 def compare_designs(args) -> int:
-    """``--compare zelasun`` (or ``fovudra``, ``zururax``, ``zuzunex``): prefill of 2,048 tokens and decode steps at batch ``--batch`` behind
+    """``--compare zelasun`` (or ``fovudra``, ``zururax``, ``zuzunex``, ``mekusun``): prefill of 2,048 tokens and decode steps at batch ``--batch`` behind
     1,024-token prompts, for the named design beside the Qwen2 decoder (and, for Fovudra, beside Zelasun, the other
-    design with recurrences; for Zururax, beside Fovudra, the other design with routed experts) at equal width, feed-forward, heads and depth.  Each model is
+    design with recurrences; for Zururax, beside Fovudra, the other design with routed experts; for Mekusun, beside Zururax, the other design with
+    a latent, and Zelasun) at equal width, feed-forward, heads and depth.  Each model is
     built at two depths (4 and 8 layers) so that the time of a layer is the difference, free of embedding and head.
     One JSON line; not the repository's headline metric."""
     import gc
@@ -323,13 +342,15 @@ def compare_designs(args) -> int:
     dtype = "bfloat16" if args.dtype == "bf16" else "float32"
     depths = (4, 8) if args.layers is None else (args.layers,)
     designs = {"zelasun": ("zelasun", "qwen2"), "fovudra": ("fovudra", "zelasun", "qwen2"),
-               "zururax": ("zururax", "fovudra", "qwen2"), "zuzunex": ("zuzunex", "fovudra", "qwen2")}[args.compare]
+               "zururax": ("zururax", "fovudra", "qwen2"), "zuzunex": ("zuzunex", "fovudra", "qwen2"),
+               "mekusun": ("mekusun", "zururax", "zelasun", "qwen2")}[args.compare]
     if args.designs:
         designs = tuple(d for d in designs if d in args.designs.split(","))
     configs = {"zelasun": lambda size, depth: zelasun_config(size, depth, args.chunk),
                "fovudra": lambda size, depth: fovudra_config(size, depth, args.chunk),
                "zururax": lambda size, depth: zururax_config(size, depth),
                "zuzunex": lambda size, depth: zuzunex_config(size, depth),
+               "mekusun": lambda size, depth: mekusun_config(size, depth),
                "qwen2": lambda size, depth: qwen2_config(size, depth)}
     out = {"compare": " beside ".join(designs), "dtype": args.dtype, "batch": args.batch, "prompt_len": PROMPT_LEN,
            "prefill_tokens": PREFILL_TOKENS, "chunk": args.chunk, "sizes": {}}
@@ -589,7 +610,7 @@ def main() -> int:
                         help="with --impl reference: its attention backend (default: DISTIE_ATTN, else auto)")
     parser.add_argument("--ref-device", default=None, help=argparse.SUPPRESS)  # "cpu": a dry run of the reference arm
     parser.add_argument("--designs", default=None, help="with --compare: only these of its designs, with commas between them")
-    parser.add_argument("--compare", default=None, choices=["zelasun", "fovudra", "zururax", "zuzunex"],
+    parser.add_argument("--compare", default=None, choices=["zelasun", "fovudra", "zururax", "zuzunex", "mekusun"],
                         help="time another design beside the Qwen2 decoder at equal layer sizes instead of the default run")
     parser.add_argument("--chunk", type=int, default=1024,
                         help="with --compare: the chunk (Zelasun) or window (Fovudra) of the design's attention")

@@ -80,6 +80,23 @@ __device__ __forceinline__ float hidden_act(float z, HiddenAct act) {
   if (act.kind == DISTIE_ACT_GELU) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
   return z > 0.f ? act.a * z * z + 0.5f * z : act.b * (expm1f(z) - z) + 0.5f * z;
 }
+// The same for epilogues that round to 16 bits, on the fast exponential.  GELU through the complementary error function
+// of |z| / sqrt 2 as a polynomial in 1 / (1 + p |x|) times exp(-x^2) (Abramowitz and Stegun, Handbook of Mathematical
+// Functions, 7.1.26: absolute error below 1.5e-7).
+__device__ __forceinline__ float hidden_act_fast(float z, HiddenAct act) {
+  if (act.kind == DISTIE_ACT_RELU2) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  }
+  if (act.kind == DISTIE_ACT_GELU) {
+    const float x = fabsf(z) * 0.70710678118654752f;
+    const float t = __fdividef(1.f, 1.f + 0.3275911f * x);
+    const float poly = t * (0.254829592f + t * (-0.284496736f + t * (1.421413741f + t * (-1.453152027f + t * 1.061405429f))));
+    const float half_tail = 0.5f * z * poly * __expf(-x * x);
+    return z > 0.f ? z - half_tail : half_tail;
+  }
+  return (z > 0.f ? act.a * z * z : act.b * (__expf(z) - 1.f - z)) + 0.5f * z;
+}
 
 // A sink in a softmax: one more term exp(sink) in the denominator that has no value.  Given the running maximum `m`
 // and sum `l` over the keys (sum of exp(s - m)), returns the factor the mix (sum of exp(s - m) v) is multiplied by:

@@ -133,7 +133,7 @@ __device__ __forceinline__ void store_accumulator(uint32_t lane_base, int row0, 
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
         v[j] = __uint_as_float(acc[j]);
-        if (EPI == GEMM_EPI_ACT) v[j] = hidden_act(v[j], act);
+        if (EPI == GEMM_EPI_ACT) v[j] = hidden_act_fast(v[j], act);
       }
       const int col = n0 + c0;
       if (rows_valid > 0 && col < N) {
@@ -953,7 +953,7 @@ gemm_tcgen05_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
         OutT* dst = out + (EPI == SKINNY_EPI_SLICE ? (size_t)split * M * ldo : 0) + row;
 #pragma unroll
         for (int j = 0; j < 16; ++j)
-          if (c0 + j < M) dst[(size_t)(c0 + j) * ldo] = from_float<OutT>(EPI == SKINNY_EPI_ACT ? hidden_act(acc[j], act) : acc[j] + b);
+          if (c0 + j < M) dst[(size_t)(c0 + j) * ldo] = from_float<OutT>(EPI == SKINNY_EPI_ACT ? hidden_act_fast(acc[j], act) : acc[j] + b);
       }
     }
   }

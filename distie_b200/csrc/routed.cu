@@ -506,7 +506,7 @@ grouped_product_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, co
         const int slot = first + local;
         const float v = c_s[warp][r][c];
         if (SWIGLU) out[(size_t)slot * N + n] = __float2bfloat16_rn(v);
-        else if (MODE == kGroupedAct) out[(size_t)slot * N + n] = __float2bfloat16_rn(hidden_act(v, act));
+        else if (MODE == kGroupedAct) out[(size_t)slot * N + n] = __float2bfloat16_rn(hidden_act_fast(v, act));
         else out32[(size_t)plan.dest[slot] * N + n] = scale_out ? v * scale_s[local] : v;
       }
     }

@@ -718,7 +718,9 @@ def test_replay_against_plain(kit, name, mode):
         ran = kit.kernel_counts
         assert all(ran.get(n) for n in ("selective_scan", "channel_delta", "average_add_rmsnorm", "routed_act", "latent_kv_write"))
         if name == "wide" and kit.dtype == torch.bfloat16:
-            assert ran.get("latent_attention_mma") and ran.get("gemm_tcgen05") and ran.get("gemm_tcgen05_grouped") is not None
+            assert ran.get("latent_attention_mma")
+            if mode in ("whole", "tail"):  # portions long enough for full tiles
+                assert ran.get("gemm_tcgen05") and ran.get("gemm_tcgen05_grouped") is not None
 
 
 @pytest.mark.parametrize("name", ["small", "awkward"])
