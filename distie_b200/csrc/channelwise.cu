@@ -17,6 +17,29 @@ __device__ __forceinline__ float exp2_unit(float x) {
   return y;
 }
 
+// 32-bit arithmetic on pairs: one instruction, each half rounded as the single operation is.
+typedef unsigned long long Pair;
+__device__ __forceinline__ Pair pack2(float lo, float hi) {
+  Pair p;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(lo), "f"(hi));
+  return p;
+}
+__device__ __forceinline__ float2 unpack2(Pair p) {
+  float2 v;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(v.x), "=f"(v.y) : "l"(p));
+  return v;
+}
+__device__ __forceinline__ Pair mul2(Pair a, Pair b) {
+  Pair p;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(p) : "l"(a), "l"(b));
+  return p;
+}
+__device__ __forceinline__ Pair fma2(Pair a, Pair b, Pair c) {
+  Pair p;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(p) : "l"(a), "l"(b), "l"(c));
+  return p;
+}
+
 // ---------------------------------------------------------------------------
 // Selective scan.  Per channel c and state n, with d = softplus(dt[t, c] + dt_bias[c]):
 //   S[n, c] <- exp(d rates[n, c]) S[n, c] + d x[t, c] B[t, n]
@@ -50,13 +73,26 @@ struct SelectArgs {
   float* tile_steps;  // [tiles, channels]
 };
 
-template <typename T, int PER, int LANES, int MODE>
+// Four neighbouring columns of a row as the element loop needs them: one 16-byte load (VEC), or what there is of them.
+template <bool VEC>
+__device__ __forceinline__ float4 load_quad(const Sliced& m, size_t row, int col, int columns) {
+  if (VEC) return m.at4(row, col);
+  float v[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) v[i] = col + i < columns ? m.at(row, col + i) : 0.f;
+  return make_float4(v[0], v[1], v[2], v[3]);
+}
+
+template <typename T, int PER, int LANES, int MODE, bool VEC>
 __global__ void __launch_bounds__(kSelectThreads) selective_scan_kernel(SelectArgs a, T* __restrict__ out) {
   constexpr int CH = kSelectThreads / LANES;  // channels of the block
   constexpr int PER_WARP = 32 / LANES;        // channels of a warp
   constexpr int NP = PER * LANES;
-  __shared__ float d_s[kSelectTile][CH];      // the step sizes; a token's read-out takes the place of its step
-  __shared__ float dx_s[kSelectTile][CH];
+  constexpr int QUADS = CH / 4;               // runs of four channels
+  constexpr int ITEMS = (kSelectTile * QUADS + kSelectThreads - 1) / kSelectThreads;  // (token, run) pairs of a thread
+  constexpr int ROWS = (kSelectTile * NP + kSelectThreads - 1) / kSelectThreads;      // numbers of B (and of C) of a thread
+  __shared__ __align__(16) float d_s[kSelectTile][CH];  // the step sizes; a token's read-out takes the place of its step
+  __shared__ __align__(16) float dx_s[kSelectTile][CH];
   __shared__ __align__(16) float b_s[kSelectTile][NP];
   __shared__ __align__(16) float c_s[kSelectTile][NP];
   const int tid = threadIdx.x, lane = tid & 31;
@@ -80,57 +116,105 @@ __global__ void __launch_bounds__(kSelectThreads) selective_scan_kernel(SelectAr
   }
   const size_t plane = (size_t)a.states * a.channels;
   float* held = MODE == kSelectWalk ? a.state + (size_t)a.seq_seat[row] * plane : a.tile_state + blockIdx.y * plane;
-  float S[PER], rate[PER];
+  const Sliced x{a.x, a.x_stride, 1, 0};
+
+  // A tile's inputs are on their way while the tile before it is walked.
+  float4 dt_r[ITEMS], x_r[ITEMS], x_now[ITEMS], gate_r[ITEMS];
+  float b_r[ROWS], c_r[ROWS];
+  auto place = [&](int item, int& tok, int& ch) {  // (token, first channel) of a thread's item
+    const int idx = item * kSelectThreads + tid;
+    tok = idx / QUADS;
+    ch = (idx % QUADS) * 4;
+  };
+  auto fetch = [&](int t0) {
+    const int count = min(kSelectTile, end - t0);
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    const int n = part * PER + i;
-    const bool live = valid && n < a.states;
-    S[i] = (live && MODE != kSelectLocal) ? held[(size_t)n * a.channels + c] : 0.f;
-    rate[i] = live ? a.rates[(size_t)n * a.channels + c] * kLog2e : 0.f;
+    for (int i = 0; i < ITEMS; ++i) {
+      int tok, ch;
+      place(i, tok, ch);
+      if (tok < count && c0 + ch < a.channels) {
+        dt_r[i] = load_quad<VEC>(a.dt, t0 + tok, c0 + ch, a.channels);
+        x_r[i] = load_quad<VEC>(x, t0 + tok, c0 + ch, a.channels);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+      const int idx = i * kSelectThreads + tid, tok = idx / NP, n = idx % NP;
+      const bool live = tok < count && n < a.states;
+      b_r[i] = live ? a.B.at(t0 + tok, n) : 0.f;
+      if (MODE != kSelectLocal) c_r[i] = live ? a.C.at(t0 + tok, n) : 0.f;
+    }
+  };
+  fetch(first);
+
+  Pair S[PER / 2], rate[PER / 2];
+#pragma unroll
+  for (int i = 0; i < PER / 2; ++i) {
+    float s[2], r[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int n = part * PER + 2 * i + e;
+      const bool live = valid && n < a.states;
+      s[e] = (live && MODE != kSelectLocal) ? held[(size_t)n * a.channels + c] : 0.f;
+      r[e] = live ? a.rates[(size_t)n * a.channels + c] * kLog2e : 0.f;
+    }
+    S[i] = pack2(s[0], s[1]);
+    rate[i] = pack2(r[0], r[1]);
   }
   float steps = 0.f;
   for (int t0 = first; t0 < end; t0 += kSelectTile) {
     const int count = min(kSelectTile, end - t0);
-    for (int idx = tid; idx < count * CH; idx += kSelectThreads) {
-      const int tok = idx / CH, ch = idx % CH;
-      float d = 0.f, dx = 0.f;
-      if (c0 + ch < a.channels) {
-        d = softplus_f(a.dt.at(t0 + tok, c0 + ch) + a.dt_bias[c0 + ch]);
-        dx = d * a.x[(size_t)(t0 + tok) * a.x_stride + c0 + ch];
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      int tok, ch;
+      place(i, tok, ch);
+      if (tok >= kSelectTile) continue;
+      float4 d = make_float4(0.f, 0.f, 0.f, 0.f), dx = d;
+      if (tok < count && c0 + ch < a.channels) {
+        float bias[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) bias[e] = (VEC || c0 + ch + e < a.channels) ? a.dt_bias[c0 + ch + e] : 0.f;
+        d = make_float4(softplus_f(dt_r[i].x + bias[0]), softplus_f(dt_r[i].y + bias[1]), softplus_f(dt_r[i].z + bias[2]),
+                        softplus_f(dt_r[i].w + bias[3]));
+        dx = make_float4(d.x * x_r[i].x, d.y * x_r[i].y, d.z * x_r[i].z, d.w * x_r[i].w);
+        x_now[i] = x_r[i];
+        if (MODE != kSelectLocal) gate_r[i] = load_quad<VEC>(a.gate, t0 + tok, c0 + ch, a.channels);
       }
-      d_s[tok][ch] = d;
-      dx_s[tok][ch] = dx;
+      *reinterpret_cast<float4*>(&d_s[tok][ch]) = d;
+      *reinterpret_cast<float4*>(&dx_s[tok][ch]) = dx;
     }
-    for (int idx = tid; idx < count * NP; idx += kSelectThreads) {
-      const int tok = idx / NP, n = idx % NP;
-      const bool live = n < a.states;
-      b_s[tok][n] = live ? a.B.at(t0 + tok, n) : 0.f;
-      if (MODE != kSelectLocal) c_s[tok][n] = live ? a.C.at(t0 + tok, n) : 0.f;
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+      const int idx = i * kSelectThreads + tid;
+      if (kSelectTile * NP % kSelectThreads != 0 && idx >= kSelectTile * NP) continue;
+      (&b_s[0][0])[idx] = b_r[i];
+      if (MODE != kSelectLocal) (&c_s[0][0])[idx] = c_r[i];
     }
+    if (t0 + kSelectTile < end) fetch(t0 + kSelectTile);
     __syncthreads();
 #pragma unroll 4
     for (int tok = 0; tok < count; ++tok) {
       const float d = d_s[tok][local], dx = dx_s[tok][local];
-      float y = 0.f;
+      const Pair d2 = pack2(d, d), dx2 = pack2(dx, dx);
+      Pair y2 = 0;
 #pragma unroll
       for (int q = 0; q < PER / 4; ++q) {
-        const float4 b = *reinterpret_cast<const float4*>(&b_s[tok][part * PER + 4 * q]);
-        const float bb[4] = {b.x, b.y, b.z, b.w};
-        float cc[4] = {0.f, 0.f, 0.f, 0.f};
-        if (MODE != kSelectLocal) {
-          const float4 v = *reinterpret_cast<const float4*>(&c_s[tok][part * PER + 4 * q]);
-          cc[0] = v.x; cc[1] = v.y; cc[2] = v.z; cc[3] = v.w;
-        }
+        const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(&b_s[tok][part * PER + 4 * q]);
+        ulonglong2 w = make_ulonglong2(0, 0);
+        if (MODE != kSelectLocal) w = *reinterpret_cast<const ulonglong2*>(&c_s[tok][part * PER + 4 * q]);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          float& s = S[4 * q + i];
-          s = exp2_unit(d * rate[4 * q + i]) * s + dx * bb[i];
-          if (MODE != kSelectLocal) y += s * cc[i];
+        for (int e = 0; e < 2; ++e) {
+          const float2 z = unpack2(mul2(d2, rate[2 * q + e]));
+          const Pair keep = pack2(exp2_unit(z.x), exp2_unit(z.y));
+          S[2 * q + e] = fma2(keep, S[2 * q + e], mul2(dx2, e ? b.y : b.x));
+          if (MODE != kSelectLocal) y2 = fma2(S[2 * q + e], e ? w.y : w.x, y2);
         }
       }
       if (MODE == kSelectLocal) {
         steps += d;
       } else {
+        const float2 halves = unpack2(y2);
+        float y = halves.x + halves.y;
 #pragma unroll
         for (int offset = PER_WARP; offset < 32; offset <<= 1) y += __shfl_xor_sync(0xffffffffu, y, offset);
         if (part == 0) d_s[tok][local] = y;  // (the channel's other threads have read the step: they took part in the sum)
@@ -138,12 +222,26 @@ __global__ void __launch_bounds__(kSelectThreads) selective_scan_kernel(SelectAr
     }
     __syncthreads();
     if (MODE != kSelectLocal) {
-      for (int idx = tid; idx < count * CH; idx += kSelectThreads) {  // (the same thread fills this place with the next tile)
-        const int tok = idx / CH, ch = idx % CH;
-        if (c0 + ch >= a.channels) continue;
-        const size_t t = t0 + tok;
-        const float y = d_s[tok][ch] + a.skip[c0 + ch] * a.x[t * a.x_stride + c0 + ch];
-        out[t * a.out_stride + c0 + ch] = from_float<T>(y * silu_f(a.gate.at(t, c0 + ch)));
+#pragma unroll
+      for (int i = 0; i < ITEMS; ++i) {  // (a thread finishes the items that it fills with the next tile)
+        int tok, ch;
+        place(i, tok, ch);
+        if (tok >= count || c0 + ch >= a.channels) continue;
+        const float4 y = *reinterpret_cast<const float4*>(&d_s[tok][ch]);
+        float skip[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) skip[e] = (VEC || c0 + ch + e < a.channels) ? a.skip[c0 + ch + e] : 0.f;
+        const float4 o = make_float4((y.x + skip[0] * x_now[i].x) * silu_f(gate_r[i].x), (y.y + skip[1] * x_now[i].y) * silu_f(gate_r[i].y),
+                                     (y.z + skip[2] * x_now[i].z) * silu_f(gate_r[i].z), (y.w + skip[3] * x_now[i].w) * silu_f(gate_r[i].w));
+        T* dst = out + (size_t)(t0 + tok) * a.out_stride + c0 + ch;
+        if (VEC) {
+          store4(dst, o);
+        } else {
+          const float v[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (c0 + ch + e < a.channels) dst[e] = from_float<T>(v[e]);
+        }
       }
     }
   }
@@ -154,9 +252,11 @@ __global__ void __launch_bounds__(kSelectThreads) selective_scan_kernel(SelectAr
   }
   if (MODE == kSelectLocal && part == 0) a.tile_steps[(size_t)blockIdx.y * a.channels + c] = steps;
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    const int n = part * PER + i;
-    if (n < a.states) held[(size_t)n * a.channels + c] = S[i];
+  for (int i = 0; i < PER / 2; ++i) {
+    const float2 s = unpack2(S[i]);
+    const int n = part * PER + 2 * i;
+    if (n < a.states) held[(size_t)n * a.channels + c] = s.x;
+    if (n + 1 < a.states) held[(size_t)(n + 1) * a.channels + c] = s.y;
   }
 }
 
@@ -169,30 +269,49 @@ __global__ void __launch_bounds__(256) selective_chain_kernel(SelectArgs a) {
   const float rate = a.rates[at] * kLog2e;
   float S = 0.f;
   int row = -1;
-#pragma unroll 4
-  for (int tile = 0; tile < a.num_tiles; ++tile) {
-    const int mine = a.token_seq[a.tiles[2 * tile]];
-    const float left = a.tile_state[tile * plane + at];  // (of a request's last tile: not made, and not used)
-    const float keep = exp2_unit(rate * a.tile_steps[(size_t)tile * a.channels + c]);
-    if (mine != row) S = a.state[(size_t)a.seq_seat[mine] * plane + at];
-    row = mine;
-    a.tile_state[tile * plane + at] = S;
-    S = keep * S + left;
+  constexpr int AHEAD = 8;  // tiles whose loads are in flight together
+  for (int base = 0; base < a.num_tiles; base += AHEAD) {
+    float left[AHEAD], steps[AHEAD];  // (of a request's last tile: not made, and not used)
+    int mine[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int tile = min(base + i, a.num_tiles - 1);
+      mine[i] = a.token_seq[a.tiles[2 * tile]];
+      left[i] = a.tile_state[tile * plane + at];
+      steps[i] = a.tile_steps[(size_t)tile * a.channels + c];
+    }
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      if (base + i >= a.num_tiles) break;
+      if (mine[i] != row) S = a.state[(size_t)a.seq_seat[mine[i]] * plane + at];
+      row = mine[i];
+      a.tile_state[(base + i) * plane + at] = S;
+      S = exp2_unit(rate * steps[i]) * S + left[i];
+    }
   }
+}
+
+template <typename T, int PER, int LANES, bool VEC>
+static cudaError_t launch_select_as(const SelectArgs& a, T* out, int rows, bool tiled, cudaStream_t stream) {
+  const unsigned blocks = (unsigned)((a.channels + kSelectThreads / LANES - 1) / (kSelectThreads / LANES));
+  if (rows > 0) selective_scan_kernel<T, PER, LANES, kSelectWalk, VEC><<<dim3(blocks, rows), kSelectThreads, 0, stream>>>(a, out);
+  if (tiled) {
+    const dim3 grid(blocks, a.num_tiles);
+    selective_scan_kernel<T, PER, LANES, kSelectLocal, VEC><<<grid, kSelectThreads, 0, stream>>>(a, out);
+    const size_t plane = (size_t)a.states * a.channels;
+    selective_chain_kernel<<<(unsigned)((plane + 255) / 256), 256, 0, stream>>>(a);
+    selective_scan_kernel<T, PER, LANES, kSelectFinish, VEC><<<grid, kSelectThreads, 0, stream>>>(a, out);
+  }
+  return cudaGetLastError();
 }
 
 template <typename T, int PER, int LANES>
 static cudaError_t launch_select(const SelectArgs& a, T* out, int rows, bool tiled, cudaStream_t stream) {
-  const unsigned blocks = (unsigned)((a.channels + kSelectThreads / LANES - 1) / (kSelectThreads / LANES));
-  if (rows > 0) selective_scan_kernel<T, PER, LANES, kSelectWalk><<<dim3(blocks, rows), kSelectThreads, 0, stream>>>(a, out);
-  if (tiled) {
-    const dim3 grid(blocks, a.num_tiles);
-    selective_scan_kernel<T, PER, LANES, kSelectLocal><<<grid, kSelectThreads, 0, stream>>>(a, out);
-    const size_t plane = (size_t)a.states * a.channels;
-    selective_chain_kernel<<<(unsigned)((plane + 255) / 256), 256, 0, stream>>>(a);
-    selective_scan_kernel<T, PER, LANES, kSelectFinish><<<grid, kSelectThreads, 0, stream>>>(a, out);
-  }
-  return cudaGetLastError();
+  auto quads = [](const Sliced& m) { return ((m.stride | m.split_stride) & 3) == 0 && ((uintptr_t)m.p & 15) == 0; };
+  const bool vec = a.channels % 4 == 0 && ((a.x_stride | a.out_stride) & 3) == 0 && (((uintptr_t)a.x | (uintptr_t)out) & 15) == 0 &&
+                   quads(a.dt) && quads(a.gate);
+  return vec ? launch_select_as<T, PER, LANES, true>(a, out, rows, tiled, stream)
+             : launch_select_as<T, PER, LANES, false>(a, out, rows, tiled, stream);
 }
 
 // Threads per channel: few where many tokens are walked (fewer loads and sums per token), more in steps of single tokens.
