@@ -5,6 +5,7 @@
 // State is read and written through a token's seat; nothing reads host-side batch data beyond counts that a step's
 // layout fixes, so captured decode steps replay these kernels.
 #include "recurrent.cuh"
+#include "tcgen05.cuh"
 
 namespace distie {
 
@@ -339,42 +340,52 @@ static cudaError_t dispatch_select(const SelectArgs& a, T* out, int rows, bool t
 // is taken from the state before the write:  o = sum_i r_i w_i S_i + v (r . k) - g (sum_i r_i a_i k_i), so both sums over
 // the state run side by side.
 //
-// Two kernels.  The first is parallel over tokens and leaves, per token and head, the rows k, w, a, r * w and v and the
-// numbers 1 / (|k|^2 + 1e-6), r . k and sum r a k.  The second walks the tokens: the columns of S (one per value
-// element) never meet, so COLS of them belong to a group of LANES threads that share their key channels (lane l holds
-// channels 4 l + 4 LANES q + e), a block of 64 threads owns 64 / LANES groups of one head of one request.  Tiles of
-// tokens come into shared memory by cp.async a tile ahead of the walk.
+// Two kernels.  The first is parallel over tokens and leaves, per token and head, one contiguous piece of memory: the
+// numbers 1 / (|k|^2 + 1e-6), r . k, sum r a k, then the rows k, w, a, r * w and v, padded with zeros to the walk's width.
+// The second walks the tokens: the columns of S (one per value element) never meet, so COLS of them belong to a group of
+// LANES threads that share their key channels (lane l holds channels 4 l + 4 LANES q + e), a block of 64 threads owns
+// 64 / LANES groups of one head of one request.  Bulk copies bring tiles of tokens into shared memory a tile ahead of the
+// walk (one elected thread; the wait on their mbarrier is bounded: when it runs out the kernel sets the error word to 6
+// and returns).
 // State layout: [seat, head, value element, key channel].
 // ---------------------------------------------------------------------------
 constexpr int kDeltaThreads = 64;
 constexpr float kDecayFactor = 0.6065306597126334f;  // exp(-1/2)
+constexpr int kDeltaNumbers = 4, kDeltaRows = 5;     // of a token and head
 
 struct DeltaArgs {
   Sliced proj, decay;  // proj: [r | k | v | rate]
   const float *decay_bias, *rate_bias;
-  float *rows, *numbers;  // [tokens, heads, 5, dim]; [tokens, heads, 4]
+  float* scratch;
   float* state;
   float* out;
   const int *seq_bounds, *seq_seat;
-  int tokens, heads, dim;
+  int tokens, heads, dim, width;  // width: dim rounded up to what the walk is compiled for
+  int* error;
+  __device__ __forceinline__ float* piece(size_t t, int head) const {
+    return scratch + (t * heads + head) * (kDeltaNumbers + kDeltaRows * width);
+  }
 };
 
 __global__ void __launch_bounds__(128) channel_delta_prepare_kernel(DeltaArgs a) {
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int n = a.heads * a.dim;
   for (int head = blockIdx.y * 4 + warp; head < a.heads; head += gridDim.y * 4) {
-    float* rows = a.rows + ((size_t)t * a.heads + head) * 5 * a.dim;
+    float* numbers = a.piece(t, head);
+    float* rows = numbers + kDeltaNumbers;
     float kk = 0.f, rk = 0.f, rak = 0.f;
+    for (int i = a.dim + lane; i < a.width; i += 32)
+      for (int which = 0; which < kDeltaRows; ++which) rows[which * a.width + i] = 0.f;
     for (int i = lane; i < a.dim; i += 32) {
       const int col = head * a.dim + i;
       const float r = a.proj.at(t, col), k = a.proj.at(t, n + col), v = a.proj.at(t, 2 * n + col);
       const float rate = sigmoid_f(a.proj.at(t, 3 * n + col) + a.rate_bias[col]);
       const float w = expf(-kDecayFactor * sigmoid_f(a.decay.at(t, col) + a.decay_bias[col]));
       rows[i] = k;
-      rows[a.dim + i] = w;
-      rows[2 * a.dim + i] = rate;
-      rows[3 * a.dim + i] = r * w;
-      rows[4 * a.dim + i] = v;
+      rows[a.width + i] = w;
+      rows[2 * a.width + i] = rate;
+      rows[3 * a.width + i] = r * w;
+      rows[4 * a.width + i] = v;
       kk += k * k;
       rk += r * k;
       rak += r * rate * k;
@@ -382,132 +393,175 @@ __global__ void __launch_bounds__(128) channel_delta_prepare_kernel(DeltaArgs a)
     kk = warp_sum(kk);
     rk = warp_sum(rk);
     rak = warp_sum(rak);
-    if (lane == 0)
-      *reinterpret_cast<float4*>(a.numbers + ((size_t)t * a.heads + head) * 4) = make_float4(1.f / (kk + 1e-6f), rk, rak, 0.f);
+    if (lane == 0) *reinterpret_cast<float4*>(numbers) = make_float4(1.f / (kk + 1e-6f), rk, rak, 0.f);
   }
 }
 
-template <int KD, int TILE, int CB>
-struct DeltaStage {
-  float rows[4][TILE][KD];  // k, w, a, r * w; zeros beyond dim
-  float v[TILE][CB];
-  float numbers[TILE][4];
+// One copy of `bytes` (a multiple of 16, both addresses on 16-byte boundaries) into shared memory, counted on `bar`.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+
+// The sums of NV values over groups of LANES neighbouring lanes with few exchanges: every round hands half of the values
+// to a neighbour and keeps the other half; when one value a lane is left, the rest of the group is summed by butterflies.
+// Afterwards lane `holder(i)` (and the lanes that agree with it in the low bits) has the sum of value i in v[0].
+template <int NV, int LANES>
+struct FoldedSum {
+  __host__ __device__ static constexpr int bits() { return NV == 2 ? 1 : NV == 4 ? 2 : 3; }
+  __host__ __device__ static constexpr int holder(int value) {
+    int lane = 0;
+    for (int b = 0; b < bits(); ++b) lane |= ((value >> (bits() - 1 - b)) & 1) << b;
+    return lane;
+  }
+  static __device__ __forceinline__ float run(float (&v)[NV], int sub) {
+#pragma unroll
+    for (int b = 0; b < bits(); ++b) {
+      const int half = NV >> (b + 1);
+      const bool upper = (sub >> b) & 1;
+#pragma unroll
+      for (int i = 0; i < NV / 2; ++i) {
+        if (i >= half) break;
+        const float give = upper ? v[i] : v[i + half], keep = upper ? v[i + half] : v[i];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1 << b);
+      }
+    }
+#pragma unroll
+    for (int offset = 1 << bits(); offset < LANES; offset <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], offset);
+    return v[0];
+  }
 };
 
+template <int KD, int TILE>
+struct DeltaStage {
+  float piece[TILE][kDeltaNumbers + kDeltaRows * KD];
+};
+
+// VEC: columns of the state start on 16-byte boundaries.
 template <int KD, int LANES, int COLS, int TILE, bool VEC>
-__global__ void __launch_bounds__(kDeltaThreads) channel_delta_kernel(DeltaArgs a) {
+__global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaArgs a) {
   constexpr int PER = KD / LANES, CB = kDeltaThreads / LANES * COLS;
-  static_assert(PER >= 4 && PER % 4 == 0, "a thread holds whole float4s of its columns");
+  using Fold = FoldedSum<2 * COLS, LANES>;  // the sums with k, then with r * w, of every column
+  static_assert(PER >= 4 && PER % 4 == 0 && 2 * COLS <= LANES, "a thread holds whole float4s of its columns");
   extern __shared__ __align__(16) unsigned char delta_smem[];
-  using Stage = DeltaStage<KD, TILE, CB>;
+  using Stage = DeltaStage<KD, TILE>;
   Stage* stages = reinterpret_cast<Stage*>(delta_smem);  // two
+  __shared__ __align__(8) uint64_t full[2];
   const int row = blockIdx.x, head = blockIdx.y;
-  const int tid = threadIdx.x, sub = tid % LANES, group = tid / LANES;
+  const int tid = threadIdx.x, sub = tid % LANES, group = tid / LANES, base = (tid & 31) & ~(LANES - 1);
   const int j0 = blockIdx.z * CB + group * COLS;
   const int first = a.seq_bounds[row], end = a.seq_bounds[row + 1];
   if (end <= first) return;
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
 
-  auto stage_tile = [&](int tile, Stage& st) {
+  constexpr uint32_t kBytes = (kDeltaNumbers + kDeltaRows * KD) * sizeof(float);
+  auto stage_tile = [&](int tile, int buffer) {  // one thread
     const int count = min(TILE, end - tile);
-    const float* src = a.rows + ((size_t)tile * a.heads + head) * 5 * a.dim;
-    const size_t token_stride = (size_t)a.heads * 5 * a.dim;
-    if (VEC) {
-      for (int idx = tid; idx < count * 4 * (KD / 4); idx += kDeltaThreads) {
-        const int i = (idx % (KD / 4)) * 4, which = (idx / (KD / 4)) % 4, tok = idx / KD;
-        const bool live = i < a.dim;
-        cp_async_f4(&st.rows[which][tok][i], src + tok * token_stride + (size_t)which * a.dim + (live ? i : 0), live);
-      }
-    } else {
-      for (int idx = tid; idx < count * 4 * KD; idx += kDeltaThreads) {
-        const int i = idx % KD, which = (idx / KD) % 4, tok = idx / (4 * KD);
-        const bool live = i < a.dim;
-        cp_async_f1(&st.rows[which][tok][i], src + tok * token_stride + (size_t)which * a.dim + (live ? i : 0), live);
-      }
-    }
-    for (int idx = tid; idx < count * CB; idx += kDeltaThreads) {
-      const int tok = idx / CB, cj = blockIdx.z * CB + idx % CB;
-      const bool live = cj < a.dim;
-      cp_async_f1(&st.v[tok][idx % CB], src + tok * token_stride + 4 * (size_t)a.dim + (live ? cj : 0), live);
-    }
-    if (tid < count) cp_async_f4(st.numbers[tid], a.numbers + ((size_t)(tile + tid) * a.heads + head) * 4, true);
-    cp_async_commit();
+    mbar_expect_tx(&full[buffer], count * kBytes);
+    for (int tok = 0; tok < count; ++tok) bulk_load(stages[buffer].piece[tok], a.piece(tile + tok, head), kBytes, &full[buffer]);
   };
-
-  stage_tile(first, stages[0]);
+  if (tid == 0) stage_tile(first, 0);
   float* held = a.state + ((size_t)a.seq_seat[row] * a.heads + head) * a.dim * a.dim;
-  float S[COLS][PER];
+  Pair S[COLS][PER / 2];
 #pragma unroll
   for (int col = 0; col < COLS; ++col)
 #pragma unroll
     for (int q = 0; q < PER / 4; ++q) {
       const int i = 4 * sub + 4 * LANES * q;
       const bool live = j0 + col < a.dim;
+      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+      const float* src = held + (size_t)(j0 + col) * a.dim + i;
       if (VEC) {
-        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (live && i < a.dim) s = *reinterpret_cast<const float4*>(held + (size_t)(j0 + col) * a.dim + i);
-        S[col][4 * q] = s.x; S[col][4 * q + 1] = s.y; S[col][4 * q + 2] = s.z; S[col][4 * q + 3] = s.w;
-      } else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[col][4 * q + e] = (live && i + e < a.dim) ? held[(size_t)(j0 + col) * a.dim + i + e] : 0.f;
+        if (live && i < a.dim) s = *reinterpret_cast<const float4*>(src);
+      } else if (live) {
+        if (i < a.dim) s.x = src[0];
+        if (i + 1 < a.dim) s.y = src[1];
+        if (i + 2 < a.dim) s.z = src[2];
+        if (i + 3 < a.dim) s.w = src[3];
       }
+      S[col][2 * q] = pack2(s.x, s.y);
+      S[col][2 * q + 1] = pack2(s.z, s.w);
     }
 
-  int buffer = 0;
-  for (int tile = first; tile < end; tile += TILE, buffer ^= 1) {
-    const int count = min(TILE, end - tile);
+  // The lane whose folded sum is the read-out's of a column stores it.
+  int out_col = -1;
+#pragma unroll
+  for (int col = 0; col < COLS; ++col)
+    if (sub == Fold::holder(COLS + col) && j0 + col < a.dim) out_col = col;
+  const size_t out_stride = (size_t)a.heads * a.dim;
+  float* out_at = a.out + (size_t)first * out_stride + head * a.dim + j0 + max(out_col, 0);
+
+  int round = 0;
+  for (int tile = first; tile < end; tile += TILE, ++round) {
+    const int count = min(TILE, end - tile), buffer = round & 1;
     const bool more = tile + TILE < end;
-    if (more) stage_tile(tile + TILE, stages[buffer ^ 1]);  // its last readers passed the barrier below
-    if (more) cp_async_wait<1>(); else cp_async_wait<0>();
-    __syncthreads();
+    if (more && tid == 0) stage_tile(tile + TILE, buffer ^ 1);  // its last readers passed the barrier below
+    if (!__syncthreads_and(mbar_wait(&full[buffer], (round >> 1) & 1))) {
+      if (tid == 0) {
+        if (a.error) atomicExch(a.error, 6);
+        mbar_wait(&full[buffer], (round >> 1) & 1);  // (bounded) no copy of its own in flight when the block leaves
+        if (more) mbar_wait(&full[buffer ^ 1], ((round + 1) >> 1) & 1);
+      }
+      return;
+    }
     const Stage& st = stages[buffer];
 #pragma unroll 2
     for (int tok = 0; tok < count; ++tok) {
-      const float4 numbers = *reinterpret_cast<const float4*>(st.numbers[tok]);
-      float k[PER], rw[PER];
+      const float* piece = st.piece[tok];
+      const float4 numbers = *reinterpret_cast<const float4*>(piece);
+      const float* rows = piece + kDeltaNumbers + 4 * sub;
+      const float* values = piece + kDeltaNumbers + 4 * KD + j0;  // (of columns past dim: zeros)
+      Pair k[PER / 2], dot_k[COLS], dot_r[COLS];
+#pragma unroll
+      for (int col = 0; col < COLS; ++col) dot_k[col] = dot_r[col] = 0;
 #pragma unroll
       for (int q = 0; q < PER / 4; ++q) {
-        const float4 kv = *reinterpret_cast<const float4*>(&st.rows[0][tok][4 * sub + 4 * LANES * q]);
-        const float4 rv = *reinterpret_cast<const float4*>(&st.rows[3][tok][4 * sub + 4 * LANES * q]);
-        k[4 * q] = kv.x; k[4 * q + 1] = kv.y; k[4 * q + 2] = kv.z; k[4 * q + 3] = kv.w;
-        rw[4 * q] = rv.x; rw[4 * q + 1] = rv.y; rw[4 * q + 2] = rv.z; rw[4 * q + 3] = rv.w;
-      }
-      float sum_k[COLS], sum_r[COLS];
-#pragma unroll
-      for (int col = 0; col < COLS; ++col) {
-        float dk[2] = {0.f, 0.f}, dr[2] = {0.f, 0.f};
-#pragma unroll
-        for (int e = 0; e < PER; ++e) {
-          dk[e & 1] += k[e] * S[col][e];
-          dr[e & 1] += rw[e] * S[col][e];
-        }
-        sum_k[col] = dk[0] + dk[1];
-        sum_r[col] = dr[0] + dr[1];
-      }
-#pragma unroll
-      for (int offset = 1; offset < LANES; offset <<= 1)
+        const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(rows + 4 * LANES * q);
+        const ulonglong2 rv = *reinterpret_cast<const ulonglong2*>(rows + 3 * KD + 4 * LANES * q);
+        k[2 * q] = kv.x;
+        k[2 * q + 1] = kv.y;
 #pragma unroll
         for (int col = 0; col < COLS; ++col) {
-          sum_k[col] += __shfl_xor_sync(0xffffffffu, sum_k[col], offset);
-          sum_r[col] += __shfl_xor_sync(0xffffffffu, sum_r[col], offset);
+          dot_k[col] = fma2(kv.x, S[col][2 * q], dot_k[col]);
+          dot_r[col] = fma2(rv.x, S[col][2 * q], dot_r[col]);
+          dot_k[col] = fma2(kv.y, S[col][2 * q + 1], dot_k[col]);
+          dot_r[col] = fma2(rv.y, S[col][2 * q + 1], dot_r[col]);
         }
-      float g[COLS], v[COLS];
+      }
+      float sums[2 * COLS];
 #pragma unroll
       for (int col = 0; col < COLS; ++col) {
-        g[col] = numbers.x * sum_k[col];
-        v[col] = st.v[tok][group * COLS + col];
-        if (sub == col && j0 + col < a.dim)
-          a.out[((size_t)(tile + tok) * a.heads + head) * a.dim + j0 + col] = sum_r[col] + v[col] * numbers.y - g[col] * numbers.z;
+        const float2 hk = unpack2(dot_k[col]), hr = unpack2(dot_r[col]);
+        sums[col] = hk.x + hk.y;
+        sums[COLS + col] = hr.x + hr.y;
       }
+      const float mine = Fold::run(sums, sub);
+      Pair g2[COLS], v2[COLS];
+      float o = 0.f;
+#pragma unroll
+      for (int col = 0; col < COLS; ++col) {
+        const float g = -numbers.x * __shfl_sync(0xffffffffu, mine, base + Fold::holder(col));
+        const float v = values[col];
+        if (col == out_col) o = mine + v * numbers.y + g * numbers.z;
+        g2[col] = pack2(g, g);
+        v2[col] = pack2(v, v);
+      }
+      if (out_col >= 0) *out_at = o;
+      out_at += out_stride;
 #pragma unroll
       for (int q = 0; q < PER / 4; ++q) {
-        const float4 wv = *reinterpret_cast<const float4*>(&st.rows[1][tok][4 * sub + 4 * LANES * q]);
-        const float4 av = *reinterpret_cast<const float4*>(&st.rows[2][tok][4 * sub + 4 * LANES * q]);
-        const float w[4] = {wv.x, wv.y, wv.z, wv.w}, rate[4] = {av.x, av.y, av.z, av.w};
+        const ulonglong2 wv = *reinterpret_cast<const ulonglong2*>(rows + KD + 4 * LANES * q);
+        const ulonglong2 av = *reinterpret_cast<const ulonglong2*>(rows + 2 * KD + 4 * LANES * q);
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-#pragma unroll
-          for (int col = 0; col < COLS; ++col)
-            S[col][4 * q + e] = w[e] * S[col][4 * q + e] + k[4 * q + e] * (v[col] - rate[e] * g[col]);
+        for (int col = 0; col < COLS; ++col) {
+          S[col][2 * q] = fma2(k[2 * q], fma2(av.x, g2[col], v2[col]), mul2(wv.x, S[col][2 * q]));
+          S[col][2 * q + 1] = fma2(k[2 * q + 1], fma2(av.y, g2[col], v2[col]), mul2(wv.y, S[col][2 * q + 1]));
+        }
       }
     }
     __syncthreads();  // everyone is done with this stage before the copies of the tile after next land in it
@@ -516,12 +570,13 @@ __global__ void __launch_bounds__(kDeltaThreads) channel_delta_kernel(DeltaArgs 
   for (int col = 0; col < COLS; ++col) {
     if (j0 + col >= a.dim) continue;
 #pragma unroll
-    for (int q = 0; q < PER / 4; ++q)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = 4 * sub + 4 * LANES * q + e;
-        if (i < a.dim) held[(size_t)(j0 + col) * a.dim + i] = S[col][4 * q + e];
-      }
+    for (int p = 0; p < PER / 2; ++p) {
+      const int i = 4 * sub + 4 * LANES * (p / 2) + 2 * (p % 2);
+      const float2 s = unpack2(S[col][p]);
+      float* dst = held + (size_t)(j0 + col) * a.dim + i;
+      if (i < a.dim) dst[0] = s.x;
+      if (i + 1 < a.dim) dst[1] = s.y;
+    }
   }
 }
 
@@ -530,7 +585,7 @@ static cudaError_t launch_delta(const DeltaArgs& a, int num_seqs, bool vec, cuda
   constexpr int TILE = KD >= 128 ? 8 : 16;
   constexpr int CB = kDeltaThreads / LANES * COLS;
   const dim3 grid(num_seqs, a.heads, (a.dim + CB - 1) / CB);
-  const size_t shared = 2 * sizeof(DeltaStage<KD, TILE, CB>);
+  const size_t shared = 2 * sizeof(DeltaStage<KD, TILE>);
   auto run = [&](auto kernel) {
     if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     kernel<<<grid, kDeltaThreads, shared, stream>>>(a);
@@ -540,18 +595,19 @@ static cudaError_t launch_delta(const DeltaArgs& a, int num_seqs, bool vec, cuda
   return cudaGetLastError();
 }
 
-// shape = 16 * lanes + columns of a thread; sizes a head has no room for fall back to the smallest.
+// lanes and columns of a thread as asked for, where a head has room for them.
 template <int KD>
 static cudaError_t dispatch_delta(const DeltaArgs& a, int num_seqs, bool vec, int lanes, int cols, cudaStream_t stream) {
   if constexpr (KD >= 128) {
     if (lanes == 32 && cols == 1) return launch_delta<KD, 32, 1>(a, num_seqs, vec, stream);
-    if (lanes == 32 && cols == 2) return launch_delta<KD, 32, 2>(a, num_seqs, vec, stream);
-    if (lanes == 32) return launch_delta<KD, 32, 4>(a, num_seqs, vec, stream);
+    if (lanes == 32) return launch_delta<KD, 32, 2>(a, num_seqs, vec, stream);
   }
   if constexpr (KD >= 64) {
     if (lanes >= 16 && cols == 1) return launch_delta<KD, 16, 1>(a, num_seqs, vec, stream);
+    if (lanes >= 16 && cols == 4) return launch_delta<KD, 16, 4>(a, num_seqs, vec, stream);
     if (lanes >= 16) return launch_delta<KD, 16, 2>(a, num_seqs, vec, stream);
   }
+  if (cols >= 4) return launch_delta<KD, 8, 4>(a, num_seqs, vec, stream);
   if (cols >= 2) return launch_delta<KD, 8, 2>(a, num_seqs, vec, stream);
   return launch_delta<KD, 8, 1>(a, num_seqs, vec, stream);
 }
@@ -599,9 +655,11 @@ extern "C" int distie_selective_scan(const float* x, int x_stride, const float* 
   return err == cudaSuccess ? 0 : (int)err;
 }
 
+static int delta_width(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+
 // Floats of scratch of the delta rule below.
 extern "C" long long distie_channel_delta_scratch_floats(int tokens, int heads, int dim) {
-  return (long long)tokens * heads * (5LL * dim + 4);
+  return (long long)tokens * heads * (kDeltaNumbers + (long long)kDeltaRows * delta_width(dim));
 }
 
 // proj [tokens, 4 heads dim (+ more)] = [r | k | v | rate], decay [tokens, heads dim] (each a matrix or slices); out
@@ -610,7 +668,7 @@ extern "C" int distie_channel_delta(const float* proj, int proj_stride, int proj
                                     const float* decay, int decay_stride, int decay_splits, long long decay_split_stride,
                                     const float* decay_bias, const float* rate_bias, float* state, float* out,
                                     float* scratch, const int* seq_bounds, const int* seq_seat, int tokens, int num_seqs,
-                                    int heads, int dim, int lanes, int cols, cudaStream_t stream) {
+                                    int heads, int dim, int lanes, int cols, int* error, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (heads < 1 || heads > 65535 || dim < 1 || num_seqs < 1 || proj_splits < 1 || decay_splits < 1 || !scratch || !state ||
       ((uintptr_t)scratch & 15))
@@ -620,8 +678,7 @@ extern "C" int distie_channel_delta(const float* proj, int proj_stride, int proj
   a.proj = Sliced{proj, proj_stride, proj_splits, proj_split_stride};
   a.decay = Sliced{decay, decay_stride, decay_splits, decay_split_stride};
   a.decay_bias = decay_bias; a.rate_bias = rate_bias;
-  a.numbers = scratch;  // first: its rows of four floats stay aligned whatever dim is
-  a.rows = scratch + (size_t)tokens * heads * 4;
+  a.scratch = scratch; a.width = delta_width(dim); a.error = error;
   a.state = state; a.out = out; a.seq_bounds = seq_bounds; a.seq_seat = seq_seat;
   a.tokens = tokens; a.heads = heads; a.dim = dim;
   channel_delta_prepare_kernel<<<dim3(tokens, tokens < 512 ? (heads + 3) / 4 : 1), 128, 0, stream>>>(a);

@@ -41,7 +41,7 @@ _ERROR_TEXT = {
     2: "a new token's page is missing from its block table (cache write)",
     3: "a block table does not cover the keys a token attends to",
     4: "a block table does not cover the keys a decoded token attends to",
-    6: "a tensor-core product gave up waiting for its own copies or instructions",
+    6: "a kernel gave up waiting for its own copies or instructions",
     7: "a router chose an expert that does not exist",
     5: "a block table does not cover the keys a portion of a prompt attends to",
 }
@@ -676,7 +676,8 @@ class DeviceKernels(KernelSet):
             function("distie_channel_delta")(
                 *self._sliced(proj, "channel_delta"), *self._sliced(decay, "channel_delta decay"), decay_bias.data_ptr(),
                 rate_bias.data_ptr(), state.data_ptr(), out.data_ptr(), scratch.data_ptr(), self._seq_index(step)[1].data_ptr(),
-                step.seq_seat.data_ptr(), tokens, step.num_seqs, heads, dim, lanes, cols, self._stream(),
+                step.seq_seat.data_ptr(), tokens, step.num_seqs, heads, dim, lanes, cols,
+                self.error_flag.data_ptr(), self._stream(),
             ),
             "channel_delta",
         )
