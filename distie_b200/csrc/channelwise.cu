@@ -349,7 +349,6 @@ static cudaError_t dispatch_select(const SelectArgs& a, T* out, int rows, bool t
 // and returns).
 // State layout: [seat, head, value element, key channel].
 // ---------------------------------------------------------------------------
-constexpr int kDeltaThreads = 64;
 constexpr float kDecayFactor = 0.6065306597126334f;  // exp(-1/2)
 constexpr int kDeltaNumbers = 4, kDeltaRows = 5;     // of a token and head
 
@@ -405,14 +404,14 @@ __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t b
 
 // The sums of NV values over groups of LANES neighbouring lanes with few exchanges: every round hands half of the values
 // to a neighbour and keeps the other half; when one value a lane is left, the rest of the group is summed by butterflies.
-// Afterwards lane `holder(i)` (and the lanes that agree with it in the low bits) has the sum of value i in v[0].
+// Afterwards v[0] of a lane is the sum of value `value_of(lane)`.
 template <int NV, int LANES>
 struct FoldedSum {
   __host__ __device__ static constexpr int bits() { return NV == 2 ? 1 : NV == 4 ? 2 : 3; }
-  __host__ __device__ static constexpr int holder(int value) {
-    int lane = 0;
-    for (int b = 0; b < bits(); ++b) lane |= ((value >> (bits() - 1 - b)) & 1) << b;
-    return lane;
+  static __device__ __forceinline__ int value_of(int lane) {
+    int value = 0;
+    for (int b = 0; b < bits(); ++b) value |= ((lane >> b) & 1) << (bits() - 1 - b);
+    return value;
   }
   static __device__ __forceinline__ float run(float (&v)[NV], int sub) {
 #pragma unroll
@@ -438,17 +437,17 @@ struct DeltaStage {
 };
 
 // VEC: columns of the state start on 16-byte boundaries.
-template <int KD, int LANES, int COLS, int TILE, bool VEC>
-__global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaArgs a) {
-  constexpr int PER = KD / LANES, CB = kDeltaThreads / LANES * COLS;
-  using Fold = FoldedSum<2 * COLS, LANES>;  // the sums with k, then with r * w, of every column
-  static_assert(PER >= 4 && PER % 4 == 0 && 2 * COLS <= LANES, "a thread holds whole float4s of its columns");
+template <int KD, int LANES, int COLS, int TILE, int THREADS, bool VEC>
+__global__ void __launch_bounds__(THREADS, 256 / THREADS) channel_delta_kernel(DeltaArgs a) {
+  constexpr int PER = KD / LANES, CB = THREADS / LANES * COLS;
+  using Fold = FoldedSum<TILE, LANES>;  // of a tile's read-outs of one column
+  static_assert(PER >= 4 && PER % 4 == 0 && TILE <= LANES, "a thread holds whole float4s of its columns");
   extern __shared__ __align__(16) unsigned char delta_smem[];
   using Stage = DeltaStage<KD, TILE>;
   Stage* stages = reinterpret_cast<Stage*>(delta_smem);  // two
   __shared__ __align__(8) uint64_t full[2];
   const int row = blockIdx.x, head = blockIdx.y;
-  const int tid = threadIdx.x, sub = tid % LANES, group = tid / LANES, base = (tid & 31) & ~(LANES - 1);
+  const int tid = threadIdx.x, sub = tid % LANES, group = tid / LANES;
   const int j0 = blockIdx.z * CB + group * COLS;
   const int first = a.seq_bounds[row], end = a.seq_bounds[row + 1];
   if (end <= first) return;
@@ -488,13 +487,11 @@ __global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaAr
       S[col][2 * q + 1] = pack2(s.z, s.w);
     }
 
-  // The lane whose folded sum is the read-out's of a column stores it.
-  int out_col = -1;
-#pragma unroll
-  for (int col = 0; col < COLS; ++col)
-    if (sub == Fold::holder(COLS + col) && j0 + col < a.dim) out_col = col;
+  // The read-outs of a tile wait as the lanes' own parts and are summed together: afterwards a lane holds the whole of one
+  // token's, which it stores.
+  const int out_tok = Fold::value_of(sub);
   const size_t out_stride = (size_t)a.heads * a.dim;
-  float* out_at = a.out + (size_t)first * out_stride + head * a.dim + j0 + max(out_col, 0);
+  float* out_at = a.out + (size_t)(first + out_tok) * out_stride + head * a.dim + j0;
 
   int round = 0;
   for (int tile = first; tile < end; tile += TILE, ++round) {
@@ -510,8 +507,14 @@ __global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaAr
       return;
     }
     const Stage& st = stages[buffer];
-#pragma unroll 2
-    for (int tok = 0; tok < count; ++tok) {
+    float part[COLS][TILE];
+#pragma unroll
+    for (int tok = 0; tok < TILE; ++tok) {
+      if (tok >= count) {
+#pragma unroll
+        for (int col = 0; col < COLS; ++col) part[col][tok] = 0.f;
+        continue;
+      }
       const float* piece = st.piece[tok];
       const float4 numbers = *reinterpret_cast<const float4*>(piece);
       const float* rows = piece + kDeltaNumbers + 4 * sub;
@@ -527,32 +530,29 @@ __global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaAr
         k[2 * q + 1] = kv.y;
 #pragma unroll
         for (int col = 0; col < COLS; ++col) {
-          dot_k[col] = fma2(kv.x, S[col][2 * q], dot_k[col]);
-          dot_r[col] = fma2(rv.x, S[col][2 * q], dot_r[col]);
-          dot_k[col] = fma2(kv.y, S[col][2 * q + 1], dot_k[col]);
-          dot_r[col] = fma2(rv.y, S[col][2 * q + 1], dot_r[col]);
+          dot_k[col] = fma2(kv.y, S[col][2 * q + 1], fma2(kv.x, S[col][2 * q], dot_k[col]));
+          dot_r[col] = fma2(rv.y, S[col][2 * q + 1], fma2(rv.x, S[col][2 * q], dot_r[col]));
         }
       }
-      float sums[2 * COLS];
+      float sum_k[COLS];
 #pragma unroll
       for (int col = 0; col < COLS; ++col) {
-        const float2 hk = unpack2(dot_k[col]), hr = unpack2(dot_r[col]);
-        sums[col] = hk.x + hk.y;
-        sums[COLS + col] = hr.x + hr.y;
+        const float2 h = unpack2(dot_k[col]);
+        sum_k[col] = h.x + h.y;
       }
-      const float mine = Fold::run(sums, sub);
+#pragma unroll
+      for (int offset = 1; offset < LANES; offset <<= 1)
+#pragma unroll
+        for (int col = 0; col < COLS; ++col) sum_k[col] += __shfl_xor_sync(0xffffffffu, sum_k[col], offset);
       Pair g2[COLS], v2[COLS];
-      float o = 0.f;
 #pragma unroll
       for (int col = 0; col < COLS; ++col) {
-        const float g = -numbers.x * __shfl_sync(0xffffffffu, mine, base + Fold::holder(col));
-        const float v = values[col];
-        if (col == out_col) o = mine + v * numbers.y + g * numbers.z;
+        const float g = -numbers.x * sum_k[col], v = values[col];
+        const float2 h = unpack2(dot_r[col]);
+        part[col][tok] = h.x + h.y + (sub == 0 ? v * numbers.y + g * numbers.z : 0.f);
         g2[col] = pack2(g, g);
         v2[col] = pack2(v, v);
       }
-      if (out_col >= 0) *out_at = o;
-      out_at += out_stride;
 #pragma unroll
       for (int q = 0; q < PER / 4; ++q) {
         const ulonglong2 wv = *reinterpret_cast<const ulonglong2*>(rows + KD + 4 * LANES * q);
@@ -564,6 +564,12 @@ __global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaAr
         }
       }
     }
+#pragma unroll
+    for (int col = 0; col < COLS; ++col) {
+      const float o = Fold::run(part[col], sub);
+      if (sub < TILE && out_tok < count && j0 + col < a.dim) out_at[col] = o;
+    }
+    out_at += TILE * out_stride;
     __syncthreads();  // everyone is done with this stage before the copies of the tile after next land in it
   }
 #pragma unroll
@@ -580,36 +586,44 @@ __global__ void __launch_bounds__(kDeltaThreads, 4) channel_delta_kernel(DeltaAr
   }
 }
 
-template <int KD, int LANES, int COLS>
-static cudaError_t launch_delta(const DeltaArgs& a, int num_seqs, bool vec, cudaStream_t stream) {
-  constexpr int TILE = KD >= 128 ? 8 : 16;
-  constexpr int CB = kDeltaThreads / LANES * COLS;
+template <int KD, int LANES, int COLS, int THREADS>
+static cudaError_t launch_delta_as(const DeltaArgs& a, int num_seqs, bool vec, cudaStream_t stream) {
+  constexpr int TILE = 8;
+  constexpr int CB = THREADS / LANES * COLS;
   const dim3 grid(num_seqs, a.heads, (a.dim + CB - 1) / CB);
   const size_t shared = 2 * sizeof(DeltaStage<KD, TILE>);
   auto run = [&](auto kernel) {
     if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
-    kernel<<<grid, kDeltaThreads, shared, stream>>>(a);
+    kernel<<<grid, THREADS, shared, stream>>>(a);
   };
-  if (vec) run(channel_delta_kernel<KD, LANES, COLS, TILE, true>);
-  else run(channel_delta_kernel<KD, LANES, COLS, TILE, false>);
+  if (vec) run(channel_delta_kernel<KD, LANES, COLS, TILE, THREADS, true>);
+  else run(channel_delta_kernel<KD, LANES, COLS, TILE, THREADS, false>);
   return cudaGetLastError();
+}
+
+template <int KD, int LANES, int COLS>
+static cudaError_t launch_delta(const DeltaArgs& a, int num_seqs, bool vec, int threads, cudaStream_t stream) {
+  if (threads >= 256) return launch_delta_as<KD, LANES, COLS, 256>(a, num_seqs, vec, stream);
+  if (threads >= 128) return launch_delta_as<KD, LANES, COLS, 128>(a, num_seqs, vec, stream);
+  return launch_delta_as<KD, LANES, COLS, 64>(a, num_seqs, vec, stream);
 }
 
 // lanes and columns of a thread as asked for, where a head has room for them.
 template <int KD>
-static cudaError_t dispatch_delta(const DeltaArgs& a, int num_seqs, bool vec, int lanes, int cols, cudaStream_t stream) {
+static cudaError_t dispatch_delta(const DeltaArgs& a, int num_seqs, bool vec, int lanes, int cols, int threads,
+                                  cudaStream_t stream) {
   if constexpr (KD >= 128) {
-    if (lanes == 32 && cols == 1) return launch_delta<KD, 32, 1>(a, num_seqs, vec, stream);
-    if (lanes == 32) return launch_delta<KD, 32, 2>(a, num_seqs, vec, stream);
+    if (lanes == 32 && cols == 1) return launch_delta<KD, 32, 1>(a, num_seqs, vec, threads, stream);
+    if (lanes == 32) return launch_delta<KD, 32, 2>(a, num_seqs, vec, threads, stream);
   }
   if constexpr (KD >= 64) {
-    if (lanes >= 16 && cols == 1) return launch_delta<KD, 16, 1>(a, num_seqs, vec, stream);
-    if (lanes >= 16 && cols == 4) return launch_delta<KD, 16, 4>(a, num_seqs, vec, stream);
-    if (lanes >= 16) return launch_delta<KD, 16, 2>(a, num_seqs, vec, stream);
+    if (lanes >= 16 && cols == 1) return launch_delta<KD, 16, 1>(a, num_seqs, vec, threads, stream);
+    if (lanes >= 16 && cols == 4) return launch_delta<KD, 16, 4>(a, num_seqs, vec, threads, stream);
+    if (lanes >= 16) return launch_delta<KD, 16, 2>(a, num_seqs, vec, threads, stream);
   }
-  if (cols >= 4) return launch_delta<KD, 8, 4>(a, num_seqs, vec, stream);
-  if (cols >= 2) return launch_delta<KD, 8, 2>(a, num_seqs, vec, stream);
-  return launch_delta<KD, 8, 1>(a, num_seqs, vec, stream);
+  if (cols >= 4) return launch_delta<KD, 8, 4>(a, num_seqs, vec, threads, stream);
+  if (cols >= 2) return launch_delta<KD, 8, 2>(a, num_seqs, vec, threads, stream);
+  return launch_delta<KD, 8, 1>(a, num_seqs, vec, threads, stream);
 }
 
 }  // namespace distie
@@ -668,7 +682,8 @@ extern "C" int distie_channel_delta(const float* proj, int proj_stride, int proj
                                     const float* decay, int decay_stride, int decay_splits, long long decay_split_stride,
                                     const float* decay_bias, const float* rate_bias, float* state, float* out,
                                     float* scratch, const int* seq_bounds, const int* seq_seat, int tokens, int num_seqs,
-                                    int heads, int dim, int lanes, int cols, int* error, cudaStream_t stream) {
+                                    int heads, int dim, int lanes, int cols, int threads, int* error,
+                                    cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (heads < 1 || heads > 65535 || dim < 1 || num_seqs < 1 || proj_splits < 1 || decay_splits < 1 || !scratch || !state ||
       ((uintptr_t)scratch & 15))
@@ -685,9 +700,9 @@ extern "C" int distie_channel_delta(const float* proj, int proj_stride, int proj
   DISTIE_LAUNCH_CHECK();
   const bool vec = dim % 4 == 0 && ((uintptr_t)state & 15) == 0;
   cudaError_t err;
-  if (dim <= 32) err = dispatch_delta<32>(a, num_seqs, vec, lanes, cols, stream);
-  else if (dim <= 64) err = dispatch_delta<64>(a, num_seqs, vec, lanes, cols, stream);
-  else if (dim <= 128) err = dispatch_delta<128>(a, num_seqs, vec, lanes, cols, stream);
-  else err = dispatch_delta<256>(a, num_seqs, vec, lanes, cols, stream);
+  if (dim <= 32) err = dispatch_delta<32>(a, num_seqs, vec, lanes, cols, threads, stream);
+  else if (dim <= 64) err = dispatch_delta<64>(a, num_seqs, vec, lanes, cols, threads, stream);
+  else if (dim <= 128) err = dispatch_delta<128>(a, num_seqs, vec, lanes, cols, threads, stream);
+  else err = dispatch_delta<256>(a, num_seqs, vec, lanes, cols, threads, stream);
   return err == cudaSuccess ? 0 : (int)err;
 }

@@ -671,12 +671,12 @@ class DeviceKernels(KernelSet):
         out = torch.empty((tokens, heads * dim), dtype=torch.float32, device=proj.device)
         floats = function("distie_channel_delta_scratch_floats")(tokens, heads, dim)
         scratch = torch.empty(floats, dtype=torch.float32, device=proj.device)
-        lanes, cols = (16, 1) if step.num_decode_tokens < tokens else (8, 1)
+        lanes, cols, threads = (16, 1, 128) if step.num_decode_tokens < tokens else (8, 1, 64)
         check(
             function("distie_channel_delta")(
                 *self._sliced(proj, "channel_delta"), *self._sliced(decay, "channel_delta decay"), decay_bias.data_ptr(),
                 rate_bias.data_ptr(), state.data_ptr(), out.data_ptr(), scratch.data_ptr(), self._seq_index(step)[1].data_ptr(),
-                step.seq_seat.data_ptr(), tokens, step.num_seqs, heads, dim, lanes, cols,
+                step.seq_seat.data_ptr(), tokens, step.num_seqs, heads, dim, lanes, cols, threads,
                 self.error_flag.data_ptr(), self._stream(),
             ),
             "channel_delta",

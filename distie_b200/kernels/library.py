@@ -70,7 +70,7 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
         "state", [P, I, P, I, I, L, P, P, I, I, L, P, I, I, L, P, P, P, P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, P]
     ),
     "distie_selective_scan_scratch_floats": ("state", [I, I, I]),
-    "distie_channel_delta": ("state", [P, I, I, L, P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P, P]),
+    "distie_channel_delta": ("state", [P, I, I, L, P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P]),
     "distie_channel_delta_scratch_floats": ("state", [I, I, I]),
     "distie_exp_gate_scan": ("state", [P, P, I, I, L, P, P, F, P, P, P, I, I, I, P, P, P, P]),
     "distie_stabilized_readout": ("state", [P, I, P, P, I, I, I, P]),
