@@ -4,6 +4,7 @@ from .engine_config import EngineConfig, resolve_dtype_name
 from .model_spec import LayerCall, LayerSpec, ModelSpec, PartSpec
 from .qwen2_config import ConfigError, Qwen2Config
 from .fovudra_config import FovudraConfig
+from .labolix_config import LabolixConfig
 from .mekusun_config import MekusunConfig
 from .zelasun_config import ZelasunConfig
 from .zururax_config import ZururaxConfig
@@ -23,6 +24,7 @@ __all__ = [
     "ConfigError",
     "EngineConfig",
     "FovudraConfig",
+    "LabolixConfig",
     "LayerCall",
     "LayerSpec",
     "MekusunConfig",

@@ -45,8 +45,10 @@ CUDA_UNITS: dict[str, list[str]] = {
     "base": ["elementwise.cu", "normed_residual.cu", "attention_generic.cu", "attention_decode.cu", "sampling.cu"],
     # bfloat16 serving only: tensor-core attention for prompts, weight-streaming products for decoding
     "bf16": ["attention_prefill.cu", "attention_decode_mma.cu", "gemm_tcgen05.cu", "attention_prefill_tcgen05.cu"],
-    # models with layer norms, gated heads, short convolutions, linear recurrences or selective scans (both dtypes)
-    "state": ["recurrent.cu", "channelwise.cu"],
+    # models with layer norms, gated heads, short convolutions or linear recurrences (both dtypes)
+    "state": ["recurrent.cu"],
+    # models with recurrences whose decay varies by channel (both dtypes); a unit of its own because it takes minutes
+    "channel": ["channelwise.cu"],
     # models whose feed-forward routes tokens to experts (both dtypes)
     "routed": ["routed.cu"],
     # models whose attention reads one latent row per token; gated and squared-ReLU activations on float32 products

@@ -90,6 +90,16 @@ __device__ __forceinline__ void store_row_f32(const float (&v)[32], float* __res
 // row: an instruction then writes four whole 128-byte lines.
 constexpr int kEpilogueStageBytes = 32 * 32 * 4;  // per epilogue warp
 
+// A gated hidden element for 16-bit stores: silu(g) * u, or with limit > 0 the capped form, which is
+// min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1).
+__device__ __forceinline__ float gated_value(float g, float u, float limit) {
+  if (limit > 0.f) {
+    const float gc = fminf(g, limit), uc = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(gc * (uc + 1.f), 1.f + __expf(-1.702f * gc));
+  }
+  return __fdividef(g * u, 1.f + __expf(-g));
+}
+
 template <int BN, int EPI>
 __device__ __forceinline__ void store_accumulator(uint32_t lane_base, int row0, int lane, int n0,
                                                   void* __restrict__ out, int ldo, int M, int N, int inter, int part,
@@ -107,12 +117,7 @@ __device__ __forceinline__ void store_accumulator(uint32_t lane_base, int row0, 
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
         const float g = __uint_as_float(gate[j]), u = __uint_as_float(up[j]);
-        if (limit > 0.f) {  // the capped form: min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1)
-          const float gc = fminf(g, limit), uc = fminf(fmaxf(u, -limit), limit);
-          v[j] = gc * (uc + 1.f) / (1.f + expf(-1.702f * gc));
-        } else {
-          v[j] = __fdividef(g * u, 1.f + __expf(-g));
-        }
+        v[j] = gated_value(g, u, limit);
       }
       const int col = n0 + c0;
       if (lane < rows_valid && col < inter)
@@ -180,7 +185,7 @@ struct QkvEpilogue {
   __nv_bfloat16* k_cache;
   __nv_bfloat16* v_cache;
   int num_heads, num_kv_heads, head_dim, page_size;
-  HiddenAct act;         // GEMM_EPI_ACT only: the activation of the plain epilogue
+  HiddenAct act;         // GEMM_EPI_ACT: the activation of the plain epilogue; GEMM_EPI_SWIGLU: act.a is the limit (0: none)
 };
 
 // The epilogue of the q/k/v projection of prompt portions: bias, rotation of q and k (pairs (j, j + head_dim / 2),
@@ -418,8 +423,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         if (qkv.head_dim == 128) store_qkv_rope<128>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
         else store_qkv_rope<64>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
       } else {
-        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage, 0.f,
-                                   qkv.act);
+        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage,
+                                   qkv.act.a, qkv.act);
       }
       // This warp has read its part of the accumulator: hand the buffer back to the MMA issuer.
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -746,8 +751,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
         if (qkv.head_dim == 128) store_qkv_rope<128>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
         else store_qkv_rope<64>(lane_base, m0 + quadrant * 32, lane, n0, part, (__nv_bfloat16*)out, ldo, M, N, qkv, trig_stage);
       } else {
-        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage, 0.f,
-                                   qkv.act);
+        store_accumulator<BN, EPI>(lane_base, m0 + quadrant * 32, lane, n0, out, ldo, M, N, inter, part, epilogue_stage,
+                                   qkv.act.a, qkv.act);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
@@ -944,7 +949,7 @@ gemm_tcgen05_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
           for (int j = j0; j < j0 + 8; ++j) {
             if (c0 + j < M) {
               const float g = sm.exchange[pair][j], u = sm.exchange[64 + pair][j];
-              out[(size_t)(c0 + j) * ldo + col] = from_float<OutT>(__fdividef(g * u, 1.f + __expf(-g)));
+              out[(size_t)(c0 + j) * ldo + col] = from_float<OutT>(gated_value(g, u, act.a));
             }
           }
         }
@@ -1075,7 +1080,8 @@ extern "C" int distie_gemm_tcgen05(const void* x, int ldx, const void* w, void* 
   return distie_gemm_tcgen05_act(x, ldx, w, out, ldo, M, N, K, epi, tile_width, 0, 0.f, 0.f, sm_count, error, stream);
 }
 
-// The same; epi 4: out[M, N] bfloat16 = act(x w^T) with the activation of code `kind` and its factors a and b.
+// The same; epi 4: out[M, N] bfloat16 = act(x w^T) with the activation of code `kind` and its factors a and b; epi 2 with
+// a > 0: the capped gate with that limit (gated_value).
 extern "C" int distie_gemm_tcgen05_act(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
                                        int epi, int tile_width, int kind, float a, float b, int sm_count, int* error,
                                        cudaStream_t stream) {
@@ -1094,7 +1100,7 @@ extern "C" int distie_gemm_tcgen05_act(const void* x, int ldx, const void* w, vo
     // Pairs of CTAs on 256-row tiles; each CTA stages half of the tile's rows of W.
     if (epi == GEMM_EPI_SWIGLU) {
       if ((status = make_map(&map_b, w, N, K, K, 128)) != 0) return status;
-      return launch_gemm_pair<256, 6, 1, GEMM_EPI_SWIGLU>(map_a, map_b, out, ldo, M, N, K, N / 2, sm_count, error, stream);
+      return launch_gemm_pair<256, 6, 1, GEMM_EPI_SWIGLU>(map_a, map_b, out, ldo, M, N, K, N / 2, sm_count, error, stream, more);
     }
     if (epi != GEMM_EPI_F32 && epi != GEMM_EPI_BF16 && epi != GEMM_EPI_ACT) return DISTIE_ERR_ARG;
     const int width = tile_width ? tile_width : pick_tile_width(M, N, 2 * kGemmBM, sm_count / 2);
@@ -1115,7 +1121,7 @@ extern "C" int distie_gemm_tcgen05_act(const void* x, int ldx, const void* w, vo
   if (epi == GEMM_EPI_SWIGLU) {
     status = make_map(&map_b, w, N, K, K, 128);
     if (status != 0) return status;
-    return launch_gemm<256, 4, GEMM_EPI_SWIGLU>(map_a, map_b, out, ldo, M, N, K, N / 2, sm_count, error, stream);
+    return launch_gemm<256, 4, GEMM_EPI_SWIGLU>(map_a, map_b, out, ldo, M, N, K, N / 2, sm_count, error, stream, more);
   }
   if (epi != GEMM_EPI_F32 && epi != GEMM_EPI_BF16 && epi != GEMM_EPI_ACT) return DISTIE_ERR_ARG;
   const int width = tile_width ? tile_width : pick_tile_width(M, N, kGemmBM, sm_count);
@@ -1310,6 +1316,7 @@ extern "C" int distie_gemm_tcgen05_skinny_splits(int N, int K, int sm_count) {
 //   mode 1: out[M, N] bfloat16 (out_dtype 1) or float32 (0) = x w^T + bias
 //   mode 2: w is [2 * inter, K]; out[M, inter] bfloat16 = silu(x Wg^T) * (x Wu^T)
 //   mode 3 (the entry point below with an activation): out[M, N] bfloat16 = act(x w^T)
+//   mode 2 with a limit has an entry point of its own: the capped gate (gated_value)
 extern "C" int distie_gemm_tcgen05_skinny_act(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
                                               int kind, float a, float b, int sm_count, int* error, cudaStream_t stream) {
   if (M <= 0) return 0;
@@ -1322,6 +1329,19 @@ extern "C" int distie_gemm_tcgen05_skinny_act(const void* x, int ldx, const void
   if (status != 0) return status;
   return dispatch_skinny_tc<SKINNY_EPI_ACT, __nv_bfloat16>(map_w, x, ldx, nullptr, (__nv_bfloat16*)out, ldo, M, N, K, 0,
                                                            (N + kGemmBM - 1) / kGemmBM, 1, error, stream, HiddenAct{kind, a, b});
+}
+
+extern "C" int distie_gemm_tcgen05_skinny_glu(const void* x, int ldx, const void* w, void* out, int ldo, int M, int N, int K,
+                                              float limit, int* error, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (M > 64 || N < 2 || (N & 1) || K < 8 || (K & 7) || (ldx & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
+    return DISTIE_ERR_UNSUPPORTED;
+  CUtensorMap map_w;
+  const int status = make_map(&map_w, w, N, K, K, 64);
+  if (status != 0) return status;
+  const int inter = N / 2;
+  return dispatch_skinny_tc<SKINNY_EPI_SWIGLU, __nv_bfloat16>(map_w, x, ldx, nullptr, (__nv_bfloat16*)out, ldo, M, N, K, inter,
+                                                              (inter + 63) / 64, 1, error, stream, HiddenAct{0, limit, 0.f});
 }
 
 extern "C" int distie_gemm_tcgen05_skinny(const void* x, int ldx, const void* w, const float* bias, void* out, int ldo,

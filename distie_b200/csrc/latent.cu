@@ -171,7 +171,7 @@ glu_act_kernel(const float* __restrict__ x, int row_stride, int slices, long lon
 
 // ---- attention over the stored rows: the size-agnostic kernel ----------------------------------------------------
 // A block takes one token, HB of its heads and one of `splits` equal parts of the keys the token sees
-// (positions 0 .. pos of its request).  A warp takes every fourth key of the part: it loads the key's row once
+// (positions 0 .. pos of its request, or with window > 0 the last `window` of them).  A warp takes every fourth key of the part: it loads the key's row once
 // (RMAX elements a lane) and uses it for all HB heads, as key (the whole row against [folded | rotated]) and as
 // value (its first `rank` columns).  Online softmax per head in float32; the warps' results are merged through
 // shared memory.  With one split the block divides by the sum, to which the head's sink adds exp(sink); with
@@ -185,7 +185,7 @@ latent_attention_kernel(const T* __restrict__ folded, const T* __restrict__ rota
                         float* __restrict__ partial, int tokens, int heads, int rank, int rot,
                         const int* __restrict__ positions, const int* __restrict__ token_seq,
                         const int* __restrict__ seq_seat, const int* __restrict__ block_table, int table_width,
-                        const T* __restrict__ k_cache, int page_size, int num_pages, float scale,
+                        const T* __restrict__ k_cache, int page_size, int num_pages, float scale, int window,
                         const float* __restrict__ sink, int splits, int first, int* __restrict__ error) {
   extern __shared__ float latent_s[];
   constexpr int kRow = RMAX * 32;
@@ -209,9 +209,9 @@ latent_attention_kernel(const T* __restrict__ folded, const T* __restrict__ rota
   const int pos = positions[t];
   const int seat = seq_seat[token_seq[t]];
   const int* table = block_table + (size_t)seat * table_width;
-  const int count = pos + 1;
-  const int per = (count + splits - 1) / splits;
-  const int begin = split * per, end = min(count, begin + per);
+  const int first_key = first_visible_key(pos, window, 0);
+  const int per = (pos + 1 - first_key + splits - 1) / splits;
+  const int begin = first_key + split * per, end = min(pos + 1, begin + per);
 
   float m[HB], l[HB], acc[HB][RMAX];
 #pragma unroll
@@ -356,8 +356,8 @@ template <typename T, int RMAX, int HB>
 static int launch_latent_attention(const void* folded, const void* rotated, void* out, float* partial, int tokens,
                                    int heads, int rank, int rot, const int* positions, const int* token_seq,
                                    const int* seq_seat, const int* block_table, int table_width, const void* k_cache,
-                                   int page_size, int num_pages, float scale, const float* sink, int splits,
-                                   int first, int count, int* error, cudaStream_t stream) {
+                                   int page_size, int num_pages, float scale, int window, const float* sink,
+                                   int splits, int first, int count, int* error, cudaStream_t stream) {
   const size_t shared = ((size_t)HB * RMAX * 32 + (size_t)kLatentWarps * HB * rank + kLatentWarps * HB * 2) * sizeof(float);
   auto kernel = latent_attention_kernel<T, RMAX, HB>;
   if (shared > 48 * 1024) {
@@ -367,7 +367,7 @@ static int launch_latent_attention(const void* folded, const void* rotated, void
   const dim3 grid(count, (heads + HB - 1) / HB, splits);
   kernel<<<grid, kLatentWarps * 32, shared, stream>>>((const T*)folded, (const T*)rotated, (T*)out, partial, tokens, heads,
                                                       rank, rot, positions, token_seq, seq_seat, block_table, table_width,
-                                                      (const T*)k_cache, page_size, num_pages, scale, sink, splits, first, error);
+                                                      (const T*)k_cache, page_size, num_pages, scale, window, sink, splits, first, error);
   DISTIE_LAUNCH_CHECK();
   if (splits > 1) {
     latent_merge_kernel<T><<<dim3(count, heads, (rank + 127) / 128), 128, 0, stream>>>(partial, (T*)out, tokens, heads, rank, splits, sink, first);
@@ -380,13 +380,13 @@ template <typename T>
 static int latent_attention_any(const void* folded, const void* rotated, void* out, float* partial, int tokens, int heads,
                                 int rank, int rot, const int* positions, const int* token_seq, const int* seq_seat,
                                 const int* block_table, int table_width, const void* k_cache, int page_size,
-                                int num_pages, float scale, const float* sink, int splits, int first, int count,
-                                int* error, cudaStream_t stream) {
+                                int num_pages, float scale, int window, const float* sink, int splits, int first,
+                                int count, int* error, cudaStream_t stream) {
   const int row = rank + rot;
 #define DISTIE_LATENT(RMAX, HB)                                                                                     \
   return launch_latent_attention<T, RMAX, HB>(folded, rotated, out, partial, tokens, heads, rank, rot, positions,  \
                                               token_seq, seq_seat, block_table, table_width, k_cache, page_size,   \
-                                              num_pages, scale, sink, splits, first, count, error, stream)
+                                              num_pages, scale, window, sink, splits, first, count, error, stream)
   if (row <= 128) DISTIE_LATENT(4, 8);
   if (row <= 256) DISTIE_LATENT(8, 8);
   if (row <= 512) DISTIE_LATENT(16, 4);
@@ -458,7 +458,7 @@ extern "C" long long distie_latent_attention_scratch_floats(int tokens, int head
 extern "C" int distie_latent_attention(const void* folded, const void* rotated, void* out, float* partial, int tokens,
                                        int heads, int rank, int rot, const int* positions, const int* token_seq,
                                        const int* seq_seat, const int* block_table, int table_width,
-                                       const void* k_cache, int page_size, int num_pages, float scale,
+                                       const void* k_cache, int page_size, int num_pages, float scale, int window,
                                        const float* sink, int splits, int first, int count, int dtype, int* error,
                                        cudaStream_t stream) {
   if (tokens <= 0 || count <= 0) return 0;
@@ -470,11 +470,11 @@ extern "C" int distie_latent_attention(const void* folded, const void* rotated, 
   if (dtype == DISTIE_BF16)
     return latent_attention_any<__nv_bfloat16>(folded, rotated, out, partial, tokens, heads, rank, rot, positions,
                                                token_seq, seq_seat, block_table, table_width, k_cache, page_size,
-                                               num_pages, scale, sink, splits, first, count, error, stream);
+                                               num_pages, scale, window, sink, splits, first, count, error, stream);
   if (dtype == DISTIE_F32)
     return latent_attention_any<float>(folded, rotated, out, partial, tokens, heads, rank, rot, positions, token_seq,
-                                       seq_seat, block_table, table_width, k_cache, page_size, num_pages, scale, sink,
-                                       splits, first, count, error, stream);
+                                       seq_seat, block_table, table_width, k_cache, page_size, num_pages, scale, window,
+                                       sink, splits, first, count, error, stream);
   return DISTIE_ERR_UNSUPPORTED;
 }
 

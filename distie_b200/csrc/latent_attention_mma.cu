@@ -26,7 +26,9 @@
 // (token, head), the unnormalised sum, its maximum (natural-log units) and its sum of weights, in the layout that
 // the size-agnostic kernel's merge reads; the sink joins in the merge.
 //
-// Key j is visible to the row at position p iff j <= p.  It depends on positions only, so the result does not depend
+// Key j is visible to the row at position p iff j <= p and (window <= 0 or j > p - window); blocks before the window of
+// the tile's first row are not visited and rows before it are not looked up (their pages may have been given back).  It
+// depends on positions only, so the result does not depend
 // on how the prompt was cut.  rank and rot multiples of 8 (16-byte copies), rank <= VC, rank + rot <= ROW; other
 // sizes are refused (-2) and the caller uses the size-agnostic kernel.
 #include "common.cuh"
@@ -81,8 +83,8 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ folded, const __nv
                             const int* __restrict__ token_seq, const int* __restrict__ seq_seat,
                             const int* __restrict__ block_table, int table_width,
                             const __nv_bfloat16* __restrict__ k_cache, int page_size, int page_shift, int num_pages,
-                            float scale_log2, const float* __restrict__ sink, float* __restrict__ partial,
-                            int first, int* __restrict__ error) {
+                            float scale_log2, int window, const float* __restrict__ sink,
+                            float* __restrict__ partial, int first, int* __restrict__ error) {
   constexpr int kLmRows = 16 * RG;            // rows of a tile: tokens of a portion, or heads of a single token
   constexpr int kLmThreads = RG * kLmParts * 32;
   constexpr int CHUNKS = ROW / 8;
@@ -120,10 +122,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ folded, const __nv
   const int seat = seq_seat[token_seq[t0]];
   const int* table = block_table + (size_t)seat * table_width;
   const int p_last = SINGLE ? p0 : p0 + rows - 1;
-  int block_begin = 0, block_end = p_last / kLmKeys + 1;
+  const int first_key = first_visible_key(p0, window, 0);  // the oldest key any row of the tile sees
+  int block_begin = first_key / kLmKeys, block_end = p_last / kLmKeys + 1;
   if (SINGLE && gridDim.z > 1) {
-    const int per = (block_end + gridDim.z - 1) / gridDim.z;
-    block_begin = min(block_end, (int)blockIdx.z * per);
+    const int per = (block_end - block_begin + gridDim.z - 1) / gridDim.z;
+    block_begin = min(block_end, block_begin + (int)blockIdx.z * per);
     block_end = min(block_end, block_begin + per);
   }
   const int live_chunks = row_len / 8;               // chunks of a row that hold data; the rest stay zero
@@ -150,7 +153,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ folded, const __nv
     for (int r = warp; r < kLmKeys; r += kLmThreads / 32) {
       const int key = kb + r;
       const __nv_bfloat16* src = k_cache;
-      bool ok = key <= p_last;
+      bool ok = key <= p_last && key >= first_key;
       if (ok) {
         const int column = page_shift >= 0 ? key >> page_shift : key / page_size;
         const int within = page_shift >= 0 ? key & (page_size - 1) : key % page_size;
@@ -248,7 +251,8 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ folded, const __nv
     // ---- mask and block maximum -------------------------------------------------------------------------------
     const int kb = block * kLmKeys + kh * 16;
     float tile_max[2] = {-INFINITY, -INFINITY};
-    if (kb + 15 <= (SINGLE ? p0 : p0 + rg * 16)) {  // wholly visible to every row of the warp
+    if (kb + 15 <= (SINGLE ? p0 : p0 + rg * 16) &&
+        kb >= first_visible_key(SINGLE ? p0 : p0 + rg * 16 + 15, window, 0)) {  // wholly visible to every row of the warp
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -259,7 +263,8 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ folded, const __nv
 #pragma unroll
         for (int r = 0; r < 4; ++r) {
           const int key = kb + i * 8 + 2 * c + (r & 1);
-          s[i][r] = key <= pos_row[r >> 1] ? s[i][r] : -INFINITY;
+          const int p = pos_row[r >> 1];
+          s[i][r] = key <= p && key >= first_visible_key(p, window, 0) ? s[i][r] : -INFINITY;
           tile_max[r >> 1] = fmaxf(tile_max[r >> 1], s[i][r]);
         }
       }
@@ -375,7 +380,7 @@ template <int ROW, int VC, int RG, bool SINGLE>
 static int launch_latent_mma(const void* folded, const void* rotated, void* out, int tokens, int heads, int rank, int rot,
                              const int* q_tiles, int num_tiles, const int* positions, const int* token_seq,
                              const int* seq_seat, const int* block_table, int table_width, const void* k_cache,
-                             int page_size, int num_pages, float scale, const float* sink, float* partial, int first,
+                             int page_size, int num_pages, float scale, int window, const float* sink, float* partial, int first,
                              int count, int splits, int* error, cudaStream_t stream) {
   constexpr int kRows = 16 * RG;
   const size_t shared = (size_t)kRows * ROW * 2 + 2 * (size_t)kLmKeys * ROW * 2 + kRows * kLmKeys * 2 +
@@ -390,7 +395,7 @@ static int launch_latent_mma(const void* folded, const void* rotated, void* out,
   kernel<<<grid, RG * kLmParts * 32, shared, stream>>>(
       (const __nv_bfloat16*)folded, (const __nv_bfloat16*)rotated, (__nv_bfloat16*)out, tokens, heads, rank, rot, q_tiles,
       positions, token_seq, seq_seat, block_table, table_width, (const __nv_bfloat16*)k_cache, page_size, page_shift,
-      num_pages, scale * 1.4426950408889634f, sink, partial, first, error);
+      num_pages, scale * 1.4426950408889634f, window, sink, partial, first, error);
   DISTIE_LAUNCH_CHECK();
   return 0;
 }
@@ -406,8 +411,8 @@ extern "C" int distie_latent_attention_tiles(const void* folded, const void* rot
                                              int rank, int rot, const int* q_tiles, int num_tiles,
                                              const int* positions, const int* token_seq, const int* seq_seat,
                                              const int* block_table, int table_width, const void* k_cache,
-                                             int page_size, int num_pages, float scale, const float* sink, int* error,
-                                             cudaStream_t stream) {
+                                             int page_size, int num_pages, float scale, int window, const float* sink,
+                                             int* error, cudaStream_t stream) {
   if (num_tiles <= 0 || tokens <= 0) return 0;
   if (heads < 1 || rank < 1 || rot < 0 || page_size < 1 || table_width < 1) return DISTIE_ERR_ARG;
   if (rank % 8 || rot % 8 || !(scale > 0.f) || 2 * (long long)num_tiles > 65535) return -2;
@@ -415,7 +420,7 @@ extern "C" int distie_latent_attention_tiles(const void* folded, const void* rot
 #define DISTIE_LATENT_MMA(ROW, VC)                                                                                   \
   return launch_latent_mma<ROW, VC, 4, false>(folded, rotated, out, tokens, heads, rank, rot, q_tiles, num_tiles,    \
                                               positions, token_seq, seq_seat, block_table, table_width, k_cache,    \
-                                              page_size, num_pages, scale, sink, nullptr, 0, 0, 1, error, stream)
+                                              page_size, num_pages, scale, window, sink, nullptr, 0, 0, 1, error, stream)
   if (row <= 128) DISTIE_LATENT_MMA(128, 128);
   if (row <= 320 && rank <= 256) DISTIE_LATENT_MMA(320, 256);
   if (row <= 576 && rank <= 512) DISTIE_LATENT_MMA(576, 512);
@@ -430,7 +435,7 @@ extern "C" int distie_latent_attention_single(const void* folded, const void* ro
                                               int tokens, int heads, int rank, int rot, const int* positions,
                                               const int* token_seq, const int* seq_seat, const int* block_table,
                                               int table_width, const void* k_cache, int page_size, int num_pages,
-                                              float scale, const float* sink, int splits, int first, int count,
+                                              float scale, int window, const float* sink, int splits, int first, int count,
                                               int* error, cudaStream_t stream) {
   if (count <= 0 || tokens <= 0) return 0;
   if (heads < 1 || rank < 1 || rot < 0 || page_size < 1 || table_width < 1 || first < 0 || first + count > tokens ||
@@ -441,7 +446,7 @@ extern "C" int distie_latent_attention_single(const void* folded, const void* ro
 #define DISTIE_LATENT_ONE(ROW, VC, RG)                                                                               \
   return launch_latent_mma<ROW, VC, RG, true>(folded, rotated, out, tokens, heads, rank, rot, nullptr, 0, positions, \
                                               token_seq, seq_seat, block_table, table_width, k_cache, page_size,    \
-                                              num_pages, scale, sink, partial, first, count, splits, error, stream)
+                                              num_pages, scale, window, sink, partial, first, count, splits, error, stream)
 #define DISTIE_LATENT_SINGLE(ROW, VC)          \
   do {                                         \
     if (heads <= 16) DISTIE_LATENT_ONE(ROW, VC, 1); \

@@ -5,6 +5,7 @@
 //  * norm_add_rmsnorm: d = sum_j scale_j * term_j (float32); residual += d * rsqrt(mean(d^2) + eps_d) * w_d
 //    (or += d when there is no w_d), written back; out = residual * rsqrt(mean(residual^2) + eps) * w, cast
 //    once at the store.  One block per row; with a list of rows only those are made and the residual stays.
+//  * add_dynamic_tanh: residual += d, written back; out = tanh(alpha * residual) * w + b, element by element.
 //  * average_add_rmsnorm: the same with an average over depth between the sum and the second norm: the sum is the
 //    layer's own result X, kept as the next of the states so far, and the residual becomes a weighted sum of them all.
 //  * qk_rope_norm_write: from the float32 projection [q | k] (a matrix or the slices of a split product) plus
@@ -123,6 +124,57 @@ norm_add_rmsnorm_vec_kernel(ResidualTerms terms, const float* __restrict__ delta
       const float4 w = *reinterpret_cast<const float4*>(weight + c);
       store4(out_row + c, make_float4(r[p].x * unit * w.x, r[p].y * unit * w.y, r[p].z * unit * w.z, r[p].w * unit * w.w));
     }
+  }
+}
+
+// residual += sum of the terms (float32, written back); out = tanh(alpha * residual) * weight + bias.  Nothing of a row is
+// measured, so the elements are spread over the machine whatever the rows are: four a thread (VEC: hidden a multiple of
+// 4, every pointer aligned to four elements) or one.  With a list of rows only those are made and the residual stays.
+// Launched as a dependent kernel: weight and bias are on their way before the producer of the terms has finished.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+add_dynamic_tanh_kernel(ResidualTerms terms, float* residual, float alpha, const float* __restrict__ weight,
+                        const float* __restrict__ bias, T* out, const int* rows_index, int hidden, long long units) {
+  grid_dependency_release();
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const bool live = idx < units;
+  const int per_row = VEC ? hidden / 4 : hidden;
+  const long long out_row = live ? idx / per_row : 0;
+  const int c = live ? (int)(idx - out_row * per_row) * (VEC ? 4 : 1) : 0;
+  if (VEC) {
+    const float4 w = *reinterpret_cast<const float4*>(weight + c), b = *reinterpret_cast<const float4*>(bias + c);
+    grid_dependency_wait();
+    if (!live) return;
+    const size_t row = rows_index ? (size_t)rows_index[out_row] : (size_t)out_row;
+    const size_t at = row * hidden + c;
+    float4 r = load4_cg(residual + at);
+    if (terms.count > 0) {
+      float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+      for (int j = 0; j < terms.count; ++j) {
+        const float4 v = load4_cg(terms.ptr[j] + at);
+        const float s = terms.scale[j];
+        d.x += s * v.x; d.y += s * v.y; d.z += s * v.z; d.w += s * v.w;
+      }
+      r.x += d.x; r.y += d.y; r.z += d.z; r.w += d.w;
+      if (!rows_index) *reinterpret_cast<float4*>(residual + at) = r;
+    }
+    store4(out + (size_t)out_row * hidden + c, make_float4(tanhf(alpha * r.x) * w.x + b.x, tanhf(alpha * r.y) * w.y + b.y,
+                                                           tanhf(alpha * r.z) * w.z + b.z, tanhf(alpha * r.w) * w.w + b.w));
+  } else {
+    const float w = weight[c], b = bias[c];
+    grid_dependency_wait();
+    if (!live) return;
+    const size_t row = rows_index ? (size_t)rows_index[out_row] : (size_t)out_row;
+    const size_t at = row * hidden + c;
+    float r = residual[at];
+    if (terms.count > 0) {
+      float d = 0.f;
+      for (int j = 0; j < terms.count; ++j) d += terms.scale[j] * terms.ptr[j][at];
+      r += d;
+      if (!rows_index) residual[at] = r;
+    }
+    out[(size_t)out_row * hidden + c] = from_float<T>(tanhf(alpha * r) * w + b);
   }
 }
 
@@ -465,6 +517,35 @@ extern "C" int distie_norm_add_rmsnorm(const float* const* term_ptrs, const floa
   }
   DISTIE_LAUNCH_CHECK();
   return 0;
+}
+
+extern "C" int distie_add_dynamic_tanh(const float* const* term_ptrs, const float* term_scales, int num_terms, float* residual,
+                                       float alpha, const float* weight, const float* bias, void* out,
+                                       const int* rows_index, int rows, int hidden, int dtype, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (hidden < 1 || num_terms < 0 || num_terms > kResidualTerms || !residual || !weight || !bias || !out) return DISTIE_ERR_ARG;
+  if (dtype != DISTIE_BF16 && dtype != DISTIE_F32) return DISTIE_ERR_UNSUPPORTED;
+  ResidualTerms terms;
+  terms.count = num_terms;
+  for (int j = 0; j < num_terms; ++j) { terms.ptr[j] = term_ptrs[j]; terms.scale[j] = term_scales[j]; }
+  uintptr_t low_bits = (uintptr_t)residual | (uintptr_t)weight | (uintptr_t)bias | (uintptr_t)out;
+  for (int j = 0; j < num_terms; ++j) low_bits |= (uintptr_t)term_ptrs[j];
+  const bool vec = hidden % 4 == 0 && (low_bits & 15) == 0;
+  const long long units = (long long)rows * (vec ? hidden / 4 : hidden);
+  const int threads = units < 148 * 256 ? 64 : 256;  // a step of few rows spreads over the machine
+  const long long blocks = (units + threads - 1) / threads;
+  if (blocks > 0x7fffffffLL) return DISTIE_ERR_UNSUPPORTED;
+  cudaError_t err;
+#define DISTIE_DYNAMIC_TANH(T, VECV)                                                                                        \
+  err = launch_dependent(add_dynamic_tanh_kernel<T, VECV>, dim3((unsigned)blocks), dim3(threads), 0, stream, terms, residual, \
+                         alpha, weight, bias, (T*)out, rows_index, hidden, units)
+  if (dtype == DISTIE_BF16) {
+    if (vec) DISTIE_DYNAMIC_TANH(__nv_bfloat16, true); else DISTIE_DYNAMIC_TANH(__nv_bfloat16, false);
+  } else {
+    if (vec) DISTIE_DYNAMIC_TANH(float, true); else DISTIE_DYNAMIC_TANH(float, false);
+  }
+#undef DISTIE_DYNAMIC_TANH
+  return err == cudaSuccess ? 0 : (int)err;
 }
 
 // As distie_norm_add_rmsnorm, with the average over depth of average_add_rmsnorm_kernel: history is [slots, rows of the

@@ -639,7 +639,7 @@ static cudaError_t launch_scan(const ScanArgs& a, int num_seqs, cudaStream_t str
 // RMS norm over groups of `group` neighbouring columns with a SiLU gate, a warp per (token, group):
 //   gate_first (bit 0 of the mode): norm(x * silu(gate)) * weight;   else: norm(x) * weight * silu(gate).
 //   bit 1 of the mode: sigmoid(gate) stands where silu(gate) does.
-// weight has `weight_len` elements and repeats along the row.
+// weight has `weight_len` elements and repeats along the row; null: no weight.
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, int x_stride, Sliced gate,
@@ -661,7 +661,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, int x_stride, 
   T* dst = out + (size_t)t * out_stride + (size_t)part * group;
   for (int i = lane; i < group; i += 32) {
     const float s = gate_f(gate_sigmoid, gate.at(t, part * group + i));
-    const float w = weight[(part * group + i) % weight_len];
+    const float w = weight ? weight[(part * group + i) % weight_len] : 1.f;
     dst[i] = from_float<T>(gate_first ? xr[i] * s * inv * w : xr[i] * inv * w * s);
   }
 }
@@ -704,7 +704,7 @@ gated_rmsnorm_vec_kernel(const float* __restrict__ x, int x_stride, Sliced gate,
     const int i = (p * LANES + lane) * 4;
     if (i < group) {
       const int at = (part * group + i) % weight_len;  // weight_len is a multiple of 4 here
-      const float4 w = *reinterpret_cast<const float4*>(weight + at);
+      const float4 w = weight ? *reinterpret_cast<const float4*>(weight + at) : make_float4(1.f, 1.f, 1.f, 1.f);
       float4 o = make_float4(v[p].x * inv * w.x, v[p].y * inv * w.y, v[p].z * inv * w.z, v[p].w * inv * w.w);
       if (!gate_first) o = make_float4(o.x * s[p].x, o.y * s[p].y, o.z * s[p].z, o.w * s[p].w);
       store4(dst + i, o);
@@ -712,6 +712,43 @@ gated_rmsnorm_vec_kernel(const float* __restrict__ x, int x_stride, Sliced gate,
   }
 }
 
+
+// ---------------------------------------------------------------------------
+// q and k of a linear attention, head by head (q's columns, then k's, then `rest` more), out of the float32 projection
+// (or its slices): each head's first rotary_dim elements rotated at the token's position, k times key_scale, the rest as
+// it is.  A block per token; its angles are made once and serve all heads.  Shared memory: rotary_dim floats.
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+rotate_heads_kernel(Sliced x, float* __restrict__ out, int out_stride, const int* __restrict__ positions,
+                    const float* __restrict__ inv_freq, float factor, int rotary_dim, int interleaved, int heads, int key_dim,
+                    float key_scale, int rest) {
+  extern __shared__ float trig_s[];
+  const int t = blockIdx.x, half = rotary_dim / 2;
+  const float pos = (float)positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf(pos * inv_freq[i], &sn, &cs);
+    trig_s[i] = cs * factor;
+    trig_s[half + i] = sn * factor;
+  }
+  __syncthreads();
+  float* dst = out + (size_t)t * out_stride;
+  const int end = heads * key_dim, per_head = key_dim - half;  // a thread takes a pair, or one of the elements behind them
+  for (int idx = threadIdx.x; idx < 2 * heads * per_head; idx += blockDim.x) {
+    const int head = idx / per_head, i = idx % per_head;
+    const float scale = head >= heads ? key_scale : 1.f;
+    const int base = head * key_dim;
+    if (i < half) {
+      const int a = base + (interleaved ? 2 * i : i), b = base + (interleaved ? 2 * i + 1 : i + half);
+      const float u = x.at(t, a), v = x.at(t, b), cs = trig_s[i], sn = trig_s[half + i];
+      dst[a] = (u * cs - v * sn) * scale;
+      dst[b] = (v * cs + u * sn) * scale;
+    } else {
+      dst[base + half + i] = x.at(t, base + half + i) * scale;
+    }
+  }
+  for (int c = 2 * end + threadIdx.x; c < 2 * end + rest; c += blockDim.x) dst[c] = x.at(t, c);
+}
 
 // ---------------------------------------------------------------------------
 // out[t, c] = act(x[t, c]) (* scale for c < scaled_columns), x a matrix or the slices of a split product.
@@ -1100,7 +1137,8 @@ extern "C" int distie_gated_rmsnorm(const float* x, int x_stride, const float* g
                                     int out_stride, int tokens, int n, int group, float eps, int gate_first, int dtype,
                                     cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (n < 1 || group < 1 || n % group || weight_len < 1 || splits < 1) return DISTIE_ERR_ARG;
+  if (n < 1 || group < 1 || n % group || (weight && weight_len < 1) || splits < 1) return DISTIE_ERR_ARG;
+  if (!weight) weight_len = 4;  // (not read)
   if (dtype != DISTIE_BF16 && dtype != DISTIE_F32) return DISTIE_ERR_UNSUPPORTED;
   const Sliced gate{gate_ptr, gate_stride, splits, split_stride};
   const int groups = n / group, warps = 4;
@@ -1130,6 +1168,21 @@ extern "C" int distie_gated_rmsnorm(const float* x, int x_stride, const float* g
   if (dtype == DISTIE_BF16) DISTIE_GATED(__nv_bfloat16);
   else DISTIE_GATED(float);
 #undef DISTIE_GATED
+  DISTIE_LAUNCH_CHECK();
+  return 0;
+}
+
+extern "C" int distie_rotate_heads(const float* x, int x_stride, int splits, long long split_stride, float* out, int out_stride,
+                                   const int* positions, const float* inv_freq, float factor, int rotary_dim, int interleaved,
+                                   int tokens, int heads, int key_dim, float key_scale, int rest, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (heads < 1 || key_dim < 1 || splits < 1 || rest < 0 || rotary_dim < 0 || (rotary_dim & 1) || rotary_dim > key_dim ||
+      (rotary_dim > 0 && !inv_freq) || out_stride < 2 * heads * key_dim + rest)
+    return DISTIE_ERR_ARG;
+  const size_t shared = (size_t)rotary_dim * sizeof(float);
+  if (shared > 48 * 1024) return DISTIE_ERR_UNSUPPORTED;
+  rotate_heads_kernel<<<tokens, 256, shared, stream>>>(Sliced{x, x_stride, splits, split_stride}, out, out_stride, positions,
+                                                       inv_freq, factor, rotary_dim, interleaved, heads, key_dim, key_scale, rest);
   DISTIE_LAUNCH_CHECK();
   return 0;
 }

@@ -507,6 +507,24 @@ class DeviceKernels(KernelSet):
         )
         self._ran("add_layernorm")
 
+    def add_dynamic_tanh(self, delta, residual, alpha, weight, bias, out, rows_index=None) -> None:
+        pairs = [] if delta is None else Terms.of(delta).flat()
+        if len(pairs) > _MAX_TERMS:  # more terms than the kernel takes: the tail is summed here, in float32
+            tail = Terms(pairs[_MAX_TERMS - 1 :]).total()
+            pairs = pairs[: _MAX_TERMS - 1] + [(tail, 1.0)]
+        pairs = [(t if t.is_contiguous() else t.contiguous(), s) for t, s in pairs]
+        pointers = (ctypes.c_void_p * max(1, len(pairs)))(*[t.data_ptr() for t, _ in pairs])
+        scales = (ctypes.c_float * max(1, len(pairs)))(*[s for _, s in pairs])
+        check(
+            function("distie_add_dynamic_tanh")(
+                pointers, scales, len(pairs), residual.data_ptr(), float(alpha), weight.data_ptr(), bias.data_ptr(),
+                out.data_ptr(), rows_index.data_ptr() if rows_index is not None else None, out.shape[0], residual.shape[1],
+                _CODE[out.dtype], self._stream(),
+            ),
+            "add_dynamic_tanh",
+        )
+        self._ran("add_dynamic_tanh")
+
     @staticmethod
     def _rows32(x: torch.Tensor, what: str) -> torch.Tensor:
         if x.dtype != torch.float32 or x.stride(-1) != 1:
@@ -622,7 +640,8 @@ class DeviceKernels(KernelSet):
         self._rows32(x, "gated_rmsnorm x")
         check(
             function("distie_gated_rmsnorm")(
-                x.data_ptr(), x.stride(0), *self._sliced(gate, "gated_rmsnorm gate"), weight.data_ptr(), weight.numel(),
+                x.data_ptr(), x.stride(0), *self._sliced(gate, "gated_rmsnorm gate"),
+                weight.data_ptr() if weight is not None else None, weight.numel() if weight is not None else 0,
                 out.data_ptr(), out.stride(0), x.shape[0], x.shape[1], group, float(eps),
                 int(bool(gate_first)) | (2 if activation == "sigmoid" else 0),
                 _CODE[out.dtype], self._stream(),
@@ -630,6 +649,21 @@ class DeviceKernels(KernelSet):
             "gated_rmsnorm",
         )
         self._ran("gated_rmsnorm")
+
+    def rotate_heads(self, qk, step, rotary, heads, key_dim, key_scale=1.0):
+        columns = qk.shape[-1]
+        out = torch.empty((step.num_tokens, columns), dtype=torch.float32, device=qk.device)
+        check(
+            function("distie_rotate_heads")(
+                *self._sliced(qk, "rotate_heads"), out.data_ptr(), out.stride(0), step.positions.data_ptr(),
+                rotary.inv_freq.data_ptr() if rotary is not None else None, float(rotary.factor) if rotary is not None else 1.0,
+                rotary.rotary_dim if rotary is not None else 0, int(rotary.interleaved) if rotary is not None else 0,
+                step.num_tokens, heads, key_dim, float(key_scale), columns - 2 * heads * key_dim, self._stream(),
+            ),
+            "rotate_heads",
+        )
+        self._ran("rotate_heads")
+        return out
 
     # -- recurrences whose decay varies by channel ------------------------------------------------------------------
     def selective_scan(self, x, dt, B, C, gate, rates, skip, dt_bias, state, step, out) -> None:
@@ -987,6 +1021,19 @@ class DeviceKernels(KernelSet):
             raise KernelError("linear_glu: gate rows and up rows are stacked, so the weight has an even number of rows")
         if limit is None and row_gate is None:
             return self.linear_swiglu(x, weight)
+        if row_gate is None and (self._skinny(x, weight) or self._tensor_core(x, weight)):  # in the product's epilogue
+            out = torch.empty((x.shape[0], weight.shape[0] // 2), dtype=self.dtype, device=x.device)
+            head = (x.data_ptr(), x.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0), x.shape[0], weight.shape[0],
+                    weight.shape[1])
+            error, stream = self.error_flag.data_ptr(), self._stream()
+            if self._skinny(x, weight):
+                check(function("distie_gemm_tcgen05_skinny_glu")(*head, float(limit), error, stream), "gemm_tcgen05_skinny_glu")
+                self._ran("gemm_tcgen05_skinny")
+            else:
+                check(function("distie_gemm_tcgen05_act")(*head, 2, 0, 0, float(limit), 0.0, self.sm_count, error, stream),
+                      "gemm_tcgen05_act")
+                self._ran("gemm_tcgen05")
+            return out
         if row_gate is not None and row_gate.dim() == 2 and row_gate.shape[-1] != 1:
             raise KernelError("linear_glu: the row gate is one logit per row")
         return self._glu_act(self.linear_split(x, weight), weight.shape[0] // 2, 0, limit, row_gate)
@@ -1052,10 +1099,11 @@ class DeviceKernels(KernelSet):
         # per head [T, dim] x [dim, kv_rank]: a batched library product (float32 accumulation; FMA-only in the float32 set)
         return torch.bmm(plain, up_keys), rotated
 
-    def latent_attention(self, folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, out) -> None:
+    def latent_attention(self, folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, out, window=None) -> None:
         if kv.k.dtype != folded.dtype or not folded.is_contiguous() or not rotated.is_contiguous() or not out.is_contiguous():
             raise KernelError("latent_attention: contiguous queries and output of the cache's type are expected")
         tokens = step.num_tokens
+        window = int(window) if window else 0
         sink_ptr = sink.data_ptr() if sink is not None else None
         # Portions of prompts: tiles of consecutive tokens of a request on the tensor cores.  Single tokens (they
         # come first in a step) and whatever the tiled kernel refuses go to the size-agnostic kernel.
@@ -1065,7 +1113,7 @@ class DeviceKernels(KernelSet):
                 folded.data_ptr(), rotated.data_ptr(), out.data_ptr(), tokens, num_heads, kv_rank, rot_dim,
                 step.q_tiles.data_ptr(), step.num_q_tiles, step.positions.data_ptr(), step.token_seq.data_ptr(),
                 step.seq_seat.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[-1], kv.k.data_ptr(),
-                kv.page_size, kv.num_pages, float(scale), sink_ptr, self.error_flag.data_ptr(), self._stream(),
+                kv.page_size, kv.num_pages, float(scale), window, sink_ptr, self.error_flag.data_ptr(), self._stream(),
             )
             if code != -2:
                 check(code, "latent_attention_tiles")
@@ -1075,7 +1123,7 @@ class DeviceKernels(KernelSet):
             return
         common = (tokens, num_heads, kv_rank, rot_dim, step.positions.data_ptr(), step.token_seq.data_ptr(),
                   step.seq_seat.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[-1], kv.k.data_ptr(),
-                  kv.page_size, kv.num_pages, float(scale), sink_ptr)
+                  kv.page_size, kv.num_pages, float(scale), window, sink_ptr)
 
         def scratch(splits: int):
             if splits <= 1:
@@ -1083,7 +1131,10 @@ class DeviceKernels(KernelSet):
             floats = function("distie_latent_attention_scratch_floats")(tokens, num_heads, kv_rank, splits)
             return torch.empty(floats, dtype=torch.float32, device=folded.device)
 
-        key_blocks = -(-max(int(step.max_kv_len), 1) // 64)
+        longest = max(int(step.max_kv_len), 1)
+        if window:
+            longest = min(longest, window + 63)  # a window may start inside a block of keys
+        key_blocks = -(-longest // 64)
         if self.dtype == torch.bfloat16:
             # Single tokens on the tensor cores: a token's heads are the rows of a tile, and ranges of whole key
             # blocks go to CTAs of their own until the machine is filled.

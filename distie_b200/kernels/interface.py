@@ -364,12 +364,12 @@ class KernelSet(ABC):
         raise NotImplementedError
 
     def latent_attention(self, folded, rotated, step: StepTensors, kv: KvSlot, num_heads: int, kv_rank: int,
-                         rot_dim: int, scale: float, sink, out) -> None:
+                         rot_dim: int, scale: float, sink, out, window: int | None = None) -> None:
         """Causal softmax attention of every token over its request's rows ``[latent | rotated key part]`` of
         ``kv.k``, shared by all heads: score ``(folded[h, t] . latent_j + rotated[t, h] . part_j) * scale`` for every
         ``j <= position``; with ``sink [heads]`` (float32) the denominator also holds ``exp(sink_h)``;
         ``out[h, t] = sum_j weight_j latent_j`` (``[heads, T, kv_rank]``, the set's dtype).  Scores, softmax and the
-        sum are float32."""
+        sum are float32.  With a ``window`` a token sees itself and the ``window - 1`` positions before it."""
         raise NotImplementedError
 
     def latent_values(self, mixed, up_values, gate, num_heads: int, value_dim: int):
@@ -386,6 +386,12 @@ class KernelSet(ABC):
         """residual += delta (float32, kept); out = (residual - mean) / sqrt(var + eps) * weight + bias, with the
         variance the mean of the squared deviations.  ``delta``: None, ``[T, hidden]``, float32 slices
         ``[S, T, hidden]`` or :class:`Terms`.  With ``rows_index`` only those rows, residual kept."""
+        raise NotImplementedError
+
+    def add_dynamic_tanh(self, delta, residual, alpha: float, weight, bias, out, rows_index=None) -> None:
+        """residual += delta (float32, kept); out = cast(tanh(alpha * residual) * weight + bias), float32 up to the one
+        cast.  ``delta``: None, ``[T, hidden]``, float32 slices ``[S, T, hidden]`` or :class:`Terms`.  With ``rows_index``
+        only those rows, residual kept."""
         raise NotImplementedError
 
     def kv_write(self, k, v, step: StepTensors, kv: KvSlot) -> None:
@@ -462,8 +468,29 @@ class KernelSet(ABC):
                       activation: str = "silu") -> None:
         """Root-mean-square norm over groups of ``group`` neighbouring columns of ``x [T, n]`` (float32) with
         a gate (float32, or slices; written ``silu`` below, ``activation="sigmoid"`` makes it ``sigmoid(gate)``): ``gate_first``: ``norm(x * silu(gate)) * weight``; else ``norm(x) * weight * silu(gate)``.
-        ``weight`` is float32 of ``n`` elements, or fewer, then repeated (``weight[column % len]``)."""
+        ``weight`` is float32 of ``n`` elements, or fewer, then repeated (``weight[column % len]``); None: no weight."""
         raise NotImplementedError
+
+    def rotate_heads(self, qk, step: StepTensors, rotary: RotaryTable | None, heads: int, key_dim: int, key_scale: float = 1.0):
+        """``qk [T, 2 * heads * key_dim (+ more)]`` float32 (any row stride, or slices): q head by head, then k.  Returns
+        float32 ``[T, n]`` of as many columns: q and k with each head's first ``rotary_dim`` elements rotated at the
+        token's position, k then times ``key_scale``; the columns behind them as they are."""
+        raise NotImplementedError
+
+    def retention(self, qkv, gate, rotary: RotaryTable | None, key_scale: float, decay, state, step: StepTensors, heads: int,
+                  key_dim: int, value_dim: int, weight, eps: float, activation: str, out) -> None:
+        """From the float32 projection ``qkv [T, 2 * heads * key_dim + heads * value_dim]`` (or slices) of a linear
+        attention with the constant ``decay [heads]`` to what its output projection reads: q and k rotated and k scaled
+        (:meth:`rotate_heads`), the state moved on and read (:meth:`linear_recurrence`, rule ``"gated"``), the read-out
+        normed and gated (:meth:`gated_rmsnorm`) into ``out [T, heads * value_dim]``.  ``weight`` None: every head is
+        normed by itself and has no weight; else all heads are normed together and multiplied by it.  The default is
+        the ops after one another; a set may merge them."""
+        qk = heads * key_dim
+        turned = self.rotate_heads(qkv, step, rotary, heads, key_dim, key_scale)
+        read = self.linear_recurrence("gated", turned[:, :qk], turned[:, qk : 2 * qk], turned[:, 2 * qk :], None, None, state, step,
+                                      heads, heads, key_dim, value_dim, decay_rate=decay)
+        group = value_dim if weight is None else heads * value_dim
+        self.gated_rmsnorm(read, gate, weight, eps, group, False, out, activation=activation)
 
     @abstractmethod
     def sample(self, logits, temperatures, uniforms, out_tokens) -> None:

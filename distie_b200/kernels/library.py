@@ -37,6 +37,7 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
         "base", [P, I, I, L, P, P, I, P, P, P, P, I, P, F, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, F, F, I, P, P]
     ),
     "distie_norm_add_rmsnorm": ("base", [P, P, I, P, F, P, P, F, P, P, I, I, I, P]),
+    "distie_add_dynamic_tanh": ("base", [P, P, I, P, F, P, P, P, P, I, I, I, P]),
     "distie_average_add_rmsnorm": ("base", [P, P, I, P, F, P, P, L, I, I, P, P, F, P, P, I, I, I, P]),
     "distie_qk_rope_norm_write": (
         "base", [P, I, I, L, P, P, I, P, P, P, P, I, P, F, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P]
@@ -66,12 +67,13 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
         "state", [I, P, I, P, I, P, I, P, I, P, I, I, L, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, P]
     ),
     "distie_activation": ("state", [P, I, I, L, P, I, I, I, F, I, I, P]),
+    "distie_rotate_heads": ("state", [P, I, I, L, P, I, P, P, F, I, I, I, I, I, F, I, P]),
     "distie_selective_scan": (
-        "state", [P, I, P, I, I, L, P, P, I, I, L, P, I, I, L, P, P, P, P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, P]
+        "channel", [P, I, P, I, I, L, P, P, I, I, L, P, I, I, L, P, P, P, P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, P]
     ),
-    "distie_selective_scan_scratch_floats": ("state", [I, I, I]),
-    "distie_channel_delta": ("state", [P, I, I, L, P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P]),
-    "distie_channel_delta_scratch_floats": ("state", [I, I, I]),
+    "distie_selective_scan_scratch_floats": ("channel", [I, I, I]),
+    "distie_channel_delta": ("channel", [P, I, I, L, P, I, I, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P]),
+    "distie_channel_delta_scratch_floats": ("channel", [I, I, I]),
     "distie_exp_gate_scan": ("state", [P, P, I, I, L, P, P, F, P, P, P, I, I, I, P, P, P, P]),
     "distie_stabilized_readout": ("state", [P, I, P, P, I, I, I, P]),
     "distie_route_top": ("routed", [P, I, P, I, I, I, I, P, P, I, I, F, I, P, I, P, I, P, I, P]),
@@ -90,10 +92,10 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     ),
     "distie_latent_q_prepare": ("latent", [P, I, I, L, I, I, I, I, P, P, F, I, I, P, P, I, P]),
     "distie_latent_attention_scratch_floats": ("latent", [I, I, I, I]),
-    "distie_latent_attention": ("latent", [P, P, P, P, I, I, I, I, P, P, P, P, I, P, I, I, F, P, I, I, I, I, P, P]),
-    "distie_latent_attention_single": ("latent", [P, P, P, P, I, I, I, I, P, P, P, P, I, P, I, I, F, P, I, I, I, P, P]),
+    "distie_latent_attention": ("latent", [P, P, P, P, I, I, I, I, P, P, P, P, I, P, I, I, F, I, P, I, I, I, I, P, P]),
+    "distie_latent_attention_single": ("latent", [P, P, P, P, I, I, I, I, P, P, P, P, I, P, I, I, F, I, P, I, I, I, P, P]),
     "distie_latent_merge": ("latent", [P, P, I, I, I, I, P, I, I, I, P]),
-    "distie_latent_attention_tiles": ("latent", [P, P, P, I, I, I, I, P, I, P, P, P, P, I, P, I, I, F, P, P, P]),
+    "distie_latent_attention_tiles": ("latent", [P, P, P, I, I, I, I, P, I, P, P, P, P, I, P, I, I, F, I, P, P, P]),
     "distie_latent_gate": ("latent", [P, I, I, I, P, I, I, L, P, I, I, P]),
     "distie_glu_act": ("latent", [P, I, I, L, I, I, I, F, F, F, P, I, I, L, P, I, I, P]),
     "distie_gated_rmsnorm": ("state", [P, I, P, I, I, L, P, I, P, I, I, I, I, F, I, I, P]),
@@ -101,6 +103,7 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     "distie_gemm_tcgen05_act": ("bf16", [P, I, P, P, I, I, I, I, I, I, I, F, F, I, P, P]),
     "distie_gemm_tcgen05_qkv": ("bf16", [P, I, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, P, P]),
     "distie_gemm_tcgen05_skinny_splits": ("bf16", [I, I, I]),
+    "distie_gemm_tcgen05_skinny_glu": ("bf16", [P, I, P, P, I, I, I, I, F, P, P]),
     "distie_gemm_tcgen05_skinny_act": ("bf16", [P, I, P, P, I, I, I, I, I, F, F, I, P, P]),
     "distie_gemm_tcgen05_skinny": ("bf16", [P, I, P, P, P, I, I, I, I, I, I, I, P, P]),
 }

@@ -19,7 +19,7 @@ the tensors are called in the checkpoint; ``bias_suffix`` what a bias adds to it
 A second family of options makes the layer run on the *prepared* path (one stacked projection ``[q | k | v | g]``
 whose float32 accumulators are finished by one kernel before anything is rounded): ``sink`` (a learned number per
 head, ``sink [heads]``: the softmax's denominator also holds ``exp(sink_h)``; no key, no value, not scaled, not
-capped), ``softcap`` (``score <- cap * tanh(score / cap)`` after the scale), ``gate="sigmoid"`` (``g`` projects to
+capped), ``sink_score`` (the same with one given number for all heads and no tensor: 0 adds one to the denominator), ``softcap`` (``score <- cap * tanh(score / cap)`` after the scale), ``gate="sigmoid"`` (``g`` projects to
 ``heads * value_dim`` numbers and the concatenated heads are multiplied by ``sigmoid(g)`` element by element),
 ``norm_first`` (an epsilon: every head of q and k is divided by its root mean square BEFORE the rotation;
 ``norm_weights=True`` then multiplies by ``<q>.norm`` and ``<k>.norm``, ``[head_dim]`` each, shared by the heads),
@@ -47,7 +47,7 @@ class GqaAttention:
     ``window`` (None: full), ``chunk`` (None: none), ``value_dim`` (None: ``head_dim``), ``gate`` (None or
     ``"head_sigmoid"``), ``scale`` (None: ``head_dim**-0.5``), ``position`` (a PartSpec), ``names``, ``bias_suffix``,
     ``values`` (``"projected"`` or ``"keys"``), ``qk_norm`` (None or an epsilon), ``keep_first`` (0); and for the
-    prepared path ``sink`` (bool), ``softcap``, ``gate="sigmoid"``, ``norm_first`` (an epsilon), ``norm_weights``
+    prepared path ``sink`` (bool), ``sink_score`` (a number), ``softcap``, ``gate="sigmoid"``, ``norm_first`` (an epsilon), ``norm_weights``
     (bool), ``q_temp`` (``(coef, every)``), ``conv`` (taps).
 
     tensors: ``q_proj``/``k_proj``/``v_proj``/``o_proj`` ``.weight`` (and ``.bias``), ``g_proj.weight`` with a
@@ -90,7 +90,8 @@ class GqaAttention:
 
     @classmethod
     def _is_prepared(cls, params) -> bool:
-        return any(params.get(key) for key in cls._PREPARED) or params.get("gate") == "sigmoid"
+        return (any(params.get(key) for key in cls._PREPARED) or params.get("sink_score") is not None
+                or params.get("gate") == "sigmoid")
 
     @classmethod
     def _name(cls, spec: PartSpec, which: str, bias: bool = False) -> str:
@@ -120,7 +121,9 @@ class GqaAttention:
             raise ValueError(f"gate {params['gate']!r}: None, 'head_sigmoid' or 'sigmoid'")
         if cls._is_prepared(params):
             if params.get("values", "projected") == "keys" or params.get("qk_norm") is not None:
-                raise ValueError("sink, softcap, gate='sigmoid', norm_first, q_temp and conv go with projected values and no qk_norm")
+                raise ValueError("sink, sink_score, softcap, gate='sigmoid', norm_first, q_temp and conv go with projected values and no qk_norm")
+            if params.get("sink") and params.get("sink_score") is not None:
+                raise ValueError("sink is learned, sink_score is given: one of the two")
             if params.get("norm_weights") and params.get("norm_first") is None:
                 raise ValueError("norm_weights goes with norm_first")
             if params.get("softcap") is not None and float(params["softcap"]) <= 0:
@@ -225,6 +228,8 @@ class GqaAttention:
         extras = {}
         if prm.get("sink"):
             extras["sink"] = w.vector(cls._name(spec, "sink"))
+        elif prm.get("sink_score") is not None:
+            extras["sink"] = torch.full((int(prm["num_heads"]),), float(prm["sink_score"]), dtype=torch.float32, device=ctx.device)
         if prm.get("norm_weights"):
             extras["q_norm"], extras["k_norm"] = (w.vector(cls._stem(spec, n) + ".norm") for n in "qk")
         if int(prm.get("conv") or 0) > 0:

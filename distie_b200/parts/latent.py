@@ -8,7 +8,7 @@ Per token, with ``h`` the mixer's input::
     c   = rms_norm(d[:kv_rank]) * w_kv                key/value latent        [kv_rank]
     r   = rotate(d[kv_rank:], position)               one rotated key part, shared by all heads
     key_h = [W_uk,h c | r],  value_h = W_uv,h c
-    score_h(i, j) = (q_plain,h(i) . W_uk,h c(j) + rotate(q_rot,h(i)) . r(j)) * scale,   j <= i
+    score_h(i, j) = (q_plain,h(i) . W_uk,h c(j) + rotate(q_rot,h(i)) . r(j)) * scale,   j <= i  (with a window: i - j < window)
     weights = exp(score) / (sum_j exp(score) + exp(sink_h))       (``sink``: one learned number per head)
     out = W_o concat_h(sigmoid((W_g h)_h) * sum_j weights_h(i, j) value_h(j))
 
@@ -41,7 +41,7 @@ from .linear import fuse_rows
 class LatentAttention:
     """params: ``num_heads``, ``head_dim`` (plain query/key dimensions per head), ``rot_dim``, ``value_dim``,
     ``kv_rank``, ``q_rank`` (None: no query latent), ``scale``, ``eps`` (of the latent norms), ``position`` (a PartSpec; its table
-    rotates the ``rot_dim`` part), ``sink`` (bool), ``gate`` (None or ``"head_sigmoid"``), ``own_latent`` (bool),
+    rotates the ``rot_dim`` part), ``window`` (None: every earlier token is seen), ``sink`` (bool), ``gate`` (None or ``"head_sigmoid"``), ``own_latent`` (bool),
     ``names`` (what the tensors' names add to the prefix).
 
     tensors: ``dq [q_rank, hidden]``, ``dq.norm [q_rank]``, ``uq [heads * (head_dim + rot_dim), q_rank]`` (or, without a
@@ -64,6 +64,7 @@ class LatentAttention:
         self.q_rank = int(prm["q_rank"]) if prm["q_rank"] is not None else None
         self.scale = float(prm["scale"])
         self.eps = float(prm["eps"])
+        self.window = int(prm["window"]) if prm.get("window") is not None else None
         self.own_latent = bool(prm.get("own_latent", True))
         self.gated = bool(prm.get("gate"))
         self.down, self.q_norm, self.kv_norm = down, q_norm, kv_norm
@@ -79,6 +80,8 @@ class LatentAttention:
         for key in ("num_heads", "head_dim", "value_dim", "kv_rank", "q_rank"):
             if (key != "q_rank" or prm[key] is not None) and int(prm[key]) < 1:
                 raise ValueError(f"{key} must be >= 1, got {prm[key]}")
+        if prm.get("window") is not None and int(prm["window"]) < 1:
+            raise ValueError(f"window must be >= 1, got {prm['window']}")
         if int(prm["rot_dim"]) < 0:
             raise ValueError(f"rot_dim must be >= 0, got {prm['rot_dim']}")
         if int(prm["kv_rank"]) + int(prm["rot_dim"]) > 1024:
@@ -117,7 +120,8 @@ class LatentAttention:
         prm = spec.params
         if not prm.get("own_latent", True):
             return None
-        return CacheNeed(1, int(prm["kv_rank"]) + int(prm["rot_dim"]), value_dim=int(prm["kv_rank"]), values_in_keys=True)
+        return CacheNeed(1, int(prm["kv_rank"]) + int(prm["rot_dim"]), prm.get("window"), value_dim=int(prm["kv_rank"]),
+                         values_in_keys=True)
 
     @classmethod
     def state_need(cls, spec: PartSpec):
@@ -170,7 +174,7 @@ class LatentAttention:
         folded, rotated = k.latent_queries(q, self.up_keys, run.step, table, self.num_heads, self.head_dim, self.rot_dim)
         mixed = torch.empty((self.num_heads, tokens, self.kv_rank), dtype=x.dtype, device=x.device)
         k.latent_attention(folded, rotated, run.step, run.kv, self.num_heads, self.kv_rank, self.rot_dim, self.scale,
-                           self.sink, mixed)
+                           self.sink, mixed, self.window)
         gate = proj[..., proj.shape[-1] - self.num_heads :] if self.gated else None
         heads_out = k.latent_values(mixed, self.up_values, gate, self.num_heads, self.value_dim)
         return k.linear_split(heads_out, self.out)  # summed by the norm that follows

@@ -1,4 +1,5 @@
-"""Dense feed-forwards, no biases: SwiGLU ``down(silu(gate(x)) * up(x))`` and ``activated`` ``down(act(up(x)))``.
+"""Dense feed-forwards, no biases: SwiGLU ``down(silu(gate(x)) * up(x))``, its capped form, and ``activated``
+``down(act(up(x)))``.
 
 Formula of the reference (worker/src/inference/qwen2/model.py:228-236).  Gate and
 up are one product against the row-stacked weight ``[2 * inter, hidden]``.
@@ -19,14 +20,17 @@ from .linear import Linear, fuse_rows
 @FEED_FORWARDS.register("swiglu")
 class SwiGluFeedForward:
     """params: ``intermediate_size``; optional ``names``: what the names of the gate, up and down matrices add to
-    the prefix (default ``gate_proj.weight``, ``up_proj.weight``, ``down_proj.weight``)."""
+    the prefix (default ``gate_proj.weight``, ``up_proj.weight``, ``down_proj.weight``); ``limit`` (None: none): the
+    hidden activation is the capped form ``g' sigmoid(1.702 g') (u' + 1)`` with ``g' = min(g, limit)`` and ``u' = clamp(u,
+    -limit, limit)`` (see :meth:`KernelSet.linear_glu`)."""
 
     _NAMES = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
 
-    def __init__(self, gate_up: Linear, down: Linear, inter: int, kernels) -> None:
+    def __init__(self, gate_up: Linear, down: Linear, inter: int, kernels, limit: float | None = None) -> None:
         self.gate_up = gate_up
         self.down = down
         self.inter = inter
+        self.limit = limit
         self.kernels = kernels
 
     @classmethod
@@ -49,11 +53,21 @@ class SwiGluFeedForward:
             Linear(w.matrix(p + down), None, ctx.kernels),
             int(spec.params["intermediate_size"]),
             ctx.kernels,
+            cls._limit(spec),
         )
+
+    @staticmethod
+    def _limit(spec: PartSpec) -> float | None:
+        limit = spec.params.get("limit")
+        if limit is not None and float(limit) <= 0:
+            raise ValueError(f"limit must be positive, got {limit}")
+        return float(limit) if limit is not None else None
 
     def forward(self, x: torch.Tensor, run: LayerRun) -> torch.Tensor:
         # The down product's float32 slices are summed by the norm that follows (or by the stream).
-        return self.kernels.linear_split(self.kernels.linear_swiglu(x, self.gate_up.weight), self.down.weight)
+        k = self.kernels
+        hidden = k.linear_swiglu(x, self.gate_up.weight) if self.limit is None else k.linear_glu(x, self.gate_up.weight, self.limit)
+        return k.linear_split(hidden, self.down.weight)
 
 
 def _softplus(z: float) -> float:

@@ -7,6 +7,8 @@ itself be a norm of a sublayer's output (:class:`~distie_b200.kernels.interface.
 norms and the addition are one kernel.
 ``layernorm``: ``(x - mean) / sqrt(variance + eps) * weight + bias`` with the variance the mean of the
 squared deviations, all in float32 up to the store.
+``dynamic_tanh``: ``tanh(alpha * x) * weight + bias``, element by element: nothing of the row is measured; float32 up to
+the store.
 """
 
 from __future__ import annotations
@@ -107,3 +109,41 @@ class LayerNorm:
             self.kernels.average_add_rmsnorm(delta, residual, None, 0.0, None)
             delta = None
         self.kernels.add_layernorm(delta, residual, self.weight, self.bias, self.eps, out, rows)
+
+
+@NORMS.register("dynamic_tanh")
+class DynamicTanh:
+    """params: ``weight``, ``bias`` and ``alpha``: what the tensors' names add to the prefix (defaults ``"weight"``,
+    ``"bias"``, ``"alpha"``).  tensors: ``<prefix><weight> [hidden]``, ``<prefix><bias> [hidden]`` and the scalar
+    ``<prefix><alpha>``."""
+
+    def __init__(self, weight, bias, alpha: float, kernels) -> None:
+        self.weight = weight
+        self.bias = bias
+        self.alpha = float(alpha)
+        self.kernels = kernels
+
+    @staticmethod
+    def _names(spec: PartSpec) -> tuple[str, str, str]:
+        return tuple(spec.prefix + spec.params.get(which, which) for which in ("weight", "bias", "alpha"))
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, hidden_size: int) -> list[TensorSpec]:
+        weight, bias, alpha = cls._names(spec)
+        return [TensorSpec(weight, (hidden_size,), "norm"), TensorSpec(bias, (hidden_size,), "bias"),
+                TensorSpec(alpha, (), "norm")]
+
+    @classmethod
+    def build(cls, spec: PartSpec, ctx: BuildContext) -> "DynamicTanh":
+        weight, bias, alpha = cls._names(spec)
+        return cls(ctx.weights.vector(weight), ctx.weights.vector(bias), ctx.weights.vector(alpha).item(), ctx.kernels)
+
+    def apply(self, delta, residual, out, rows=None) -> None:
+        """``residual += delta`` (if any; a :class:`Terms` is summed in the kernel), ``out = norm(residual)``."""
+        if isinstance(delta, Averaged):  # averages and norms of a sublayer's output move the residual on by themselves
+            self.kernels.average_add_rmsnorm(delta, residual, None, 0.0, None)
+            delta = None
+        if isinstance(delta, Normed):
+            self.kernels.norm_add_rmsnorm(delta.value, delta.weight, delta.eps, residual, None, 0.0, None)
+            delta = None
+        self.kernels.add_dynamic_tanh(delta, residual, self.alpha, self.weight, self.bias, out, rows)

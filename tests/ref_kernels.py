@@ -136,6 +136,24 @@ def add_layernorm(delta, residual, weight, bias, eps, dtype, rows_index=None):
     return (summed if rows_index is None else residual), out
 
 
+def add_dynamic_tanh(delta, residual, alpha, weight, bias, dtype, rows_index=None):
+    """Returns (new residual, normed), like add_rmsnorm."""
+    d = flat_sum(delta)
+    summed = residual if d is None else residual + d
+    source = summed if rows_index is None else summed[rows_index.long()]
+    out = (torch.tanh(alpha * source) * weight.float() + bias.float()).to(dtype)
+    return (summed if rows_index is None else residual), out
+
+
+def rotate_heads(qk, step: StepTensors, rotary, heads, key_dim, key_scale=1.0):
+    out = whole(qk).clone()
+    tokens, end = step.num_tokens, heads * key_dim
+    for first, scale in ((0, 1.0), (end, key_scale)):
+        part = out[:tokens, first : first + end].reshape(tokens, heads, key_dim)
+        out[:tokens, first : first + end] = (rotate(part, step.positions[:tokens], rotary) * scale).reshape(tokens, end)
+    return out
+
+
 def token_seats(step: StepTensors):
     return step.seq_seat[step.token_seq[: step.num_tokens].long()].long()
 
@@ -230,7 +248,7 @@ def linear_recurrence(rule, q, k, v, decay, write, state, step: StepTensors, hea
 def gated_rmsnorm(x, gate, weight, eps, group, gate_first, dtype, activation="silu"):
     tokens, n = x.shape
     xf, gf = x.float(), (_silu(whole(gate)) if activation == "silu" else torch.sigmoid(whole(gate)))
-    w = weight.float().repeat(n // weight.numel())
+    w = weight.float().repeat(n // weight.numel()) if weight is not None else 1.0
     if gate_first:
         xf = xf * gf
     parts = xf.reshape(tokens, n // group, group)
@@ -548,13 +566,13 @@ def latent_queries(q, up_keys, step: StepTensors, rotary, num_heads, dim, rot_di
     return folded.contiguous(), rotated.contiguous()
 
 
-def latent_attention(folded, rotated, step: StepTensors, kv: KvSlot, num_heads, kv_rank, rot_dim, scale, sink):
+def latent_attention(folded, rotated, step: StepTensors, kv: KvSlot, num_heads, kv_rank, rot_dim, scale, sink, window=None):
     tokens = step.num_tokens
     out = torch.zeros((num_heads, tokens, kv_rank), dtype=folded.dtype, device=folded.device)
     for t in range(tokens):
         pos = int(step.positions[t])
         seat = int(step.seq_seat[int(step.token_seq[t])])
-        keys = torch.arange(0, pos + 1, device=folded.device)
+        keys = torch.arange(max(0, pos - int(window) + 1) if window else 0, pos + 1, device=folded.device)
         pages = kv.block_table[seat, keys // kv.page_size].long()
         if bool(((pages < 0) | (pages >= kv.num_pages)).any()):
             raise IndexError("a block table does not cover the keys a token attends to")
@@ -562,7 +580,7 @@ def latent_attention(folded, rotated, step: StepTensors, kv: KvSlot, num_heads, 
         scores = (folded[:, t].float() @ rows[:, :kv_rank].T + rotated[t].float() @ rows[:, kv_rank:].T) * scale  # [H, n]
         if sink is not None:
             scores = torch.cat([scores, sink.float()[:, None]], dim=1)
-        probs = torch.softmax(scores, dim=-1)[:, : pos + 1]
+        probs = torch.softmax(scores, dim=-1)[:, : keys.numel()]
         out[:, t] = (probs @ rows[:, :kv_rank]).to(folded.dtype)
     return out
 
@@ -685,8 +703,8 @@ class RefKernels(KernelSet):
     def latent_queries(self, q, up_keys, step, rotary, num_heads, dim, rot_dim):
         return latent_queries(q, up_keys, step, rotary, num_heads, dim, rot_dim, self.dtype)
 
-    def latent_attention(self, folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, out):
-        out.copy_(latent_attention(folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink))
+    def latent_attention(self, folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, out, window=None):
+        out.copy_(latent_attention(folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, window))
 
     def latent_values(self, mixed, up_values, gate, num_heads, value_dim):
         return latent_values(mixed, up_values, gate, num_heads, value_dim, self.dtype)
@@ -696,6 +714,15 @@ class RefKernels(KernelSet):
         if rows_index is None and delta is not None:
             residual.copy_(new_residual)
         out.copy_(normed)
+
+    def add_dynamic_tanh(self, delta, residual, alpha, weight, bias, out, rows_index=None):
+        new_residual, normed = add_dynamic_tanh(delta, residual, alpha, weight, bias, self.dtype, rows_index)
+        if rows_index is None and delta is not None:
+            residual.copy_(new_residual)
+        out.copy_(normed)
+
+    def rotate_heads(self, qk, step, rotary, heads, key_dim, key_scale=1.0):
+        return rotate_heads(qk, step, rotary, heads, key_dim, key_scale)
 
     def kv_write(self, k, v, step, kv):
         kv_write(k, v, step, kv)
