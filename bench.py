@@ -316,6 +316,27 @@ def mekusun_config(size: dict, layers: int) -> dict:
             "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "layers": [pattern[i % 4] for i in range(layers)]}
 
 
+def labolix_config(size: dict, layers: int, window: int) -> dict:
+    """The Labolix design at a Qwen2.5 layer's width, feed-forward and heads: attention with heads of 128 for keys and
+    values, wholly rotated, its long waves slowed by their wavelength; attention through a latent of 512 (heads of 128
+    plain and 64 rotated dimensions, values of 128) over a window of ``window`` positions; retention with heads of 128;
+    the capped dense feed-forward everywhere."""
+    heads, kv = size["heads"], size["kv_heads"]
+    mlp = {"kind": "dense", "ff": size["ff"], "limit": 7.0}
+    attention = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+        "rot": {"dims": 128, "base": 1e6, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "mask": {"size": window},
+        "rot": {"base": 1e6, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    retention = {"type": "retention", "mlp": mlp, "mixer": {
+        "heads": heads, "dim": 128, "vdim": 128, "rot": {"base": 1e6, "dims": 128},
+        "decay": [1.0 - 2.0 ** -(5 + 5 * h / max(1, heads - 1)) for h in range(heads)]}}
+    pattern = [retention, latent, retention, attention]
+    return {"architecture": "Labolix", "vocab": COMPARE_VOCAB, "width": size["width"], "norm": {"eps": 1e-6},
+            "logit_softcap": 30.0, "layers": [pattern[i % 4] for i in range(layers)]}
+
+
 def qwen2_config(size: dict, layers: int) -> dict:
     return {"architectures": ["Qwen2ForCausalLM"], "vocab_size": COMPARE_VOCAB, "hidden_size": size["width"],
             "intermediate_size": size["ff"], "num_hidden_layers": layers, "num_attention_heads": size["heads"],
@@ -324,10 +345,10 @@ def qwen2_config(size: dict, layers: int) -> dict:
 
 
 def compare_designs(args) -> int:
-    """``--compare zelasun`` (or ``fovudra``, ``zururax``, ``zuzunex``, ``mekusun``): prefill of 2,048 tokens and decode steps at batch ``--batch`` behind
+    """``--compare zelasun`` (or ``fovudra``, ``zururax``, ``zuzunex``, ``mekusun``, ``labolix``): prefill of 2,048 tokens and decode steps at batch ``--batch`` behind
     1,024-token prompts, for the named design beside the Qwen2 decoder (and, for Fovudra, beside Zelasun, the other
     design with recurrences; for Zururax, beside Fovudra, the other design with routed experts; for Mekusun, beside Zururax, the other design with
-    a latent, and Zelasun) at equal width, feed-forward, heads and depth.  Each model is
+    a latent, and Zelasun; for Labolix, beside Fovudra, the other design with a constant decay, and Zururax) at equal width, feed-forward, heads and depth.  Each model is
     built at two depths (4 and 8 layers) so that the time of a layer is the difference, free of embedding and head.
     One JSON line; not the repository's headline metric."""
     import gc
@@ -343,7 +364,7 @@ def compare_designs(args) -> int:
     depths = (4, 8) if args.layers is None else (args.layers,)
     designs = {"zelasun": ("zelasun", "qwen2"), "fovudra": ("fovudra", "zelasun", "qwen2"),
                "zururax": ("zururax", "fovudra", "qwen2"), "zuzunex": ("zuzunex", "fovudra", "qwen2"),
-               "mekusun": ("mekusun", "zururax", "zelasun", "qwen2")}[args.compare]
+               "mekusun": ("mekusun", "zururax", "zelasun", "qwen2"), "labolix": ("labolix", "fovudra", "zururax", "qwen2")}[args.compare]
     if args.designs:
         designs = tuple(d for d in designs if d in args.designs.split(","))
     configs = {"zelasun": lambda size, depth: zelasun_config(size, depth, args.chunk),
@@ -351,6 +372,7 @@ def compare_designs(args) -> int:
                "zururax": lambda size, depth: zururax_config(size, depth),
                "zuzunex": lambda size, depth: zuzunex_config(size, depth),
                "mekusun": lambda size, depth: mekusun_config(size, depth),
+               "labolix": lambda size, depth: labolix_config(size, depth, args.chunk),
                "qwen2": lambda size, depth: qwen2_config(size, depth)}
     out = {"compare": " beside ".join(designs), "dtype": args.dtype, "batch": args.batch, "prompt_len": PROMPT_LEN,
            "prefill_tokens": PREFILL_TOKENS, "chunk": args.chunk, "sizes": {}}
@@ -610,10 +632,10 @@ def main() -> int:
                         help="with --impl reference: its attention backend (default: DISTIE_ATTN, else auto)")
     parser.add_argument("--ref-device", default=None, help=argparse.SUPPRESS)  # "cpu": a dry run of the reference arm
     parser.add_argument("--designs", default=None, help="with --compare: only these of its designs, with commas between them")
-    parser.add_argument("--compare", default=None, choices=["zelasun", "fovudra", "zururax", "zuzunex", "mekusun"],
+    parser.add_argument("--compare", default=None, choices=["zelasun", "fovudra", "zururax", "zuzunex", "mekusun", "labolix"],
                         help="time another design beside the Qwen2 decoder at equal layer sizes instead of the default run")
     parser.add_argument("--chunk", type=int, default=1024,
-                        help="with --compare: the chunk (Zelasun) or window (Fovudra) of the design's attention")
+                        help="with --compare: the chunk (Zelasun) or window (Fovudra, Labolix) of the design's attention")
     parser.add_argument("--only-size", default=None, choices=["1.5b", "7b"], help="with --compare: one of the sizes")
     args = parser.parse_args()
     if args.gpus != 1:

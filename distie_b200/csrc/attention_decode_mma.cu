@@ -94,7 +94,9 @@ struct ProjectionInput {
   int write_new;           // 0: the cache already holds the token's key and value (a layer that reads another's cache)
 };
 
-template <int D, int STAGES, int NH, bool PAGE16, bool FUSED>
+// RAGGED: keys of key_dim and values of value_dim elements, multiples of 8 up to D: the rest of a tile's row is filled with
+// zeros as it is copied, and only value_dim columns are stored (the partial results keep rows of D).
+template <int D, int STAGES, int NH, bool PAGE16, bool FUSED, bool RAGGED = false>
 __global__ void __launch_bounds__(kMmaDecodeWarps * 32)
 attention_decode_mma_kernel(const ProjectionInput proj,
                             const __nv_bfloat16* __restrict__ q, int q_row_stride, __nv_bfloat16* __restrict__ out,
@@ -104,12 +106,13 @@ attention_decode_mma_kernel(const ProjectionInput proj,
                             const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                             int num_heads, int group_size, int head_chunks, int num_kv_heads, int page_size,
                             int page_shift, int num_pages, int window, int key_chunk, int keep_first, float scale_log2, int cluster_merge,
-                            const ScoreExtras extras, int* __restrict__ error) {
+                            const ScoreExtras extras, int key_dim, int value_dim, int* __restrict__ error) {
   constexpr int CPR = D / 8;                 // 16-byte chunks per row of keys or values
   constexpr int ROW_BYTES = D * 2;
   constexpr int TILE_BYTES = 16 * ROW_BYTES;  // 16 keys (or values)
   constexpr int COPIES = 16 * CPR / 32;       // chunks a lane copies per tile
   constexpr int MT = D / 16;                  // 16-dim row tiles of O^T, and k-steps of S^T
+  const int KD = RAGGED ? key_dim : D, VD = RAGGED ? value_dim : D;
   extern __shared__ __align__(128) unsigned char dyn[];
   // The ring of the main loop ([warp][stage][K tile | V tile]) and the merge area of the tail share the
   // dynamic shared memory.
@@ -203,6 +206,7 @@ attention_decode_mma_kernel(const ProjectionInput proj,
   // (row id / CPR, chunk id % CPR) goes to row * ROW_BYTES + ((chunk ^ (row & 7)) * 16), K and V alike.
   constexpr int RPI = 32 / CPR;  // rows of a tile that one copy instruction of the warp covers
   const int row0 = lane / CPR, ch = lane % CPR;  // this lane's row within those, and its chunk of the row
+  const bool k_live = !RAGGED || ch * 8 < KD, v_live = !RAGGED || ch * 8 < VD;
   auto issue = [&](int grp, int stage) {
     const int base_key = group_base(grp);
     const int lo = grp < window_groups ? split_lo : 0, hi = grp < window_groups ? split_hi : kept - 1;
@@ -214,18 +218,17 @@ attention_decode_mma_kernel(const ProjectionInput proj,
       const int page = live ? page_of(base_key) : 0;
       const bool page_ok = live && page >= 0 && page < num_pages;
       if (live && !page_ok && error) atomicExch(error, 4);
-      const size_t at = (((size_t)(page_ok ? page : 0) * num_kv_heads + kv_head) * page_size +
-                         (base_key & (page_size - 1)) + row0) * D + ch * 8;
-      const __nv_bfloat16* k_src = k_cache + at;
-      const __nv_bfloat16* v_src = v_cache + at;
+      const size_t at = ((size_t)(page_ok ? page : 0) * num_kv_heads + kv_head) * page_size + (base_key & (page_size - 1)) + row0;
+      const __nv_bfloat16* k_src = k_cache + at * KD + ch * 8;
+      const __nv_bfloat16* v_src = v_cache + at * VD + ch * 8;
       const bool whole = page_ok && base_key >= lo && base_key + 15 <= hi;
 #pragma unroll
       for (int i = 0; i < COPIES; ++i) {
         const int row = i * RPI + row0;
         const bool ok = whole || (page_ok && base_key + row >= lo && base_key + row <= hi);
         const uint32_t offset = (uint32_t)(row * ROW_BYTES + ((ch ^ (row & 7)) << 4));
-        cp_async16(k_dst + offset, ok ? k_src + i * RPI * D : k_cache, ok ? 16 : 0);
-        cp_async16(v_dst + offset, ok ? v_src + i * RPI * D : v_cache, ok ? 16 : 0);
+        cp_async16(k_dst + offset, ok && k_live ? k_src + i * RPI * KD : k_cache, ok && k_live ? 16 : 0);
+        cp_async16(v_dst + offset, ok && v_live ? v_src + i * RPI * VD : v_cache, ok && v_live ? 16 : 0);
       }
     } else {
 #pragma unroll
@@ -241,12 +244,12 @@ attention_decode_mma_kernel(const ProjectionInput proj,
             if (error) atomicExch(error, 4);
             ok = false;
           } else {
-            at = (((size_t)page * num_kv_heads + kv_head) * page_size + within) * D + ch * 8;
+            at = ((size_t)page * num_kv_heads + kv_head) * page_size + within;
           }
         }
         const uint32_t offset = (uint32_t)(row * ROW_BYTES + ((ch ^ (row & 7)) << 4));
-        cp_async16(k_dst + offset, k_cache + at, ok ? 16 : 0);
-        cp_async16(v_dst + offset, v_cache + at, ok ? 16 : 0);
+        cp_async16(k_dst + offset, ok && k_live ? k_cache + at * KD + ch * 8 : k_cache, ok && k_live ? 16 : 0);
+        cp_async16(v_dst + offset, ok && v_live ? v_cache + at * VD + ch * 8 : v_cache, ok && v_live ? 16 : 0);
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -270,11 +273,12 @@ attention_decode_mma_kernel(const ProjectionInput proj,
 #pragma unroll
     for (int nh = 0; nh < NH; ++nh) {
       const int hd = nh * 8 + g;
-      const __nv_bfloat16* row = q + (size_t)t * q_row_stride + (size_t)(head0 + hd) * D + 2 * c;
+      const __nv_bfloat16* row = q + (size_t)t * q_row_stride + (size_t)(head0 + hd) * KD + 2 * c;
 #pragma unroll
       for (int ks = 0; ks < MT; ++ks) {
-        qb[nh][ks][0] = hd < heads_here ? __ldcg(reinterpret_cast<const unsigned int*>(row + 16 * ks)) : 0u;
-        qb[nh][ks][1] = hd < heads_here ? __ldcg(reinterpret_cast<const unsigned int*>(row + 16 * ks + 8)) : 0u;
+        const bool low = hd < heads_here && (!RAGGED || 16 * ks < KD), high = hd < heads_here && (!RAGGED || 16 * ks + 8 < KD);
+        qb[nh][ks][0] = low ? __ldcg(reinterpret_cast<const unsigned int*>(row + 16 * ks)) : 0u;
+        qb[nh][ks][1] = high ? __ldcg(reinterpret_cast<const unsigned int*>(row + 16 * ks + 8)) : 0u;
       }
     }
   } else {
@@ -511,7 +515,7 @@ attention_decode_mma_kernel(const ProjectionInput proj,
     const int head = head0 + hd;
     if (num_splits == 1) {
       const float inv = extras.sink ? sink_inverse_log2(m_all, l_all, extras.sink[head]) : (l_all > 0.f ? 1.f / l_all : 0.f);
-      out[(size_t)t * out_row_stride + (size_t)head * D + e] = __float2bfloat16_rn(acc * inv);
+      if (!RAGGED || e < VD) out[(size_t)t * out_row_stride + (size_t)head * VD + e] = __float2bfloat16_rn(acc * inv);
     } else if (cluster_merge) {
       cl_o[hd][e] = acc;
       if (e == 0) { cl_m[hd] = m_all; cl_l[hd] = l_all; }
@@ -554,7 +558,7 @@ attention_decode_mma_kernel(const ProjectionInput proj,
         acc += os[s] * weight;
       }
       const float inv = extras.sink ? sink_inverse_log2(m_all, l_all, extras.sink[head0 + hd]) : (l_all > 0.f ? 1.f / l_all : 0.f);
-      out[(size_t)t * out_row_stride + (size_t)(head0 + hd) * D + e] = __float2bfloat16_rn(acc * inv);
+      if (!RAGGED || e < VD) out[(size_t)t * out_row_stride + (size_t)(head0 + hd) * VD + e] = __float2bfloat16_rn(acc * inv);
     }
     cluster_barrier_exit();  // no CTA leaves while another may still read its shared memory
   }
@@ -563,13 +567,13 @@ attention_decode_mma_kernel(const ProjectionInput proj,
 // Combines the partial results of the splits of one (token, head): maxima are base-2 exponents.
 // A row of head_dim floats takes head_dim / 4 threads (four floats each); the block's 256 threads
 // hold 256 / (head_dim / 4) rows at a time, so that the loads of many splits are in flight together,
-// and the rows meet in shared memory.  The order of the additions is fixed by the split count alone.
+// and the rows meet in shared memory; of the result value_dim columns are stored.  The order of the additions is fixed by the split count alone.
 constexpr int kMergeThreads = 256;
 
 __global__ void __launch_bounds__(kMergeThreads)
 attention_decode_mma_merge_kernel(const float* __restrict__ scratch_o, const float* __restrict__ scratch_ml,
                                   __nv_bfloat16* __restrict__ out, int out_row_stride, int num_heads, int head_dim,
-                                  int num_splits, const float* __restrict__ sink) {
+                                  int value_dim, int num_splits, const float* __restrict__ sink) {
   __shared__ float sh_max[kMergeThreads / 32];
   __shared__ float sh_l[kMergeThreads / 16];
   __shared__ float4 sh_acc[kMergeThreads];
@@ -604,7 +608,7 @@ attention_decode_mma_merge_kernel(const float* __restrict__ scratch_o, const flo
   sh_acc[threadIdx.x] = acc;
   if (piece == 0) sh_l[mine] = l;
   __syncthreads();
-  if (threadIdx.x < per_row) {
+  if (threadIdx.x < per_row && piece * 4 < value_dim) {
     float l_all = 0.f;
     float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int r = 0; r < rows; ++r) {
@@ -617,7 +621,7 @@ attention_decode_mma_merge_kernel(const float* __restrict__ scratch_o, const flo
     uint2 packed;
     packed.x = *reinterpret_cast<uint32_t*>(&lo);
     packed.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(out + (size_t)t * out_row_stride + (size_t)head * head_dim + piece * 4) = packed;
+    *reinterpret_cast<uint2*>(out + (size_t)t * out_row_stride + (size_t)head * value_dim + piece * 4) = packed;
   }
 }
 
@@ -641,8 +645,13 @@ static int launch_decode_mma(const ProjectionInput* proj, const void* q, int q_r
                              const int* block_table, int table_width, const void* k_cache, const void* v_cache,
                              int tokens, int num_heads, int num_kv_heads, int head_dim, int page_size, int num_pages,
                              int window, int key_chunk, int keep_first, float scale, int num_splits, int* error,
-                             cudaStream_t stream, const ScoreExtras extras = ScoreExtras()) {
+                             cudaStream_t stream, const ScoreExtras extras = ScoreExtras(), int key_dim = 0, int value_dim = 0) {
   if (tokens <= 0) return 0;
+  // (key_dim 0: keys and values fill the kernel's head_dim)
+  const bool ragged = key_dim > 0 && (key_dim != head_dim || value_dim != head_dim);
+  if (key_dim <= 0) key_dim = value_dim = head_dim;
+  if (key_dim > head_dim || value_dim < 1 || value_dim > head_dim || (key_dim & 7) || (value_dim & 7) || (ragged && proj))
+    return DISTIE_ERR_ARG;
   if (keep_first < 0 || (proj && keep_first)) return DISTIE_ERR_ARG;
   if (num_heads < 1 || num_kv_heads < 1 || num_heads % num_kv_heads != 0 || page_size < 1 || table_width < 1 ||
       num_splits < 1 || num_splits > 65535 || (num_splits > kMmaDecodeClusterSplits && scratch == nullptr) || (q_row_stride & 7) ||
@@ -668,7 +677,7 @@ static int launch_decode_mma(const ProjectionInput* proj, const void* q, int q_r
         cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, device) != cudaSuccess || sm_count < 1)
       sm_count = 148;
   }
-  const int stages = distie_attention_decode_mma_stages(tokens, num_kv_heads * chunks, num_splits, sm_count);
+  const int stages = ragged ? 2 : distie_attention_decode_mma_stages(tokens, num_kv_heads * chunks, num_splits, sm_count);
   // Dynamic shared memory: the larger of the ring (warps x stages x loads x 512 bytes) and the merge areas.
   const size_t ring_bytes = (size_t)kMmaDecodeWarps * stages * 2 * 16 * head_dim * 2;  // K and V tiles of 16 rows
   const size_t merge_bytes = (size_t)kMmaDecodeWarps * 16 * (head_dim + 1) * sizeof(float) + 16 * head_dim * sizeof(float);
@@ -686,6 +695,15 @@ static int launch_decode_mma(const ProjectionInput* proj, const void* q, int q_r
       (err = cudaFuncSetAttribute(attention_decode_mma_kernel<DV, SV, NV, false, true>,                             \
                                   cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024)) != cudaSuccess)         \
     return (int)err
+#define DISTIE_MMA_DECODE_SMEM_RAGGED(DV, NV)                                                                     \
+  if ((err = cudaFuncSetAttribute(attention_decode_mma_kernel<DV, 2, NV, true, false, true>,                        \
+                                  cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024)) != cudaSuccess ||       \
+      (err = cudaFuncSetAttribute(attention_decode_mma_kernel<DV, 2, NV, false, false, true>,                       \
+                                  cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024)) != cudaSuccess)         \
+    return (int)err
+    DISTIE_MMA_DECODE_SMEM_RAGGED(64, 1); DISTIE_MMA_DECODE_SMEM_RAGGED(64, 2);
+    DISTIE_MMA_DECODE_SMEM_RAGGED(128, 1); DISTIE_MMA_DECODE_SMEM_RAGGED(128, 2);
+#undef DISTIE_MMA_DECODE_SMEM_RAGGED
     DISTIE_MMA_DECODE_SMEM(64, 2, 1); DISTIE_MMA_DECODE_SMEM(64, 3, 1); DISTIE_MMA_DECODE_SMEM(128, 2, 1); DISTIE_MMA_DECODE_SMEM(128, 3, 1);
     DISTIE_MMA_DECODE_SMEM(64, 2, 2); DISTIE_MMA_DECODE_SMEM(64, 3, 2); DISTIE_MMA_DECODE_SMEM(128, 2, 2); DISTIE_MMA_DECODE_SMEM(128, 3, 2);
 #undef DISTIE_MMA_DECODE_SMEM
@@ -701,22 +719,35 @@ static int launch_decode_mma(const ProjectionInput* proj, const void* q, int q_r
 #define DISTIE_MMA_DECODE_FUSED(DV, SV, NV, PV)                                                                    \
   if (proj) DISTIE_MMA_DECODE_PAGE(DV, SV, NV, PV, true);                                                           \
   else DISTIE_MMA_DECODE_PAGE(DV, SV, NV, PV, false)
-#define DISTIE_MMA_DECODE_PAGE(DV, SV, NV, PV, FV)                                                                 \
-  err = launch_dependent_cluster(8, cluster, attention_decode_mma_kernel<DV, SV, NV, PV, FV>, grid, dim3(kMmaDecodeWarps * 32), \
+#define DISTIE_MMA_DECODE_PAGE(DV, SV, NV, PV, FV) DISTIE_MMA_DECODE_ANY(grid, DV, SV, NV, PV, FV)
+#define DISTIE_MMA_DECODE_ANY(GRID, ...)                                                                           \
+  err = launch_dependent_cluster(8, cluster, attention_decode_mma_kernel<__VA_ARGS__>, GRID, dim3(kMmaDecodeWarps * 32), \
                          shared, stream, projection, (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, out_row_stride, \
                          scratch_o, scratch_ml, positions, token_seq, seq_seat, block_table, table_width,          \
                          (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, num_heads, group, chunks,   \
-                         num_kv_heads, page_size, page_shift, num_pages, window, key_chunk, keep_first, scale_log2, cluster_merge, extras, error)
+                         num_kv_heads, page_size, page_shift, num_pages, window, key_chunk, keep_first, scale_log2, cluster_merge, extras, key_dim, value_dim, error)
 #define DISTIE_MMA_DECODE_BY_STAGES(DV, NV)   \
   if (stages == 2) { DISTIE_MMA_DECODE(DV, 2, NV) } \
   else { DISTIE_MMA_DECODE(DV, 3, NV) }
-  if (head_dim == 64) {
+  if (ragged) {
+    const bool page16 = page_shift >= 4;
+#define DISTIE_MMA_DECODE_RAGGED(DV, NV)                                       \
+  if (page16) { DISTIE_MMA_DECODE_ANY(grid, DV, 2, NV, true, false, true); }   \
+  else { DISTIE_MMA_DECODE_ANY(grid, DV, 2, NV, false, false, true); }
+    if (head_dim == 64) {
+      if (column_tiles == 1) { DISTIE_MMA_DECODE_RAGGED(64, 1) } else { DISTIE_MMA_DECODE_RAGGED(64, 2) }
+    } else {
+      if (column_tiles == 1) { DISTIE_MMA_DECODE_RAGGED(128, 1) } else { DISTIE_MMA_DECODE_RAGGED(128, 2) }
+    }
+#undef DISTIE_MMA_DECODE_RAGGED
+  } else if (head_dim == 64) {
     if (column_tiles == 1) { DISTIE_MMA_DECODE_BY_STAGES(64, 1); } else { DISTIE_MMA_DECODE_BY_STAGES(64, 2); }
   } else {
     if (column_tiles == 1) { DISTIE_MMA_DECODE_BY_STAGES(128, 1); } else { DISTIE_MMA_DECODE_BY_STAGES(128, 2); }
   }
 #undef DISTIE_MMA_DECODE_BY_STAGES
 #undef DISTIE_MMA_DECODE_PAGE
+#undef DISTIE_MMA_DECODE_ANY
 #undef DISTIE_MMA_DECODE_FUSED
 #undef DISTIE_MMA_DECODE
   if (err != cudaSuccess) return (int)err;
@@ -724,7 +755,7 @@ static int launch_decode_mma(const ProjectionInput* proj, const void* q, int q_r
     const dim3 merge_grid(tokens, num_heads);
     err = launch_dependent_family(8, attention_decode_mma_merge_kernel, merge_grid, dim3(kMergeThreads), 0, stream,
                            (const float*)scratch_o, (const float*)scratch_ml, (__nv_bfloat16*)out, out_row_stride,
-                           num_heads, head_dim, num_splits, extras.sink);
+                           num_heads, head_dim, value_dim, num_splits, extras.sink);
     if (err != cudaSuccess) return (int)err;
   }
   return 0;
@@ -768,6 +799,23 @@ extern "C" int distie_attention_decode_mma_capped(const void* q, int q_row_strid
                            block_table, table_width, k_cache, v_cache, tokens, num_heads, num_kv_heads, head_dim,
                            page_size, num_pages, window, key_chunk, keep_first, scale, num_splits, error, stream,
                            make_score_extras(scale, softcap, sink));
+}
+
+// The same for heads that do not fill a tile: keys of key_dim and values of value_dim elements (multiples of 8, at most
+// head_dim, which is 64 or 128 and the width of the partial results in `scratch`).
+extern "C" int distie_attention_decode_mma_ragged(const void* q, int q_row_stride, void* out, int out_row_stride,
+                                                  float* scratch, const int* positions, const int* token_seq,
+                                                  const int* seq_seat, const int* block_table, int table_width,
+                                                  const void* k_cache, const void* v_cache, int tokens, int num_heads,
+                                                  int num_kv_heads, int head_dim, int page_size, int num_pages, int window,
+                                                  int key_chunk, int keep_first, float scale, float softcap,
+                                                  const float* sink, int key_dim, int value_dim, int num_splits, int* error,
+                                                  cudaStream_t stream) {
+  if (key_dim < 1) return DISTIE_ERR_ARG;
+  return launch_decode_mma(nullptr, q, q_row_stride, out, out_row_stride, scratch, positions, token_seq, seq_seat,
+                           block_table, table_width, k_cache, v_cache, tokens, num_heads, num_kv_heads, head_dim,
+                           page_size, num_pages, window, key_chunk, keep_first, scale, num_splits, error, stream,
+                           make_score_extras(scale, softcap, sink), key_dim, value_dim);
 }
 
 // The same for a step of single tokens that starts from the q/k/v projection: `slices` [splits, tokens, row_stride]

@@ -43,7 +43,11 @@
 //
 // Every wait on an mbarrier is bounded; when one runs out the CTA sets the error word to 6, every role
 // stops at its next wait, the producers wait (bounded) for their copies in flight, and tensor memory is
-// released.  head_dim 64 or 128; page sizes 8, 16, ..., 128.
+// released.  Page sizes 8, 16, ..., 128.
+//
+// Sizes: keys of up to DK = 64 or 128 elements and values of up to DV = 64 or 128, multiples of 8 and of one another
+// independent.  A head smaller than its tile is padded on the way in: the copies fill what lies past the end of a key's
+// or value's row with zeros.  (The columns of Q past the head's end hold the next head's: they meet the zeros of K.)
 #include "tcgen05.cuh"
 
 namespace distie {
@@ -58,11 +62,11 @@ constexpr int kAttnKStages = 2, kAttnVStages = 3;  // V of a block is needed a b
 constexpr int kAttnHalf = kAttnRows * 128;  // bytes of one [128 rows x 64 elements] swizzled half tile
 constexpr float kAttnRaise = 8.f;  // the maximum in use is raised when a row exceeds it by this much (base 2)
 
-template <int D>
+template <int DK, int DV>
 struct AttnShared {
-  alignas(1024) unsigned char q[kAttnRows * D * 2];
-  alignas(1024) unsigned char k[kAttnKStages][kAttnKeys * D * 2];
-  alignas(1024) unsigned char v[kAttnVStages][kAttnKeys * D * 2];
+  alignas(1024) unsigned char q[kAttnRows * (DK > DV ? DK : DV) * 2];  // at the end: the output tile
+  alignas(1024) unsigned char k[kAttnKStages][kAttnKeys * DK * 2];
+  alignas(1024) unsigned char v[kAttnVStages][kAttnKeys * DV * 2];
   uint64_t q_full;
   uint64_t k_full[kAttnKStages], k_empty[kAttnKStages];
   uint64_t v_full[kAttnVStages], v_empty[kAttnVStages];
@@ -108,7 +112,7 @@ __device__ __forceinline__ uint64_t add_pairs(uint64_t a, uint64_t b) {
   return d;
 }
 
-template <int D>
+template <int DK, int DV>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                  const __grid_constant__ CUtensorMap map_v,
@@ -116,15 +120,15 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                  int out_row_stride, const int* __restrict__ q_tiles,
                                  const int* __restrict__ positions, const int* __restrict__ token_seq,
                                  const int* __restrict__ seq_seat, const int* __restrict__ block_table,
-                                 int table_width, int group_size, int num_kv_heads, int page_shift, int num_pages,
-                                 int window, int key_chunk, int keep_first, float scale_log2, float cap, float cap_pre,
+                                 int table_width, int group_size, int num_kv_heads, int key_dim, int value_dim,
+                                 int page_shift, int num_pages, int window, int key_chunk, int keep_first, float scale_log2, float cap, float cap_pre,
                                  const float* __restrict__ sink_logits, int* __restrict__ error) {
   // cap > 0: a raw score s becomes tanh(s * cap_pre) (cap_pre = scale / cap) and scale_log2 is cap * log2(e): the
   // cap's own factor rides the multiplication by scale_log2 that every score goes through anyway.
   // sink_logits: one float per head whose exponential joins the row's sum at the end (null: none).
   extern __shared__ unsigned char raw[];
-  auto& sm = *reinterpret_cast<AttnShared<D>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
-  constexpr int HALVES = D / 64;
+  auto& sm = *reinterpret_cast<AttnShared<DK, DV>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
+  constexpr int K_HALVES = DK / 64, V_HALVES = DV / 64;
   constexpr uint32_t TMEM_COLS = 512;
   constexpr uint32_t O_COL = 256;  // S0 | S1 | O of group 0 | O of group 1
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -214,10 +218,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     // ---- producers: warp 0 fetches Q and K, the last warp V; lane pg takes page pg of a block -----------------
     const bool for_k = warp == 0;
     if (for_k && lane == 0) {
-      mbar_expect_tx(&sm.q_full, kAttnRows * D * 2);
-      for (int h = 0; h < HALVES; ++h) tma_load_2d(sm.q + h * kAttnHalf, &map_q, &sm.q_full, head * D + h * 64, t0);
+      mbar_expect_tx(&sm.q_full, kAttnRows * DK * 2);
+      for (int h = 0; h < K_HALVES; ++h) tma_load_2d(sm.q + h * kAttnHalf, &map_q, &sm.q_full, head * key_dim + h * 64, t0);
     }
-    const int stages = for_k ? kAttnKStages : kAttnVStages;
+    const int stages = for_k ? kAttnKStages : kAttnVStages, halves = for_k ? K_HALVES : V_HALVES;
     const CUtensorMap* map = for_k ? &map_k : &map_v;
     uint64_t* full = for_k ? sm.k_full : sm.v_full;
     uint64_t* empty = for_k ? sm.k_empty : sm.v_empty;
@@ -235,12 +239,12 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         break;
       }
       if (!__all_sync(0xffffffffu, mbar_wait_unless(&empty[s], (use & 1) ^ 1, failed))) { ok = false; break; }
-      if (lane == 0) mbar_expect_tx(&full[s], (uint32_t)count * page_size * D * 2);
+      if (lane == 0) mbar_expect_tx(&full[s], (uint32_t)(count * page_size * halves * 128));
       __syncwarp();
       if (mine) {
         unsigned char* stage = (for_k ? sm.k[s] : sm.v[s]) + lane * page_size * 128;
         const int row = (page * num_kv_heads + kv_head) * page_size;
-        for (int h = 0; h < HALVES; ++h) tma_load_2d(stage + h * kAttnHalf, map, &full[s], h * 64, row);
+        for (int h = 0; h < halves; ++h) tma_load_2d(stage + h * kAttnHalf, map, &full[s], h * 64, row);
       }
       issued = j + 1;
     }
@@ -254,7 +258,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     // ---- MMA issuer ------------------------------------------------------------------------------------------
     if (lane == 0) {
       constexpr uint32_t idesc_s = instr_desc(kAttnKeys);
-      constexpr uint32_t idesc_o = instr_desc(D, true);
+      constexpr uint32_t idesc_o = instr_desc(DV, true);
       const uint64_t q_desc = smem_desc(sm.q);
       bool ok = mbar_wait_unless(&sm.q_full, 0, failed);
       // S of block j into buffer j & 1.  Both groups have that buffer's last S in registers and their P
@@ -265,7 +269,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const uint64_t k_desc = smem_desc(sm.k[ks]);
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
           const uint64_t step = (uint64_t)(((kk >> 2) * kAttnHalf + (kk & 3) * 32) >> 4);
           umma_bf16(tmem + s * kAttnKeys, q_desc + step, k_desc + step, idesc_s, kk > 0 ? 1u : 0u);
         }
@@ -288,7 +292,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             // P of the group: 32 columns at the start of its half of the S buffer, 16 keys are 8 columns;
             // its keys are rows g * 64 ... of the V block.
             const uint64_t v_step = (uint64_t)(((g * kAttnGroupKeys + kk * 16) * 128) >> 4);
-            umma_bf16_ts(tmem + O_COL + g * D, tmem + s * kAttnKeys + g * kAttnGroupKeys + kk * 8, v_desc + v_step,
+            umma_bf16_ts(tmem + O_COL + g * DV, tmem + s * kAttnKeys + g * kAttnGroupKeys + kk * 8, v_desc + v_step,
                          idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
           }
           umma_commit(&sm.pv_done[g]);
@@ -305,7 +309,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     const int g = (warp - 2) >> 2;
     const int r = quadrant * 32 + lane;
     const uint32_t lane_base = tmem + ((uint32_t)(quadrant * 32) << 16);
-    const uint32_t o_addr = lane_base + O_COL + g * D;
+    const uint32_t o_addr = lane_base + O_COL + g * DV;
     const int limit = min(pos0 + r, last_pos);                      // newest key this row may see
     const int oldest = first_visible_key(limit, window, key_chunk);  // oldest key inside its window or chunk
     float m_used = -INFINITY, l = 0.f;
@@ -367,7 +371,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         if (!wait_all(&sm.pv_done[g], (j - 1) & 1)) { ok = false; break; }
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-        for (int c0 = 0; c0 < D; c0 += 32) {
+        for (int c0 = 0; c0 < DV; c0 += 32) {
           uint32_t v[32];
           tmem_load_32(o_addr + c0, v);
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -408,7 +412,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         const int row = g * kAttnGroupKeys + (r & (kAttnGroupKeys - 1));
         if (r < kAttnGroupKeys && !needed(j, row >> page_shift)) {
 #pragma unroll
-          for (int h = 0; h < HALVES; ++h) {
+          for (int h = 0; h < V_HALVES; ++h) {
             uint4* dst = reinterpret_cast<uint4*>(sm.v[vs] + h * kAttnHalf + row * 128);
 #pragma unroll
             for (int i = 0; i < 8; ++i) dst[i] = make_uint4(0u, 0u, 0u, 0u);
@@ -448,14 +452,15 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
       // leaves as one: 128 rows of whole lines, where the threads' own stores are 16 bytes of 32 different
       // rows per instruction and take a microsecond and a half to drain.  A partial tile (the end of a
       // request) is stored by the threads, row by row.
-      constexpr int SIDE_DIMS = D / 2;
-      const bool whole = rows == kAttnRows;  // (the same for every thread of the CTA)
-      __nv_bfloat16* dst = out + (size_t)(t0 + r) * out_row_stride + (size_t)head * D + g * SIDE_DIMS;
+      // So is a tile of heads that do not fill it: a copy would reach into the next head's columns.
+      constexpr int SIDE_DIMS = DV / 2;
+      const bool whole = rows == kAttnRows && value_dim == DV;  // (the same for every thread of the CTA)
+      __nv_bfloat16* dst = out + (size_t)(t0 + r) * out_row_stride + (size_t)head * value_dim + g * SIDE_DIMS;
 #pragma unroll
       for (int c0 = 0; c0 < SIDE_DIMS; c0 += 32) {
         uint32_t a[32], b[32];
         tmem_load_32(lane_base + O_COL + g * SIDE_DIMS + c0, a);
-        tmem_load_32(lane_base + O_COL + D + g * SIDE_DIMS + c0, b);
+        tmem_load_32(lane_base + O_COL + DV + g * SIDE_DIMS + c0, b);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (whole || r < rows) {
 #pragma unroll
@@ -473,7 +478,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 w[e] = *reinterpret_cast<const uint32_t*>(&pair);
               }
               asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(at), "r"(w[0]), "r"(w[1]), "r"(w[2]), "r"(w[3]) : "memory");
-            } else {
+            } else if (g * SIDE_DIMS + c0 + i < value_dim) {
               store8(dst + c0 + i, y);
             }
           }
@@ -485,9 +490,9 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         if (lane == 0) mbar_arrive(&sm.store_ready);
         if (warp == 2 && wait_all(&sm.store_ready, 0) && lane == 0) {
 #pragma unroll
-          for (int h = 0; h < HALVES; ++h)
+          for (int h = 0; h < V_HALVES; ++h)
             asm volatile("cp.async.bulk.tensor.2d.global.shared::cta.bulk_group [%0, {%1, %2}], [%3];" ::"l"(&map_out),
-                         "r"(head * D + h * 64), "r"(t0), "r"(smem_u32(sm.q + h * kAttnHalf)) : "memory");
+                         "r"(head * DV + h * 64), "r"(t0), "r"(smem_u32(sm.q + h * kAttnHalf)) : "memory");
           asm volatile("cp.async.bulk.commit_group;" ::: "memory");
           asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");  // shared memory is read before the CTA may end
         }
@@ -505,25 +510,25 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
   if (threadIdx.x == 0 && sm.failed && error) atomicCAS(error, 0, 6);
 }
 
-template <int D>
+template <int DK, int DV>
 static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v,
                                const CUtensorMap& map_out, void* out,
                                int out_row_stride, const int* q_tiles, int num_tiles, const int* positions,
                                const int* token_seq, const int* seq_seat, const int* block_table, int table_width,
-                               int num_heads, int num_kv_heads, int page_shift, int num_pages, int window, int key_chunk, int keep_first,
-                               float scale_log2, float cap, float cap_pre, const float* sink, int* error, cudaStream_t stream) {
-  const size_t shared = sizeof(AttnShared<D>) + 1024;
+                               int num_heads, int num_kv_heads, int key_dim, int value_dim, int page_shift, int num_pages,
+                               int window, int key_chunk, int keep_first, float scale_log2, float cap, float cap_pre, const float* sink, int* error, cudaStream_t stream) {
+  const size_t shared = sizeof(AttnShared<DK, DV>) + 1024;
   static bool configured = false;
   if (!configured) {
-    const cudaError_t err = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel<D>,
+    const cudaError_t err = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel<DK, DV>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     if (err != cudaSuccess) return (int)err;
     configured = true;
   }
   const cudaError_t err = launch_dependent_family(
-      32, attention_prefill_tcgen05_kernel<D>, dim3(num_heads, num_tiles), dim3(kAttnThreads), shared, stream, map_q,
+      32, attention_prefill_tcgen05_kernel<DK, DV>, dim3(num_heads, num_tiles), dim3(kAttnThreads), shared, stream, map_q,
       map_k, map_v, map_out, (__nv_bfloat16*)out, out_row_stride, q_tiles, positions, token_seq, seq_seat, block_table,
-      table_width, num_heads / num_kv_heads, num_kv_heads, page_shift, num_pages, window, key_chunk, keep_first, scale_log2,
+      table_width, num_heads / num_kv_heads, num_kv_heads, key_dim, value_dim, page_shift, num_pages, window, key_chunk, keep_first, scale_log2,
       cap, cap_pre, sink, error);
   return err == cudaSuccess ? 0 : (int)err;
 }
@@ -534,20 +539,20 @@ using namespace distie;
 
 // Tokens per tile of `q_tiles` ([num_tiles, 2] int32: first token of the tile, number of rows <= 128).
 // q is [tokens, >= num_heads * head_dim] bfloat16 with row stride q_row_stride; the caches are
-// [num_pages, num_kv_heads, page_size, head_dim].  Returns DISTIE_ERR_UNSUPPORTED for a head_dim other
-// than 64 and 128 or a page size that is not 8, 16, ..., 128.
+// [num_pages, num_kv_heads, page_size, head_dim] (values: value_dim).  Returns DISTIE_ERR_UNSUPPORTED for a head_dim or
+// value_dim above 128 or no multiple of 8, or a page size that is not 8, 16, ..., 128.
 extern "C" int distie_attention_prefill_tcgen05(const void* q, int q_row_stride, void* out, int out_row_stride,
                                                 const int* q_tiles, int num_tiles, const int* positions,
                                                 const int* token_seq, const int* seq_seat, const int* block_table,
                                                 int table_width, const void* k_cache, const void* v_cache, int tokens,
-                                                int num_heads, int num_kv_heads, int head_dim, int page_size,
+                                                int num_heads, int num_kv_heads, int head_dim, int value_dim, int page_size,
                                                 int num_pages, int window, int key_chunk, int keep_first, float scale,
                                                 float softcap, const float* sink, int* error, cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
   if (tokens < 1 || num_heads < 1 || num_kv_heads < 1 || num_heads % num_kv_heads != 0 || table_width < 1 ||
       num_pages < 1 || num_tiles > 65535 || keep_first < 0)
     return DISTIE_ERR_ARG;
-  if ((head_dim != 64 && head_dim != 128) || page_size < 8 || page_size > 128 || (page_size & (page_size - 1)) ||
+  if (head_dim < 8 || head_dim > 128 || (head_dim & 7) || value_dim < 8 || value_dim > 128 || (value_dim & 7) || page_size < 8 || page_size > 128 || (page_size & (page_size - 1)) ||
       (q_row_stride & 7) || (out_row_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
       ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15))
     return DISTIE_ERR_UNSUPPORTED;
@@ -556,18 +561,23 @@ extern "C" int distie_attention_prefill_tcgen05(const void* q, int q_row_stride,
   CUtensorMap map_q, map_k, map_v, map_out;
   int status = make_map(&map_q, q, tokens, num_heads * head_dim, q_row_stride, kAttnRows);
   if (status != 0) return status;
-  if ((status = make_map(&map_out, out, tokens, num_heads * head_dim, out_row_stride, kAttnRows)) != 0) return status;
+  if ((status = make_map(&map_out, out, tokens, num_heads * value_dim, out_row_stride, kAttnRows)) != 0) return status;
   const long long cache_rows = (long long)num_pages * num_kv_heads * page_size;
   if (cache_rows > 0x7fffffffLL) return DISTIE_ERR_UNSUPPORTED;
   if ((status = make_map(&map_k, k_cache, (int)cache_rows, head_dim, head_dim, page_size)) != 0) return status;
-  if ((status = make_map(&map_v, v_cache, (int)cache_rows, head_dim, head_dim, page_size)) != 0) return status;
+  if ((status = make_map(&map_v, v_cache, (int)cache_rows, value_dim, value_dim, page_size)) != 0) return status;
   const float cap = softcap > 0.f ? softcap : 0.f, cap_pre = cap > 0.f ? scale / cap : 0.f;
   const float scale_log2 = (cap > 0.f ? cap : scale) * 1.4426950408889634f;
-  if (head_dim == 64)
-    return launch_attention_tc<64>(map_q, map_k, map_v, map_out, out, out_row_stride, q_tiles, num_tiles, positions, token_seq,
-                                   seq_seat, block_table, table_width, num_heads, num_kv_heads, page_shift, num_pages,
-                                   window, key_chunk, keep_first, scale_log2, cap, cap_pre, sink, error, stream);
-  return launch_attention_tc<128>(map_q, map_k, map_v, map_out, out, out_row_stride, q_tiles, num_tiles, positions, token_seq,
-                                  seq_seat, block_table, table_width, num_heads, num_kv_heads, page_shift, num_pages,
-                                  window, key_chunk, keep_first, scale_log2, cap, cap_pre, sink, error, stream);
+#define DISTIE_ATTENTION_TC(DKV, DVV)                                                                                          \
+  return launch_attention_tc<DKV, DVV>(map_q, map_k, map_v, map_out, out, out_row_stride, q_tiles, num_tiles, positions, token_seq, \
+                                       seq_seat, block_table, table_width, num_heads, num_kv_heads, head_dim, value_dim,         \
+                                       page_shift, num_pages, window, key_chunk, keep_first, scale_log2, cap, cap_pre, sink,     \
+                                       error, stream)
+  if (head_dim <= 64) {
+    if (value_dim <= 64) DISTIE_ATTENTION_TC(64, 64);
+    DISTIE_ATTENTION_TC(64, 128);
+  }
+  if (value_dim <= 64) DISTIE_ATTENTION_TC(128, 64);
+  DISTIE_ATTENTION_TC(128, 128);
+#undef DISTIE_ATTENTION_TC
 }

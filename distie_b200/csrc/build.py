@@ -46,7 +46,7 @@ CUDA_UNITS: dict[str, list[str]] = {
     # bfloat16 serving only: tensor-core attention for prompts, weight-streaming products for decoding
     "bf16": ["attention_prefill.cu", "attention_decode_mma.cu", "gemm_tcgen05.cu", "attention_prefill_tcgen05.cu"],
     # models with layer norms, gated heads, short convolutions or linear recurrences (both dtypes)
-    "state": ["recurrent.cu"],
+    "state": ["recurrent.cu", "retention.cu"],
     # models with recurrences whose decay varies by channel (both dtypes); a unit of its own because it takes minutes
     "channel": ["channelwise.cu"],
     # models whose feed-forward routes tokens to experts (both dtypes)

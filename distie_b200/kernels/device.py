@@ -26,6 +26,7 @@ from .library import KernelError, check, function
 _CODE = {torch.float32: 0, torch.bfloat16: 1}
 _DECODE_HEAD_DIMS = (16, 32, 64, 128, 256)
 _PREFILL_HEAD_DIMS = (64, 128)  # tensor-core attention for portions of prompts (bfloat16)
+_RAGGED_FROM = 32               # heads (keys or values) from this size on are padded to a tensor-core tile
 _SKINNY_ROWS = 64               # weight-streaming products (tcgen05, weights as the 128-row operand) take up to 64 rows
 _CLUSTER_SPLITS = 8             # splits of a decode attention that one cluster of CTAs merges itself
 _TENSOR_CORE_ROWS = 128         # from here on the tcgen05 kernel's 128-row tiles are full; in between: the library
@@ -400,27 +401,39 @@ class DeviceKernels(KernelSet):
             raise KernelError("attention: the sink is one float32 per head")
         extras = softcap > 0.0 or sink is not None
         value_dim = kv.v.shape[-1]
-        same = value_dim == head_dim  # every kernel but the size-agnostic one wants values as large as keys
-        n_dec = step.num_decode_tokens if head_dim in _DECODE_HEAD_DIMS and same else 0
+        same = value_dim == head_dim
+        # Heads that fill no tile of the tensor-core kernels (and have no kernel of their own size) are padded on the
+        # way in; values may then have another size than keys.
+        ragged = (self.dtype == torch.bfloat16 and not (same and head_dim in _DECODE_HEAD_DIMS) and head_dim % 8 == 0
+                  and value_dim % 8 == 0 and _RAGGED_FROM <= max(head_dim, value_dim) <= max(_PREFILL_HEAD_DIMS)
+                  and qkv.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and kv.k.is_contiguous() and kv.v.is_contiguous())
+        tile_dim = (64 if max(head_dim, value_dim) <= 64 else 128) if ragged else head_dim
+        n_dec = step.num_decode_tokens if ragged or (head_dim in _DECODE_HEAD_DIMS and same) else 0
         element = qkv.element_size()
         if n_dec > 0:
             splits = self.plan_splits(n_dec, num_heads, num_kv_heads, step.max_kv_len)
-            tensor_cores = self.dtype == torch.bfloat16 and head_dim in _PREFILL_HEAD_DIMS
+            tensor_cores = self.dtype == torch.bfloat16 and tile_dim in _PREFILL_HEAD_DIMS
             if tensor_cores and splits <= 2 * _CLUSTER_SPLITS:
                 splits = min(splits, _CLUSTER_SPLITS)  # merged inside the kernel, by a cluster of CTAs
             in_kernel_merge = splits == 1 or (tensor_cores and splits <= _CLUSTER_SPLITS)
             scratch = None
             if not in_kernel_merge:
-                floats = function("distie_attention_decode_scratch_floats")(n_dec, num_heads, head_dim, splits)
+                floats = function("distie_attention_decode_scratch_floats")(n_dec, num_heads, tile_dim, splits)
                 scratch = torch.empty(floats, dtype=torch.float32, device=qkv.device)
             head = [
                 qkv.data_ptr(), qkv.stride(0), out.data_ptr(), out.stride(0),
                 scratch.data_ptr() if scratch is not None else None, step.positions.data_ptr(),
                 step.token_seq.data_ptr(), step.seq_seat.data_ptr(), kv.block_table.data_ptr(),
                 kv.block_table.shape[-1], kv.k.data_ptr(), kv.v.data_ptr(), n_dec, num_heads, num_kv_heads,
-                head_dim, kv.page_size, kv.num_pages, window, chunk,
+                tile_dim, kv.page_size, kv.num_pages, window, chunk,
             ]
-            if tensor_cores and extras:
+            if ragged:
+                check(
+                    function("distie_attention_decode_mma_ragged")(*head, keep_first, float(scale), softcap, sink_ptr, head_dim,
+                                                                   value_dim, splits, self.error_flag.data_ptr(), self._stream()),
+                    "attention_decode_mma",
+                )
+            elif tensor_cores and extras:
                 check(
                     function("distie_attention_decode_mma_capped")(*head, keep_first, float(scale), softcap, sink_ptr, splits,
                                                                    self.error_flag.data_ptr(), self._stream()),
@@ -440,12 +453,12 @@ class DeviceKernels(KernelSet):
                 )
             self._ran("attention_decode_mma" if tensor_cores else "attention_decode", 1 if in_kernel_merge else 2)
         rest = step.num_tokens - n_dec
-        tiled = (rest > 0 and self.dtype == torch.bfloat16 and head_dim in _PREFILL_HEAD_DIMS and step.num_q_tiles
-                 and n_dec == step.num_decode_tokens and same)
+        tiled = (rest > 0 and self.dtype == torch.bfloat16 and tile_dim in _PREFILL_HEAD_DIMS and step.num_q_tiles
+                 and n_dec == step.num_decode_tokens)
         if tiled and self._attention_tcgen05(qkv, out, step, kv, num_heads, num_kv_heads, head_dim, window, chunk, scale,
                                              keep_first, softcap, sink_ptr):
             pass
-        elif tiled:
+        elif tiled and not ragged:
             check(
                 function("distie_attention_prefill")(
                     qkv.data_ptr(), qkv.stride(0), out.data_ptr(), out.stride(0), step.q_tiles.data_ptr(),
@@ -479,7 +492,7 @@ class DeviceKernels(KernelSet):
             qkv.data_ptr(), qkv.stride(0), out.data_ptr(), out.stride(0), step.q_tiles.data_ptr(), step.num_q_tiles,
             step.positions.data_ptr(), step.token_seq.data_ptr(), step.seq_seat.data_ptr(),
             kv.block_table.data_ptr(), kv.block_table.shape[-1], kv.k.data_ptr(), kv.v.data_ptr(), qkv.shape[0],
-            num_heads, num_kv_heads, head_dim, kv.page_size, kv.num_pages, window, chunk, keep_first, float(scale),
+            num_heads, num_kv_heads, head_dim, kv.v.shape[-1], kv.page_size, kv.num_pages, window, chunk, keep_first, float(scale),
             float(softcap), sink_ptr, self.error_flag.data_ptr(), self._stream(),
         )
         if code == -2:
@@ -664,6 +677,64 @@ class DeviceKernels(KernelSet):
         )
         self._ran("rotate_heads")
         return out
+
+    def _trig(self, step, rotary):
+        """``[T, rotary_dim]`` float32: cosines, then sines, of every token's angles; made once per step and encoding."""
+        if rotary is None or not rotary.rotary_dim:
+            return None
+        key = ("trig", rotary.inv_freq.data_ptr(), rotary.rotary_dim, float(rotary.factor))
+        made = step.derived.get(key)
+        if made is None:
+            made = torch.empty((step.num_tokens, rotary.rotary_dim), dtype=torch.float32, device=self.device)
+            check(
+                function("distie_rope_rows")(
+                    step.positions.data_ptr(), step.token_seq.data_ptr(), step.seq_seat.data_ptr(), None, 1,
+                    rotary.inv_freq.data_ptr(), float(rotary.factor), step.num_tokens, rotary.rotary_dim, 1, 1, 1,
+                    made.data_ptr(), None, self.error_flag.data_ptr(), self._stream(),
+                ),
+                "rope_rows",
+            )
+            self._ran("rope_rows")
+            step.derived[key] = made
+        return made
+
+    def retention(self, qkv, gate, rotary, key_scale, decay, state, step, heads, key_dim, value_dim, weight, eps, activation, out) -> None:
+        """Heads that are normed by themselves: single tokens in one kernel; portions of prompts in chunks on the tensor
+        cores (16-bit engine).  Everything else: the ops after one another."""
+        singles, tokens = step.num_decode_tokens, step.num_tokens
+        portions = tokens > singles
+        chunked = self.dtype == torch.bfloat16 and key_dim <= 128 and value_dim <= 128 and step.num_q_tiles > 0
+        if weight is not None or key_dim > 256 or value_dim > 4096 or (portions and not chunked) or not state.is_contiguous():
+            super().retention(qkv, gate, rotary, key_scale, decay, state, step, heads, key_dim, value_dim, weight, eps, activation, out)
+            return
+        rows, gates = self._sliced(qkv, "retention"), self._sliced(gate, "retention gate")
+        turned = rotary.rotary_dim if rotary is not None else 0
+        interleaved = int(rotary.interleaved) if rotary is not None else 0
+        sigmoid = int(activation == "sigmoid")
+        tail = (heads, key_dim, value_dim, sigmoid, float(eps), out.data_ptr(), out.stride(0), _CODE[out.dtype], self._stream())
+        if portions:
+            trig = self._trig(step, rotary)
+            floats = function("distie_retention_scratch_floats")(step.num_q_tiles, heads, key_dim, value_dim)
+            chunks = torch.empty(floats, dtype=torch.float32, device=qkv.device)
+            check(
+                function("distie_retention_chunks")(
+                    *rows, *gates, trig.data_ptr() if trig is not None else None, turned, interleaved, float(key_scale),
+                    decay.data_ptr(), state.data_ptr(), chunks.data_ptr(), step.q_tiles.data_ptr(), step.num_q_tiles,
+                    step.token_seq.data_ptr(), step.seq_seat.data_ptr(), *tail,
+                ),
+                "retention_chunks",
+            )
+            self._ran("retention_chunks", 3)
+        if singles:
+            check(
+                function("distie_retention_single")(
+                    *rows, *gates, step.positions.data_ptr(), rotary.inv_freq.data_ptr() if turned else None,
+                    float(rotary.factor) if rotary is not None else 1.0, turned, interleaved, float(key_scale),
+                    decay.data_ptr(), state.data_ptr(), step.token_seq.data_ptr(), step.seq_seat.data_ptr(), singles, *tail,
+                ),
+                "retention_single",
+            )
+            self._ran("retention_single")
 
     # -- recurrences whose decay varies by channel ------------------------------------------------------------------
     def selective_scan(self, x, dt, B, C, gate, rates, skip, dt_bias, state, step, out) -> None:

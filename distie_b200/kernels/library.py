@@ -47,7 +47,10 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     "distie_attention_prefill": ("bf16", [P, I, P, I, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, F, P, P, P]),
     "distie_attention_prefill_tile": ("bf16", []),
     "distie_attention_prefill_tcgen05": (
-        "bf16", [P, I, P, I, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, F, F, P, P, P]
+        "bf16", [P, I, P, I, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, F, P, P, P]
+    ),
+    "distie_attention_decode_mma_ragged": (
+        "bf16", [P, I, P, I, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, F, F, P, I, I, I, P, P]
     ),
     "distie_attention_decode_mma_stages": ("bf16", [I, I, I, I]),
     "distie_attention_decode_mma": ("bf16", [P, I, P, I, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, I, P, P]),
@@ -67,6 +70,13 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
         "state", [I, P, I, P, I, P, I, P, I, P, I, I, L, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, P]
     ),
     "distie_activation": ("state", [P, I, I, L, P, I, I, I, F, I, I, P]),
+    "distie_retention_scratch_floats": ("state", [I, I, I, I]),
+    "distie_retention_chunks": (
+        "state", [P, I, I, L, P, I, I, L, P, I, I, F, P, P, P, P, I, P, P, I, I, I, I, F, P, I, I, P]
+    ),
+    "distie_retention_single": (
+        "state", [P, I, I, L, P, I, I, L, P, P, F, I, I, F, P, P, P, P, I, I, I, I, I, F, P, I, I, P]
+    ),
     "distie_rotate_heads": ("state", [P, I, I, L, P, I, P, P, F, I, I, I, I, I, F, I, P]),
     "distie_selective_scan": (
         "channel", [P, I, P, I, I, L, P, P, I, I, L, P, I, I, L, P, P, P, P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, P]
@@ -107,7 +117,7 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     "distie_gemm_tcgen05_skinny_act": ("bf16", [P, I, P, P, I, I, I, I, I, F, F, I, P, P]),
     "distie_gemm_tcgen05_skinny": ("bf16", [P, I, P, P, P, I, I, I, I, I, I, I, P, P]),
 }
-_RESULT = {"distie_attention_decode_scratch_floats": c_longlong, "distie_route_plan_words": c_longlong,
+_RESULT = {"distie_retention_scratch_floats": c_longlong, "distie_attention_decode_scratch_floats": c_longlong, "distie_route_plan_words": c_longlong,
            "distie_latent_attention_scratch_floats": c_longlong, "distie_selective_scan_scratch_floats": c_longlong,
            "distie_channel_delta_scratch_floats": c_longlong}
 

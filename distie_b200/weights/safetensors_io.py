@@ -178,7 +178,7 @@ def save_file(tensors: Mapping[str, torch.Tensor], path: str, metadata: Mapping[
         handle.write(struct.pack("<Q", len(blob)))
         handle.write(blob)
         for name in order:
-            tensor = tensors[name].detach().contiguous().cpu()
+            tensor = tensors[name].detach().contiguous().cpu().reshape(-1)
             if tensor.numel() == 0:
                 continue
             raw = tensor.view(torch.uint8) if tensor.dtype != torch.bool else tensor.to(torch.uint8)

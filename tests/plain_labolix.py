@@ -256,9 +256,10 @@ def tensor_shapes(cfg):
     return shapes
 
 
-def random_weights(cfg, seed, gain=1.5):
+def random_weights(cfg, seed, gain=1.2):
     """Weights rounded to bfloat16 (as checkpoints store them), sized so that activations stay of order one, the norms
-    bend, a feed-forward's limits are met and sinks take a share."""
+    bend, a feed-forward's limits are met and sinks take a share.  A retention layer's keys lean towards its queries: a
+    read-out that is almost nothing would be blown up to full size by its norm, rounding and all."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in tensor_shapes(cfg).items():
@@ -273,6 +274,9 @@ def random_weights(cfg, seed, gain=1.5):
             t = torch.randn(shape, generator=g) * 1.5
         elif len(shape) == 2:
             t = torch.randn(shape, generator=g) * gain / math.sqrt(shape[1])
+            layer = cfg["layers"][int(name.split(".", 1)[0][1:])] if name.startswith("l") else None
+            if layer is not None and layer["type"] == "retention" and name.endswith("mix.k"):
+                t = 0.8 * out[name[:-1] + "q"] + 0.6 * t
         else:
             t = 1.0 + torch.randn(shape, generator=g) * 0.3
         out[name] = t.to(torch.bfloat16).float()

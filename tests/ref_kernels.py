@@ -274,6 +274,8 @@ def norm_add_rmsnorm(delta, delta_weight, delta_eps, residual, weight, eps, dtyp
         d = d * torch.rsqrt((d * d).mean(-1, keepdim=True) + delta_eps) * delta_weight.float()
     summed = residual if d is None else residual + d
     source = summed if rows_index is None else summed[rows_index.long()]
+    if weight is None:  # only the residual is moved on
+        return (summed if rows_index is None else residual), None
     out = (source * torch.rsqrt((source * source).mean(-1, keepdim=True) + eps) * weight.float()).to(dtype)
     return (summed if rows_index is None else residual), out
 

@@ -371,6 +371,46 @@ def test_attention_mixed_batch(kernel_sets, dtype, heads, kv_heads, head_dim, pa
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize(
+    "heads,kv_heads,head_dim,value_dim,page,window,chunk,keep_first,softcap,sink",
+    [(4, 4, 96, 32, 16, None, None, 0, 0.0, True), (6, 1, 64, 32, 16, None, None, 0, 0.0, False), (6, 3, 80, 48, 8, 37, None, 0, 0.0, True),
+     (8, 2, 128, 64, 16, 100, None, 5, 0.0, False), (2, 2, 32, 96, 16, None, 50, 0, 0.0, False), (20, 1, 64, 128, 32, None, None, 0, 2.5, True),
+     (18, 2, 96, 96, 16, 64, None, 17, 0.0, False), (3, 1, 112, 120, 4, 9, None, 2, 1.5, True), (5, 5, 40, 8, 16, None, 128, 0, 0.0, True),
+     (1, 1, 8, 128, 64, 130, None, 0, 0.0, False), (10, 2, 48, 48, 128, None, None, 0, 0.0, False)],
+)
+def test_attention_of_heads_that_fill_no_tile(kernel_sets, dtype, heads, kv_heads, head_dim, value_dim, page, window, chunk, keep_first,
+                                              softcap, sink):
+    """Keys and values of sizes of their own, padded on the way into the tensor-core kernels' tiles: portions beside single
+    tokens, with every mask and score option; then one token behind thousands (its keys split over many CTAs and merged)
+    and four behind hundreds (merged inside a cluster).  The cache's unused rows and the pages around hold numbers that
+    would show."""
+    from distie_b200.kernels.interface import KvSlot
+
+    ks = kernel_sets[dtype]
+    g = torch.Generator(device="cuda").manual_seed(head_dim + value_dim)
+    sinks = torch.randn(heads, generator=g, device="cuda") if sink else None
+    for tokens_per_seq, pasts in (([1, 23, 1, 200, 1], [130, 45, 0, 310, 63]), ([1], [6000]), ([1, 1, 1, 1], [700, 1300, 15, 900])):
+        lengths = [p + n for p, n in zip(pasts, tokens_per_seq)]
+        keys = filled_cache_for(dtype, kv_heads, head_dim, page, lengths)
+        values = torch.randn(*keys.k.shape[:3], value_dim, generator=g, device="cuda").to(dtype)
+        kv = KvSlot(keys.k, values, keys.block_table, page, keys.num_pages)
+        step = step_of(tokens_per_seq, pasts, list(range(len(lengths))))
+        q = torch.randn(step.num_tokens, heads * head_dim, generator=g, device="cuda").to(dtype)
+        out = torch.full((step.num_tokens, heads * value_dim), float("nan"), dtype=dtype, device="cuda")
+        ks.kernel_counts.clear()
+        ks.attention(q, out, step, kv, heads, kv_heads, head_dim, window, head_dim**-0.5, chunk, keep_first, softcap, sinks)
+        ks.check_errors()
+        want = ref.attention(q, step, kv, heads, kv_heads, head_dim, window, head_dim**-0.5, chunk, keep_first, softcap, sinks)
+        close(out, want, dtype, f"attention, {tokens_per_seq}")
+        if dtype == torch.bfloat16:
+            assert ks.kernel_counts.get("attention_decode_mma")
+            if max(tokens_per_seq) > 1:
+                assert ks.kernel_counts.get("attention_prefill_tcgen05" if page >= 8 else "attention_generic")
+            else:
+                assert not ks.kernel_counts.get("attention_generic")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("head_dim,heads,kv_heads", [(128, 12, 2), (64, 6, 1), (128, 40, 2)])
 @pytest.mark.parametrize("splits", [1, 2, 3, 8, 13, 17, 40])
 def test_decode_attention_at_every_split_count(kernel_sets, dtype, head_dim, heads, kv_heads, splits, monkeypatch):
