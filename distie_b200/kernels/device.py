@@ -407,7 +407,7 @@ class DeviceKernels(KernelSet):
         ragged = (self.dtype == torch.bfloat16 and not (same and head_dim in _DECODE_HEAD_DIMS) and head_dim % 8 == 0
                   and value_dim % 8 == 0 and _RAGGED_FROM <= max(head_dim, value_dim) <= max(_PREFILL_HEAD_DIMS)
                   and qkv.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and kv.k.is_contiguous() and kv.v.is_contiguous())
-        tile_dim = (64 if max(head_dim, value_dim) <= 64 else 128) if ragged else head_dim
+        tile_dim = (64 if max(head_dim, value_dim) <= 64 else 128) if ragged else (head_dim if same else 0)  # 0: no tiles
         n_dec = step.num_decode_tokens if ragged or (head_dim in _DECODE_HEAD_DIMS and same) else 0
         element = qkv.element_size()
         if n_dec > 0:
