@@ -52,13 +52,21 @@
 
 namespace distie {
 
+// FLAT: keys and values do not come from pages but from matrices whose rows are keys, in blocks of 128 rows that the block
+// table names (a row of it per request of the step): a key of head h is [columns h * key_dim .. of map_k | the row of
+// map_kr, shared by all heads], a query [columns h * key_dim .. of map_q | columns h * rot_dim .. of map_qr], a value
+// columns h * value_dim .. of map_v.  DK is key_dim, 64 or 128, plus 64 for the shared part (up to 64 elements, the rest
+// zeros from its map).  Attention through a latent runs this way on portions of prompts, its keys and values expanded.
+
 constexpr int kAttnRows = 128;     // query rows of a tile = lanes of tensor memory
 constexpr int kAttnKeys = 128;     // keys per block
 constexpr int kAttnGroupKeys = kAttnKeys / 2;  // keys of a block that one softmax group owns
 constexpr int kAttnSoftmaxWarps = 8;
 constexpr int kAttnVProducerWarp = 2 + kAttnSoftmaxWarps;  // behind the softmax warps
 constexpr int kAttnThreads = (3 + kAttnSoftmaxWarps) * 32;
-constexpr int kAttnKStages = 2, kAttnVStages = 3;  // V of a block is needed a block time after its stage is freed, K two
+constexpr int kAttnKStages = 2;
+// V of a block is needed a block time after its stage is freed, K two; keys of more than 128 elements leave room for two.
+__host__ __device__ constexpr int attn_v_stages(int key_tile) { return key_tile > 128 ? 2 : 3; }
 constexpr int kAttnHalf = kAttnRows * 128;  // bytes of one [128 rows x 64 elements] swizzled half tile
 constexpr float kAttnRaise = 8.f;  // the maximum in use is raised when a row exceeds it by this much (base 2)
 
@@ -66,10 +74,10 @@ template <int DK, int DV>
 struct AttnShared {
   alignas(1024) unsigned char q[kAttnRows * (DK > DV ? DK : DV) * 2];  // at the end: the output tile
   alignas(1024) unsigned char k[kAttnKStages][kAttnKeys * DK * 2];
-  alignas(1024) unsigned char v[kAttnVStages][kAttnKeys * DV * 2];
+  alignas(1024) unsigned char v[attn_v_stages(DK)][kAttnKeys * DV * 2];
   uint64_t q_full;
   uint64_t k_full[kAttnKStages], k_empty[kAttnKStages];
-  uint64_t v_full[kAttnVStages], v_empty[kAttnVStages];
+  uint64_t v_full[attn_v_stages(DK)], v_empty[attn_v_stages(DK)];
   uint64_t s_full[2];
   uint64_t p_full[2][2];  // [group][S buffer]
   uint64_t pv_done[2];    // [group]
@@ -112,15 +120,16 @@ __device__ __forceinline__ uint64_t add_pairs(uint64_t a, uint64_t b) {
   return d;
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool FLAT>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                  const __grid_constant__ CUtensorMap map_v,
-                                 const __grid_constant__ CUtensorMap map_out, __nv_bfloat16* __restrict__ out,
+                                 const __grid_constant__ CUtensorMap map_out, const __grid_constant__ CUtensorMap map_qr,
+                                 const __grid_constant__ CUtensorMap map_kr, __nv_bfloat16* __restrict__ out,
                                  int out_row_stride, const int* __restrict__ q_tiles,
                                  const int* __restrict__ positions, const int* __restrict__ token_seq,
                                  const int* __restrict__ seq_seat, const int* __restrict__ block_table,
-                                 int table_width, int group_size, int num_kv_heads, int key_dim, int value_dim,
+                                 int table_width, int group_size, int num_kv_heads, int key_dim, int rot_dim, int value_dim,
                                  int page_shift, int num_pages, int window, int key_chunk, int keep_first, float scale_log2, float cap, float cap_pre,
                                  const float* __restrict__ sink_logits, int* __restrict__ error) {
   // cap > 0: a raw score s becomes tanh(s * cap_pre) (cap_pre = scale / cap) and scale_log2 is cap * log2(e): the
@@ -129,6 +138,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
   extern __shared__ unsigned char raw[];
   auto& sm = *reinterpret_cast<AttnShared<DK, DV>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
   constexpr int K_HALVES = DK / 64, V_HALVES = DV / 64;
+  constexpr int kAttnVStages = attn_v_stages(DK);
   constexpr uint32_t TMEM_COLS = 512;
   constexpr uint32_t O_COL = 256;  // S0 | S1 | O of group 0 | O of group 1
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -139,6 +149,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     prefetch_tensor_map(&map_k);
     prefetch_tensor_map(&map_v);
     prefetch_tensor_map(&map_out);
+    if (FLAT) {
+      prefetch_tensor_map(&map_qr);
+      prefetch_tensor_map(&map_kr);
+    }
   }
   if (threadIdx.x == 0) {
     mbar_init(&sm.q_full, 1);
@@ -183,7 +197,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
   const int kv_head = head / group_size;
   const int t0 = q_tiles[2 * tile], rows = q_tiles[2 * tile + 1];
   const int pos0 = positions[t0];
-  const int seat = seq_seat[token_seq[t0]];
+  const int seat = FLAT ? token_seq[t0] : seq_seat[token_seq[t0]];  // the tile's row of the block table
   const int last_pos = pos0 + rows - 1;
   const int first_key = first_visible_key(pos0, window, key_chunk);
   const int block_first = first_key / kAttnKeys;
@@ -219,7 +233,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     const bool for_k = warp == 0;
     if (for_k && lane == 0) {
       mbar_expect_tx(&sm.q_full, kAttnRows * DK * 2);
-      for (int h = 0; h < K_HALVES; ++h) tma_load_2d(sm.q + h * kAttnHalf, &map_q, &sm.q_full, head * key_dim + h * 64, t0);
+      for (int h = 0; h < K_HALVES; ++h) {
+        if (FLAT && h == K_HALVES - 1) tma_load_2d(sm.q + h * kAttnHalf, &map_qr, &sm.q_full, head * rot_dim, t0);
+        else tma_load_2d(sm.q + h * kAttnHalf, &map_q, &sm.q_full, head * key_dim + h * 64, t0);
+      }
     }
     const int stages = for_k ? kAttnKStages : kAttnVStages, halves = for_k ? K_HALVES : V_HALVES;
     const CUtensorMap* map = for_k ? &map_k : &map_v;
@@ -243,8 +260,12 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
       __syncwarp();
       if (mine) {
         unsigned char* stage = (for_k ? sm.k[s] : sm.v[s]) + lane * page_size * 128;
-        const int row = (page * num_kv_heads + kv_head) * page_size;
-        for (int h = 0; h < halves; ++h) tma_load_2d(stage + h * kAttnHalf, map, &full[s], h * 64, row);
+        const int row = (FLAT ? page : page * num_kv_heads + kv_head) * page_size;
+        const int column = FLAT ? kv_head * (for_k ? key_dim : value_dim) : 0;
+        for (int h = 0; h < halves; ++h) {
+          if (FLAT && for_k && h == K_HALVES - 1) tma_load_2d(stage + h * kAttnHalf, &map_kr, &full[s], 0, row);
+          else tma_load_2d(stage + h * kAttnHalf, map, &full[s], column + h * 64, row);
+        }
       }
       issued = j + 1;
     }
@@ -510,25 +531,25 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
   if (threadIdx.x == 0 && sm.failed && error) atomicCAS(error, 0, 6);
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool FLAT>
 static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v,
-                               const CUtensorMap& map_out, void* out,
+                               const CUtensorMap& map_out, const CUtensorMap& map_qr, const CUtensorMap& map_kr, void* out,
                                int out_row_stride, const int* q_tiles, int num_tiles, const int* positions,
                                const int* token_seq, const int* seq_seat, const int* block_table, int table_width,
-                               int num_heads, int num_kv_heads, int key_dim, int value_dim, int page_shift, int num_pages,
+                               int num_heads, int num_kv_heads, int key_dim, int rot_dim, int value_dim, int page_shift, int num_pages,
                                int window, int key_chunk, int keep_first, float scale_log2, float cap, float cap_pre, const float* sink, int* error, cudaStream_t stream) {
   const size_t shared = sizeof(AttnShared<DK, DV>) + 1024;
   static bool configured = false;
   if (!configured) {
-    const cudaError_t err = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel<DK, DV>,
+    const cudaError_t err = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel<DK, DV, FLAT>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     if (err != cudaSuccess) return (int)err;
     configured = true;
   }
   const cudaError_t err = launch_dependent_family(
-      32, attention_prefill_tcgen05_kernel<DK, DV>, dim3(num_heads, num_tiles), dim3(kAttnThreads), shared, stream, map_q,
-      map_k, map_v, map_out, (__nv_bfloat16*)out, out_row_stride, q_tiles, positions, token_seq, seq_seat, block_table,
-      table_width, num_heads / num_kv_heads, num_kv_heads, key_dim, value_dim, page_shift, num_pages, window, key_chunk, keep_first, scale_log2,
+      32, attention_prefill_tcgen05_kernel<DK, DV, FLAT>, dim3(num_heads, num_tiles), dim3(kAttnThreads), shared, stream, map_q,
+      map_k, map_v, map_out, map_qr, map_kr, (__nv_bfloat16*)out, out_row_stride, q_tiles, positions, token_seq, seq_seat, block_table,
+      table_width, num_heads / num_kv_heads, num_kv_heads, key_dim, rot_dim, value_dim, page_shift, num_pages, window, key_chunk, keep_first, scale_log2,
       cap, cap_pre, sink, error);
   return err == cudaSuccess ? 0 : (int)err;
 }
@@ -569,10 +590,10 @@ extern "C" int distie_attention_prefill_tcgen05(const void* q, int q_row_stride,
   const float cap = softcap > 0.f ? softcap : 0.f, cap_pre = cap > 0.f ? scale / cap : 0.f;
   const float scale_log2 = (cap > 0.f ? cap : scale) * 1.4426950408889634f;
 #define DISTIE_ATTENTION_TC(DKV, DVV)                                                                                          \
-  return launch_attention_tc<DKV, DVV>(map_q, map_k, map_v, map_out, out, out_row_stride, q_tiles, num_tiles, positions, token_seq, \
-                                       seq_seat, block_table, table_width, num_heads, num_kv_heads, head_dim, value_dim,         \
-                                       page_shift, num_pages, window, key_chunk, keep_first, scale_log2, cap, cap_pre, sink,     \
-                                       error, stream)
+  return launch_attention_tc<DKV, DVV, false>(map_q, map_k, map_v, map_out, map_q, map_k, out, out_row_stride, q_tiles,          \
+                                              num_tiles, positions, token_seq, seq_seat, block_table, table_width, num_heads,   \
+                                              num_kv_heads, head_dim, 0, value_dim, page_shift, num_pages, window, key_chunk,   \
+                                              keep_first, scale_log2, cap, cap_pre, sink, error, stream)
   if (head_dim <= 64) {
     if (value_dim <= 64) DISTIE_ATTENTION_TC(64, 64);
     DISTIE_ATTENTION_TC(64, 128);
@@ -580,4 +601,42 @@ extern "C" int distie_attention_prefill_tcgen05(const void* q, int q_row_stride,
   if (value_dim <= 64) DISTIE_ATTENTION_TC(128, 64);
   DISTIE_ATTENTION_TC(128, 128);
 #undef DISTIE_ATTENTION_TC
+}
+
+// Portions of prompts whose keys and values are rows of matrices (the kernel's FLAT form).  q [tokens, heads * dim], q_rot
+// [tokens, heads * rot], keys [rows, heads * dim] and values [rows, heads * value_dim] with row stride kv_stride, shared
+// [rows, rot], out [tokens, heads * value_dim]: bfloat16.  `rows` is a multiple of 128; block_table [requests of the step,
+// table_width] names, for every block of 128 positions of a request, its block of 128 rows.  window <= 0: none.  sink: one
+// float per head or null.  Returns DISTIE_ERR_UNSUPPORTED for a dim that is neither 64 nor 128, a rot of 0, above 64 or no
+// multiple of 8, a value_dim above 128 or no multiple of 8.
+extern "C" int distie_attention_flat_tcgen05(const void* q, const void* q_rot, const void* keys, const void* shared,
+                                             const void* values, int kv_stride, void* out, const int* q_tiles, int num_tiles,
+                                             const int* positions, const int* token_seq, const int* block_table, int table_width,
+                                             int tokens, int rows, int num_heads, int dim, int rot, int value_dim, int window,
+                                             float scale, const float* sink, int* error, cudaStream_t stream) {
+  if (num_tiles <= 0) return 0;
+  if (tokens < 1 || num_heads < 1 || table_width < 1 || rows < 128 || (rows & 127) || num_tiles > 65535) return DISTIE_ERR_ARG;
+  if ((dim != 64 && dim != 128) || rot < 8 || rot > 64 || (rot & 7) || value_dim < 8 || value_dim > 128 || (value_dim & 7) ||
+      (kv_stride & 7) || (((uintptr_t)q | (uintptr_t)q_rot | (uintptr_t)keys | (uintptr_t)shared | (uintptr_t)values | (uintptr_t)out) & 15))
+    return DISTIE_ERR_UNSUPPORTED;
+  CUtensorMap map_q, map_qr, map_k, map_kr, map_v, map_out;
+  int status;
+  if ((status = make_map(&map_q, q, tokens, num_heads * dim, num_heads * dim, kAttnRows)) != 0) return status;
+  if ((status = make_map(&map_qr, q_rot, tokens, num_heads * rot, num_heads * rot, kAttnRows)) != 0) return status;
+  if ((status = make_map(&map_k, keys, rows, num_heads * dim, kv_stride, kAttnKeys)) != 0) return status;
+  if ((status = make_map(&map_kr, shared, rows, rot, rot, kAttnKeys)) != 0) return status;
+  if ((status = make_map(&map_v, values, rows, num_heads * value_dim, kv_stride, kAttnKeys)) != 0) return status;
+  if ((status = make_map(&map_out, out, tokens, num_heads * value_dim, num_heads * value_dim, kAttnRows)) != 0) return status;
+#define DISTIE_ATTENTION_FLAT(DKV, DVV)                                                                                      \
+  return launch_attention_tc<DKV, DVV, true>(map_q, map_k, map_v, map_out, map_qr, map_kr, out, num_heads * value_dim, q_tiles, \
+                                             num_tiles, positions, token_seq, nullptr, block_table, table_width, num_heads,   \
+                                             num_heads, dim, rot, value_dim, 7, rows / 128, window, 0, 0,                     \
+                                             scale * 1.4426950408889634f, 0.f, 0.f, sink, error, stream)
+  if (dim == 64) {
+    if (value_dim <= 64) DISTIE_ATTENTION_FLAT(128, 64);
+    DISTIE_ATTENTION_FLAT(128, 128);
+  }
+  if (value_dim <= 64) DISTIE_ATTENTION_FLAT(192, 64);
+  DISTIE_ATTENTION_FLAT(192, 128);
+#undef DISTIE_ATTENTION_FLAT
 }

@@ -4,8 +4,10 @@
 //
 //   latent_kv_write   float32 projection [q latent | kv latent | key part | ...] (or its slices) -> both RMS norms,
 //                     the rotation of the key part, the token's row into its page, the normed query latent out.
-//   latent_q_prepare  float32 query projection (per head [plain | to rotate]) -> plain part [heads, T, dim] and
-//                     rotated part [T, heads, rot] in the engine's type.
+//   latent_q_prepare  float32 query projection (per head [plain | to rotate]) -> plain part (by heads, then tokens, or
+//                     the other way round) and rotated part [T, heads, rot] in the engine's type.
+//   latent_gather     a request's cached rows out of their pages into matrices, for portions whose keys and values
+//                     are expanded per head by a product.
 //   latent_attention  (kernels below) causal softmax over the request's rows with a sink in the denominator.
 //   latent_gate       [heads, T, vdim] -> [T, heads * vdim] times sigmoid(gate[t, head]).
 //   glu_act           float32 [T, 2 ff] (gate columns, then up columns) -> SwiGLU or its capped form, optionally
@@ -87,32 +89,57 @@ latent_kv_write_kernel(const float* __restrict__ proj, int row_stride, int slice
   for (int c = rotary_dim + threadIdx.x; c < rot_dim; c += blockDim.x) dst[kv_rank + c] = from_float<T>(part[c]);
 }
 
-// One block per token: every head's plain columns to plain[head, t, :], its rotated columns to rotated[t, head, :].
+// A token's heads shared out over gridDim.y blocks: every head's plain columns to plain[head * head_stride + t * token_stride],
+// its rotated columns to rotated[t, head, :].  The token's angles are made once per block.  Shared memory: rotary_dim floats.
 template <typename T>
 __global__ void __launch_bounds__(256)
-latent_q_prepare_kernel(const float* __restrict__ q, int row_stride, int slices, long long slice_stride, int tokens,
-                        int heads, int dim, int rot_dim, const int* __restrict__ positions,
-                        const float* __restrict__ inv_freq, float factor, int rotary_dim, int interleaved,
-                        T* __restrict__ plain, T* __restrict__ rotated) {
+latent_q_prepare_kernel(const float* __restrict__ q, int row_stride, int slices, long long slice_stride, int heads, int dim,
+                        int rot_dim, const int* __restrict__ positions, const float* __restrict__ inv_freq, float factor,
+                        int rotary_dim, int interleaved, T* __restrict__ plain, long long head_stride, long long token_stride,
+                        T* __restrict__ rotated, int quads) {
+  extern __shared__ float row_s[];
   const int t = blockIdx.x;
-  const float* src = q + (size_t)t * row_stride;
+  const int per_block = (heads + gridDim.y - 1) / gridDim.y;
+  const int h0 = blockIdx.y * per_block, count = min(heads, h0 + per_block) - h0;
+  if (count <= 0) return;
   const int per_head = dim + rot_dim;
-  for (int c = threadIdx.x; c < heads * dim; c += blockDim.x) {
-    const int h = c / dim, d = c % dim;
-    plain[((size_t)h * tokens + t) * dim + d] = from_float<T>(sum_slices(src + h * per_head + d, slices, slice_stride));
-  }
-  const int pos = positions[t];
+  const float* src = q + (size_t)t * row_stride + h0 * per_head;
   const int half = rotary_dim / 2, loose = rot_dim - rotary_dim;
-  for (int c = threadIdx.x; c < heads * (half + loose); c += blockDim.x) {
+  const float pos = (float)positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf(pos * inv_freq[i], &sn, &cs);
+    row_s[i] = cs * factor;
+    row_s[half + i] = sn * factor;
+  }
+  if (quads) {  // four neighbours a thread: sizes and strides multiples of 4, aligned pointers
+    const int per = dim / 4;
+    for (int c = threadIdx.x; c < count * per; c += blockDim.x) {
+      const int h = c / per, d = 4 * (c % per);
+      const float* p = src + h * per_head + d;
+      float4 v = *reinterpret_cast<const float4*>(p);
+      for (int s = 1; s < slices; ++s) {
+        const float4 w = *reinterpret_cast<const float4*>(p + (size_t)s * slice_stride);
+        v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+      }
+      store4(plain + (size_t)(h0 + h) * head_stride + (size_t)t * token_stride + d, v);
+    }
+  } else {
+    for (int c = threadIdx.x; c < count * dim; c += blockDim.x) {
+      const int h = c / dim, d = c % dim;
+      plain[(size_t)(h0 + h) * head_stride + (size_t)t * token_stride + d] =
+          from_float<T>(sum_slices(src + h * per_head + d, slices, slice_stride));
+    }
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < count * (half + loose); c += blockDim.x) {
     const int h = c / (half + loose), i = c % (half + loose);
     const float* part = src + h * per_head + dim;
-    T* dst = rotated + ((size_t)t * heads + h) * rot_dim;
+    T* dst = rotated + ((size_t)t * heads + h0 + h) * rot_dim;
     if (i < half) {
       int a, b;
       rotary_pair(i, rotary_dim, interleaved, a, b);
-      float sn, cs;
-      sincosf((float)pos * inv_freq[i], &sn, &cs);
-      sn *= factor; cs *= factor;
+      const float cs = row_s[i], sn = row_s[half + i];
       const float u = sum_slices(part + a, slices, slice_stride), v = sum_slices(part + b, slices, slice_stride);
       dst[a] = from_float<T>(u * cs - v * sn);
       dst[b] = from_float<T>(v * cs + u * sn);
@@ -120,6 +147,34 @@ latent_q_prepare_kernel(const float* __restrict__ q, int row_stride, int slices,
       const int e = rotary_dim + i - half;
       dst[e] = from_float<T>(sum_slices(part + e, slices, slice_stride));
     }
+  }
+}
+
+// Cached rows [latent | rotated key part] of the step's requests, out of their pages, into two matrices of whole rows:
+// latents [rows, rank] and parts [rows, rot].  `blocks` [rows / 128, 4]: seat, first position, and the range of positions
+// [from, to) that are there; the others become zeros.  A warp takes a row, 16 bytes a lane.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ k_cache, const int* __restrict__ block_table, int table_width, int page_size,
+                     int num_pages, int rank8, int rot8, const int4* __restrict__ blocks, int rows, uint4* __restrict__ latents,
+                     uint4* __restrict__ parts, int* __restrict__ error) {
+  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const int4 block = blocks[row >> 7];  // x: seat, y: first position, z: from, w: to
+  const int pos = block.y + (row & 127);
+  const uint4* src = nullptr;
+  if (pos >= block.z && pos < block.w) {
+    const int column = pos / page_size;
+    const int page = column < table_width ? block_table[(size_t)block.x * table_width + column] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (lane == 0 && error) atomicExch(error, 5);
+    } else {
+      src = k_cache + ((size_t)page * page_size + pos % page_size) * (size_t)(rank8 + rot8);
+    }
+  }
+  for (int i = lane; i < rank8 + rot8; i += 32) {
+    const uint4 v = src ? src[i] : make_uint4(0u, 0u, 0u, 0u);
+    if (i < rank8) latents[(size_t)row * rank8 + i] = v;
+    else parts[(size_t)row * rot8 + i - rank8] = v;
   }
 }
 
@@ -431,22 +486,41 @@ extern "C" int distie_latent_kv_write(const float* proj, int row_stride, int sli
 
 extern "C" int distie_latent_q_prepare(const float* q, int row_stride, int slices, long long slice_stride, int tokens,
                                        int heads, int dim, int rot_dim, const int* positions, const float* inv_freq,
-                                       float factor, int rotary_dim, int interleaved, void* plain, void* rotated,
-                                       int dtype, cudaStream_t stream) {
+                                       float factor, int rotary_dim, int interleaved, void* plain, long long head_stride,
+                                       long long token_stride, void* rotated, int dtype, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (heads < 1 || dim < 1 || rot_dim < 0 || slices < 1 || (rotary_dim & 1) || rotary_dim < 0 || rotary_dim > rot_dim ||
-      (rotary_dim > 0 && !inv_freq))
+  if (heads < 1 || heads > 65535 || dim < 1 || rot_dim < 0 || slices < 1 || (rotary_dim & 1) || rotary_dim < 0 ||
+      rotary_dim > rot_dim || (rotary_dim > 0 && !inv_freq) || rotary_dim > 8192)
     return DISTIE_ERR_ARG;
+  const int quads = dim % 4 == 0 && rot_dim % 4 == 0 && row_stride % 4 == 0 && slice_stride % 4 == 0 && head_stride % 4 == 0 &&
+                    token_stride % 4 == 0 && (((uintptr_t)q | (uintptr_t)plain) & 15) == 0;
+  const dim3 grid(tokens, tokens < 512 ? heads : 1);
+  const int threads = tokens < 512 ? 128 : 256;
+  const size_t shared = (size_t)rotary_dim * sizeof(float);
   if (dtype == DISTIE_BF16)
-    latent_q_prepare_kernel<<<tokens, 256, 0, stream>>>(q, row_stride, slices, slice_stride, tokens, heads, dim, rot_dim,
-                                                        positions, inv_freq, factor, rotary_dim, interleaved,
-                                                        (__nv_bfloat16*)plain, (__nv_bfloat16*)rotated);
+    latent_q_prepare_kernel<<<grid, threads, shared, stream>>>(q, row_stride, slices, slice_stride, heads, dim, rot_dim, positions,
+                                                               inv_freq, factor, rotary_dim, interleaved, (__nv_bfloat16*)plain,
+                                                               head_stride, token_stride, (__nv_bfloat16*)rotated, quads);
   else if (dtype == DISTIE_F32)
-    latent_q_prepare_kernel<<<tokens, 256, 0, stream>>>(q, row_stride, slices, slice_stride, tokens, heads, dim, rot_dim,
-                                                        positions, inv_freq, factor, rotary_dim, interleaved,
-                                                        (float*)plain, (float*)rotated);
+    latent_q_prepare_kernel<<<grid, threads, shared, stream>>>(q, row_stride, slices, slice_stride, heads, dim, rot_dim, positions,
+                                                               inv_freq, factor, rotary_dim, interleaved, (float*)plain, head_stride,
+                                                               token_stride, (float*)rotated, quads);
   else
     return DISTIE_ERR_UNSUPPORTED;
+  DISTIE_LAUNCH_CHECK();
+  return 0;
+}
+
+// bfloat16 rows of rank + rot elements (multiples of 8) out of the pages; `rows` a multiple of 128.
+extern "C" int distie_latent_gather(const void* k_cache, const int* block_table, int table_width, int page_size, int num_pages,
+                                    int rank, int rot, const int* blocks, int rows, void* latents, void* parts, int* error,
+                                    cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (rank < 8 || (rank & 7) || rot < 8 || (rot & 7) || page_size < 1 || table_width < 1 || (rows & 127)) return DISTIE_ERR_ARG;
+  if (((uintptr_t)k_cache | (uintptr_t)blocks | (uintptr_t)latents | (uintptr_t)parts) & 15) return DISTIE_ERR_UNSUPPORTED;
+  latent_gather_kernel<<<(rows + 7) / 8, 256, 0, stream>>>((const uint4*)k_cache, block_table, table_width, page_size, num_pages,
+                                                           rank / 8, rot / 8, (const int4*)blocks, rows, (uint4*)latents,
+                                                           (uint4*)parts, error);
   DISTIE_LAUNCH_CHECK();
   return 0;
 }

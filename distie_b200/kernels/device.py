@@ -18,6 +18,7 @@ from __future__ import annotations
 import torch
 
 import ctypes
+from dataclasses import replace
 
 from . import library
 from .interface import KernelSet, Normed, StepTensors, Terms
@@ -35,6 +36,8 @@ _RULES = {"delta": 0, "ssd": 1, "gated": 2}
 _ACTS = {"relu2": 1, "gelu": 2, "xielu": 3}
 _SCORINGS = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
 _PLAIN_ACTS = {"none": 0, "silu": 1, "tanh": 2}
+_EXPAND_QUERIES = 64            # queries a cached row must serve on average for its expansion to keys and values to pay
+_EXPAND_BYTES = 1 << 30         # and the most that the expanded keys and values of a step may take
 _GROUPED_TENSOR_CORE_PAIRS = 512  # (token, expert) pairs from which the routed products run on the tcgen05 tile kernel
 
 _ERROR_TEXT = {
@@ -1152,23 +1155,108 @@ class DeviceKernels(KernelSet):
         )
         self._ran("latent_kv_write")
 
-    def latent_queries(self, q, up_keys, step, rotary, num_heads, dim, rot_dim):
+    def _latent_q(self, q, step, rotary, num_heads, dim, rot_dim, by_token: bool):
+        """(plain, rotated): ``plain [heads, T, dim]``, or ``[T, heads, dim]`` by token; ``rotated [T, heads, rot_dim]``."""
+        library.load_unit("latent")
         tokens = step.num_tokens
-        plain = torch.empty((num_heads, tokens, dim), dtype=self.dtype, device=q.device)
+        plain = torch.empty((tokens, num_heads, dim) if by_token else (num_heads, tokens, dim), dtype=self.dtype, device=q.device)
         rotated = torch.empty((tokens, num_heads, rot_dim), dtype=self.dtype, device=q.device)
+        head_stride, token_stride = (dim, num_heads * dim) if by_token else (tokens * dim, dim)
         check(
             function("distie_latent_q_prepare")(
                 *self._sliced(q, "latent_queries"), tokens, num_heads, dim, rot_dim, step.positions.data_ptr(),
                 rotary.inv_freq.data_ptr() if rotary is not None else None,
                 float(rotary.factor) if rotary is not None else 1.0, rotary.rotary_dim if rotary is not None else 0,
-                int(rotary.interleaved) if rotary is not None else 0, plain.data_ptr(), rotated.data_ptr(), self.code,
-                self._stream(),
+                int(rotary.interleaved) if rotary is not None else 0, plain.data_ptr(), head_stride, token_stride,
+                rotated.data_ptr(), self.code, self._stream(),
             ),
             "latent_q_prepare",
         )
         self._ran("latent_q_prepare")
+        return plain, rotated
+
+    def latent_queries(self, q, up_keys, step, rotary, num_heads, dim, rot_dim):
+        plain, rotated = self._latent_q(q, step, rotary, num_heads, dim, rot_dim, by_token=False)
         # per head [T, dim] x [dim, kv_rank]: a batched library product (float32 accumulation; FMA-only in the float32 set)
         return torch.bmm(plain, up_keys), rotated
+
+    def _expansion_plan(self, step, seqs, window: int):
+        """Which rows the step's portions read, in blocks of 128 positions: ``(blocks [n, 4], table [requests, width],
+        rows)`` on the device, or None when the portions are too short against what they read (every row is expanded
+        once, whatever the number of queries).  Made once per step and window."""
+        key = ("expansion_plan", window)
+        if key in step.derived:
+            return step.derived[key]
+        blocks, spans, work = [], {}, 0
+        for row, s in enumerate(seqs):
+            if s.q_len < 2:
+                continue
+            end = s.past_len + s.q_len
+            first = max(0, s.past_len - window + 1) if window else 0
+            spans[row] = (first // 128, len(blocks))
+            blocks += [(s.seat, 128 * b, first, end) for b in range(first // 128, -(-end // 128))]
+            work += s.q_len * (end - first)
+        made = None
+        if blocks and work >= _EXPAND_QUERIES * 128 * len(blocks):
+            width = max(b[3] for b in blocks)
+            table = torch.full((len(seqs), -(-width // 128)), -1, dtype=torch.int32)
+            for row, (first_block, at) in spans.items():
+                count = -(-(seqs[row].past_len + seqs[row].q_len) // 128) - first_block
+                table[row, first_block : first_block + count] = torch.arange(at, at + count, dtype=torch.int32)
+            made = (torch.tensor(blocks, dtype=torch.int32).to(self.device), table.to(self.device), 128 * len(blocks))
+        step.derived[key] = made
+        return made
+
+    def latent_heads(self, q, up_keys, up_values, up_rows, gate, step, seqs, kv, rotary, num_heads, dim, rot_dim, value_dim, kv_rank,
+                     scale, sink, window=None):
+        """Portions of prompts long enough to pay for it: the rows they read are gathered from their pages, one product
+        makes every head's keys and values of them, and the tcgen05 attention runs over those (dim 64 or 128, up to 64
+        rotated dimensions, values of up to 128).  Everything else: queries folded into the latent's space."""
+        singles, tokens = step.num_decode_tokens, step.num_tokens
+        columns = num_heads * (dim + value_dim)
+        plan = None
+        if (self.dtype == torch.bfloat16 and seqs and tokens > singles and step.num_q_tiles and dim in (64, 128)
+                and 8 <= rot_dim <= 64 and rot_dim % 8 == 0 and value_dim % 8 == 0 and value_dim <= 128 and kv_rank % 8 == 0
+                and scale > 0 and up_rows.dtype == torch.bfloat16 and kv.k.dtype == torch.bfloat16):
+            plan = self._expansion_plan(step, seqs, int(window) if window else 0)
+        if plan is None or 2 * plan[2] * columns > _EXPAND_BYTES:
+            return super().latent_heads(q, up_keys, up_values, up_rows, gate, step, seqs, kv, rotary, num_heads, dim, rot_dim, value_dim,
+                                        kv_rank, scale, sink, window)
+        blocks, table, rows = plan
+        error, stream = self.error_flag.data_ptr(), self._stream()
+        plain, rotated = self._latent_q(q, step, rotary, num_heads, dim, rot_dim, by_token=True)
+        latents = torch.empty((rows, kv_rank), dtype=self.dtype, device=q.device)
+        parts = torch.empty((rows, rot_dim), dtype=self.dtype, device=q.device)
+        check(
+            function("distie_latent_gather")(
+                kv.k.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[-1], kv.page_size, kv.num_pages, kv_rank, rot_dim,
+                blocks.data_ptr(), rows, latents.data_ptr(), parts.data_ptr(), error, stream,
+            ),
+            "latent_gather",
+        )
+        self._ran("latent_gather")
+        expanded = self.linear(latents, up_rows)  # [rows, heads * dim keys | heads * value_dim values]
+        out = torch.empty((tokens, num_heads * value_dim), dtype=self.dtype, device=q.device)
+        check(
+            function("distie_attention_flat_tcgen05")(
+                plain.data_ptr(), rotated.data_ptr(), expanded.data_ptr(), parts.data_ptr(),
+                expanded.data_ptr() + 2 * num_heads * dim, expanded.stride(0), out.data_ptr(), step.q_tiles.data_ptr(),
+                step.num_q_tiles, step.positions.data_ptr(), step.token_seq.data_ptr(), table.data_ptr(), table.shape[1], tokens,
+                rows, num_heads, dim, rot_dim, value_dim, int(window) if window else 0, float(scale),
+                sink.data_ptr() if sink is not None else None, error, stream,
+            ),
+            "attention_flat_tcgen05",
+        )
+        self._ran("attention_flat_tcgen05")
+        if gate is not None:
+            self.head_gate(out[singles:], gate[..., singles:, :], num_heads)
+        if singles:  # the step's single tokens come first
+            few = replace(step, token_ids=step.token_ids[:singles], positions=step.positions[:singles],
+                          token_seq=step.token_seq[:singles], num_tokens=singles, q_tiles=None, num_q_tiles=0, derived={})
+            out[:singles] = super().latent_heads(q[..., :singles, :], up_keys, up_values, up_rows,
+                                                 gate[..., :singles, :] if gate is not None else None, few, seqs, kv, rotary, num_heads,
+                                                 dim, rot_dim, value_dim, kv_rank, scale, sink, window)
+        return out
 
     def latent_attention(self, folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, out, window=None) -> None:
         if kv.k.dtype != folded.dtype or not folded.is_contiguous() or not rotated.is_contiguous() or not out.is_contiguous():

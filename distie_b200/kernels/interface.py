@@ -379,6 +379,19 @@ class KernelSet(ABC):
         no gate)."""
         raise NotImplementedError
 
+    def latent_heads(self, q, up_keys, up_values, up_rows, gate, step: StepTensors, seqs, kv: KvSlot, rotary: RotaryTable | None,
+                     num_heads: int, dim: int, rot_dim: int, value_dim: int, kv_rank: int, scale: float, sink,
+                     window: int | None = None):
+        """From the float32 query projection (as :meth:`latent_queries` takes it) to what the output projection reads,
+        ``[T, heads * value_dim]``; the step's rows are in the cache already.  ``up_rows [heads * (dim + value_dim),
+        kv_rank]``: all heads' key rows, then all heads' value rows (``up_keys`` and ``up_values`` hold the same numbers);
+        ``seqs``: the step's requests as the host knows them (or None).  The default folds the queries into the latent's
+        space; a set may instead expand the latents of long portions to keys and values of every head."""
+        folded, rotated = self.latent_queries(q, up_keys, step, rotary, num_heads, dim, rot_dim)
+        mixed = torch.empty((num_heads, step.num_tokens, kv_rank), dtype=folded.dtype, device=folded.device)
+        self.latent_attention(folded, rotated, step, kv, num_heads, kv_rank, rot_dim, scale, sink, mixed, window)
+        return self.latent_values(mixed, up_values, gate, num_heads, value_dim)
+
     # -- layer norm, gates, short convolutions and linear recurrences (layers with per-request state) --------
     # Where a float32 input is marked "or slices" it may also be ``[S, T, n]``, the slices of a split product
     # (:meth:`linear_split`) or a view of their columns: the op adds them up while it loads.

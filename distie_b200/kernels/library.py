@@ -100,7 +100,11 @@ _SIGNATURES: dict[str, tuple[str, list]] = {
     "distie_latent_kv_write": (
         "latent", [P, I, I, L, I, P, I, P, I, F, P, I, P, P, P, P, I, P, F, I, I, P, I, I, I, I, I, P, P]
     ),
-    "distie_latent_q_prepare": ("latent", [P, I, I, L, I, I, I, I, P, P, F, I, I, P, P, I, P]),
+    "distie_latent_q_prepare": ("latent", [P, I, I, L, I, I, I, I, P, P, F, I, I, P, L, L, P, I, P]),
+    "distie_latent_gather": ("latent", [P, P, I, I, I, I, I, P, I, P, P, P, P]),
+    "distie_attention_flat_tcgen05": (
+        "bf16", [P, P, P, P, P, I, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, P, P]
+    ),
     "distie_latent_attention_scratch_floats": ("latent", [I, I, I, I]),
     "distie_latent_attention": ("latent", [P, P, P, P, I, I, I, I, P, P, P, P, I, P, I, I, F, I, P, I, I, I, I, P, P]),
     "distie_latent_attention_single": ("latent", [P, P, P, P, I, I, I, I, P, P, P, P, I, P, I, I, F, I, P, I, I, I, P, P]),

@@ -16,7 +16,8 @@ Only ``[c | r]`` is cached, one row per token (a cache group of one kv head whos
 ``kv_rank`` columns of its keys).  Nothing is expanded per head when the cache is read: since
 ``q_plain . (W_uk c) = (W_uk^T q_plain) . c``, the plain part of a query is folded into the latent's space
 (``kv_rank`` numbers per head), the attention mixes cached latents, and ``W_uv`` is applied to the mix.  A step
-of one token and a portion of a prompt run the same ops.
+of one token and a portion of a prompt run the same op (:meth:`KernelSet.latent_heads`), which may instead expand the
+latents to keys and values where a portion is long enough to be worth it.
 
 A layer with ``own_latent=False`` has no ``W_dkv``: it reads the rows that the owner of its cache slot stored
 (after that layer's norm and rotation), with its own ``W_uk``, ``W_uv``, queries, sink, gate and output.
@@ -53,7 +54,7 @@ class LatentAttention:
     _NAMES = {"q": "q", "dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk",
               "uv": "uv", "sink": "sink", "g": "g", "o": "o"}
 
-    def __init__(self, prm: dict, kernels, position, down, q_norm, kv_norm, up_q, up_keys, up_values, sink, out) -> None:
+    def __init__(self, prm: dict, kernels, position, down, q_norm, kv_norm, up_q, up_rows, up_values, sink, out) -> None:
         self.kernels = kernels
         self.position = position
         self.num_heads = int(prm["num_heads"])
@@ -68,7 +69,9 @@ class LatentAttention:
         self.own_latent = bool(prm.get("own_latent", True))
         self.gated = bool(prm.get("gate"))
         self.down, self.q_norm, self.kv_norm = down, q_norm, kv_norm
-        self.up_q, self.up_keys, self.up_values = up_q, up_keys, up_values
+        self.up_q, self.up_rows, self.up_values = up_q, up_rows, up_values
+        keys = self.num_heads * self.head_dim  # up_rows: all heads' key rows, then all heads' value rows
+        self.up_keys = up_rows[:keys].view(self.num_heads, self.head_dim, self.kv_rank)
         self.sink, self.out = sink, out
 
     @classmethod
@@ -141,12 +144,12 @@ class LatentAttention:
         if prm.get("gate"):
             stacked.append(w.matrix(cls._name(spec, "g")))
         position = build_part(POSITION_ENCODINGS, prm.get("position") or PartSpec("none"), ctx)
-        up_keys = w.matrix(cls._name(spec, "uk")).reshape(heads, dim, rank).contiguous()              # [h, dim, rank]
+        up_rows = fuse_rows([w.matrix(cls._name(spec, "uk")), w.matrix(cls._name(spec, "uv"))])
         up_values = w.matrix(cls._name(spec, "uv")).reshape(heads, vdim, rank).transpose(1, 2).contiguous()  # [h, rank, vdim]
         return cls(
             dict(prm), ctx.kernels, position, fuse_rows(stacked),
             None if direct else w.vector(cls._name(spec, "dq_norm")), w.vector(cls._name(spec, "dkv_norm")) if own else None,
-            None if direct else w.matrix(cls._name(spec, "uq")), up_keys, up_values,
+            None if direct else w.matrix(cls._name(spec, "uq")), up_rows, up_values,
             w.vector(cls._name(spec, "sink")) if prm.get("sink") else None, w.matrix(cls._name(spec, "o")),
         )
 
@@ -171,10 +174,8 @@ class LatentAttention:
             k.latent_kv_write(proj, run.step, run.kv if self.own_latent else None, table, self.q_rank, self.q_norm,
                               self.kv_rank, self.kv_norm, self.rot_dim, self.eps, q_latent)
             q = k.linear(q_latent, self.up_q, None, torch.float32)
-        folded, rotated = k.latent_queries(q, self.up_keys, run.step, table, self.num_heads, self.head_dim, self.rot_dim)
-        mixed = torch.empty((self.num_heads, tokens, self.kv_rank), dtype=x.dtype, device=x.device)
-        k.latent_attention(folded, rotated, run.step, run.kv, self.num_heads, self.kv_rank, self.rot_dim, self.scale,
-                           self.sink, mixed, self.window)
         gate = proj[..., proj.shape[-1] - self.num_heads :] if self.gated else None
-        heads_out = k.latent_values(mixed, self.up_values, gate, self.num_heads, self.value_dim)
+        heads_out = k.latent_heads(q, self.up_keys, self.up_values, self.up_rows, gate, run.step, run.seqs, run.kv, table,
+                                   self.num_heads, self.head_dim, self.rot_dim, self.value_dim, self.kv_rank, self.scale,
+                                   self.sink, self.window)
         return k.linear_split(heads_out, self.out)  # summed by the norm that follows

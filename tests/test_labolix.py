@@ -625,6 +625,74 @@ def test_latent_attention_over_a_window_with_sinks(kit, heads, dim, rot, dims, v
         _close(torch.cat(got), want, 3e-5 if kit.dtype == torch.float32 else 3e-2, "latent attention")
 
 
+@pytest.mark.parametrize("heads,dim,rot,dims,vdim,rank,page,window,gated", [
+    (4, 64, 32, 32, 64, 128, 16, 70, False), (3, 128, 64, 64, 128, 256, 16, 200, False), (2, 64, 64, 48, 40, 64, 4, None, True),
+    (5, 128, 8, 8, 96, 72, 32, 129, False), (1, 64, 16, 16, 128, 512, 16, 1, False), (6, 128, 48, 32, 64, 128, 24, 1000, True),
+    (2, 32, 16, 16, 32, 64, 16, 60, False)])
+def test_latents_of_long_portions_expanded_to_keys_and_values(kit, heads, dim, rot, dims, vdim, rank, page, window, gated):
+    """The whole way from the query projection to the heads' outputs, three requests in a step: a single token behind a
+    long past, a long portion behind a past that is no multiple of a block, and one from position 0.  The rows before each
+    window are taken out of the block tables; marked rows sit at page, block and window borders, old ones the strongest."""
+    g = torch.Generator().manual_seed(rank + dim)
+    eps, base, scale = 1e-5, 100.0, 0.5
+    dev, on_gpu = kit.device, kit.device.type == "cuda"
+    pasts, counts = ([300, 261, 0], [1, 150, 140]) if on_gpu else ([40, 21, 0], [1, 30, 17])
+    lengths = [p + c for p, c in zip(pasts, counts)]
+    reach = window or 10 ** 6
+    up_k, up_v = torch.randn(heads, dim, rank, generator=g) / math.sqrt(rank), torch.randn(heads, vdim, rank, generator=g) / math.sqrt(rank)
+    sink = torch.linspace(-2.0, 3.0, heads)
+    if kit.dtype != torch.float32:
+        up_k, up_v = up_k.to(torch.bfloat16).float(), up_v.to(torch.bfloat16).float()
+    a = torch.randn(rank, generator=g)
+    a = a / a.norm()
+    columns = heads * (dim + rot)
+    freqs = pl.plain_frequencies(base, dims)
+    table = RotaryTable(torch.tensor(freqs, dtype=torch.float32, device=dev), dims, True)
+    width = pages_needed(max(lengths), page)
+    pages = 3 * width + 1
+    slab = torch.full((pages, 1, page, rank + rot), 7.0, dtype=kit.dtype, device=dev)
+    host = torch.full((3, width), -1, dtype=torch.int32)
+    order = torch.randperm(3 * width, generator=g).to(torch.int32).reshape(3, width)
+    qs, gates, wanted = [], [], []
+    for r, n in enumerate(lengths):
+        q = torch.randn(n, heads, dim + rot, generator=g)
+        q[..., :dim] += 2.0 * torch.einsum("hdr,r->hd", up_k, a) * math.sqrt(rank / dim)
+        c = torch.randn(n, rank, generator=g)
+        marks = {0: 5.0, **{j: 1.0 + (j * 5 % 7) * 0.3 for j in range(3, n, 9)}, **{b: 3.0 - b / n for b in range(page, n, 3 * page)},
+                 **{j: 2.5 for j in (127, 128, pasts[r] - 1, pasts[r], n - reach, n - reach - 1) if 0 <= j < n}}
+        for j, s in marks.items():
+            c[j] += s * a * math.sqrt(rank) / 3
+        part, gate = torch.randn(n, 1, rot, generator=g), torch.randn(n, heads, generator=g)
+        positions = torch.arange(n)
+        with pl.stored_as(torch.bfloat16 if kit.dtype != torch.float32 else None):
+            cd, rd = pl.stored(c.double()), pl.stored(part.double())
+            qd = torch.cat([pl.stored(q[..., :dim].double()), pl.stored(pl.turn(q[..., dim:].double(), positions, freqs, pl.neighbours))], -1)
+            keys = torch.cat([torch.einsum("hdr,tr->thd", up_k.double(), cd), rd.expand(n, heads, rot)], -1)
+            o = pl.attend(qd, keys, torch.einsum("hvr,tr->thv", up_v.double(), cd), scale, sink.double(), window)
+        if gated:
+            o = o * torch.sigmoid(gate.double())[..., None]
+        wanted.append(o.reshape(n, heads * vdim)[pasts[r] :])
+        qs.append(q.reshape(n, columns)[pasts[r] :])
+        gates.append(gate[pasts[r] :])
+        first = max(0, pasts[r] - reach + 1) // page
+        held = pages_needed(n, page)
+        host[r, first:held] = order[r, first:held]
+        for j in range(first * page, n):
+            slab[int(order[r, j // page]), 0, j % page] = torch.cat([cd[j], rd[j, 0]]).to(dev, kit.dtype)
+    kv = KvSlot(slab, slab[..., :rank], host.to(dev), page, pages)
+    step, layout = step_for(kit, [(r, [0] * counts[r], pasts[r], ()) for r in range(3)])
+    rows = torch.cat([in_slices(q) for q in qs], 1).to(dev)
+    up_rows = torch.cat([up_k.reshape(-1, rank), up_v.reshape(-1, rank)]).to(dev, kit.dtype)
+    keys_first = up_rows[: heads * dim].view(heads, dim, rank)
+    values_turned = up_rows[heads * dim :].view(heads, vdim, rank).transpose(1, 2).contiguous()
+    got = kit.latent_heads(rows, keys_first, values_turned, up_rows, in_slices(torch.cat(gates)).to(dev) if gated else None, step,
+                           layout.seqs, kv, table, heads, dim, rot, vdim, rank, scale, sink.to(dev), window)
+    kit.check_errors()
+    _close(got.float(), torch.cat(wanted), 3e-5 if kit.dtype == torch.float32 else 3e-2, "heads")
+    if on_gpu:
+        assert bool(kit.kernel_counts.get("attention_flat_tcgen05")) == (kit.dtype == torch.bfloat16 and dim >= 64)
+
+
 # -- each kind of layer alone in a model, then all of them ---------------------------------------------------
 ALONE = {
     "attention": [_attention(2, 1, 10, 6, 0.4, _rot(40.0, 6, BY_WAVE), None)],
