@@ -145,6 +145,32 @@ __device__ __forceinline__ float capped_log2(float s, const ScoreExtras& x) {
   return (x.cap * 1.4426950408889634f) * tanh_fast(s * x.cap_pre);
 }
 
+// The sum of `slices` numbers `stride` floats apart, in their order, seven loads in flight together: a product whose K was
+// split leaves its parts like this, and a plain loop would wait for every one of them in turn.
+__device__ __forceinline__ float sum_slices(const float* p, int slices, long long stride) {
+  float v = p[0];
+  for (int s = 1; s < slices; s += 7) {
+    float d[7];
+#pragma unroll
+    for (int u = 0; u < 7; ++u) d[u] = s + u < slices ? p[(size_t)(s + u) * stride] : 0.f;
+#pragma unroll
+    for (int u = 0; u < 7; ++u) v += d[u];
+  }
+  return v;
+}
+__device__ __forceinline__ float4 sum_slices4(const float* p, int slices, long long stride) {
+  float4 v = *reinterpret_cast<const float4*>(p);
+  for (int s = 1; s < slices; s += 7) {
+    float4 d[7];
+#pragma unroll
+    for (int u = 0; u < 7; ++u)
+      d[u] = s + u < slices ? *reinterpret_cast<const float4*>(p + (size_t)(s + u) * stride) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int u = 0; u < 7; ++u) { v.x += d[u].x; v.y += d[u].y; v.z += d[u].z; v.w += d[u].w; }
+  }
+  return v;
+}
+
 // Sum over a block of up to 1024 threads; `scratch` holds 32 floats of shared memory.
 // Every thread gets the result.  Safe to call repeatedly with the same scratch.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {

@@ -19,12 +19,6 @@
 
 namespace distie {
 
-__device__ __forceinline__ float sum_slices(const float* p, int slices, long long slice_stride) {
-  float v = p[0];
-  for (int s = 1; s < slices; ++s) v += p[(size_t)s * slice_stride];
-  return v;
-}
-
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 
 // The pair (a, b) of a rotation of `rotary_dim` dimensions: neighbours (interleaved) or half a rotation apart.
@@ -116,13 +110,8 @@ latent_q_prepare_kernel(const float* __restrict__ q, int row_stride, int slices,
     const int per = dim / 4;
     for (int c = threadIdx.x; c < count * per; c += blockDim.x) {
       const int h = c / per, d = 4 * (c % per);
-      const float* p = src + h * per_head + d;
-      float4 v = *reinterpret_cast<const float4*>(p);
-      for (int s = 1; s < slices; ++s) {
-        const float4 w = *reinterpret_cast<const float4*>(p + (size_t)s * slice_stride);
-        v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
-      }
-      store4(plain + (size_t)(h0 + h) * head_stride + (size_t)t * token_stride + d, v);
+      store4(plain + (size_t)(h0 + h) * head_stride + (size_t)t * token_stride + d,
+             sum_slices4(src + h * per_head + d, slices, slice_stride));
     }
   } else {
     for (int c = threadIdx.x; c < count * dim; c += blockDim.x) {

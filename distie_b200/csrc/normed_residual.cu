@@ -150,11 +150,18 @@ add_dynamic_tanh_kernel(ResidualTerms terms, float* residual, float alpha, const
     float4 r = load4_cg(residual + at);
     if (terms.count > 0) {
       float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-      for (int j = 0; j < terms.count; ++j) {
-        const float4 v = load4_cg(terms.ptr[j] + at);
-        const float s = terms.scale[j];
-        d.x += s * v.x; d.y += s * v.y; d.z += s * v.z; d.w += s * v.w;
+#pragma unroll
+      for (int j0 = 0; j0 < kResidualTerms; j0 += 12) {  // up to twelve terms in flight together
+        if (j0 >= terms.count) break;
+        float4 v[12];
+#pragma unroll
+        for (int j = 0; j < 12; ++j)
+          v[j] = j0 + j < terms.count ? load4_cg(terms.ptr[j0 + j] + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 12; ++j) {
+          const float s = j0 + j < terms.count ? terms.scale[j0 + j] : 0.f;
+          d.x += s * v[j].x; d.y += s * v[j].y; d.z += s * v[j].z; d.w += s * v[j].w;
+        }
       }
       r.x += d.x; r.y += d.y; r.z += d.z; r.w += d.w;
       if (!rows_index) *reinterpret_cast<float4*>(residual + at) = r;
@@ -300,10 +307,7 @@ struct SlicedRows {
   int splits;
   long long split_stride;
   __device__ __forceinline__ float at(size_t row, int col) const {
-    const float* q = p + row * stride + col;
-    float v = q[0];
-    for (int s = 1; s < splits; ++s) v += q[(size_t)s * split_stride];
-    return v;
+    return sum_slices(p + row * stride + col, splits, split_stride);
   }
 };
 

@@ -544,25 +544,46 @@ retention_single_kernel(Sliced qkv, Sliced gate, const int* __restrict__ positio
   }
   grid_dependency_wait();
   const int qk = heads * key_dim;
-  if ((int)threadIdx.x < loose) {  // key_dim <= 256: a thread per pair or element
+  const float* row = qkv.p + (size_t)t * qkv.stride;
+  const float* z_row = gate.p + (size_t)t * gate.stride + head * value_dim;
+  {
+    // Everything the thread reads of the projection is requested before any of it is used: a pair (or an element behind
+    // the pairs; key_dim <= 256) of q and of k, and its first elements of v and of the gate.
     const int i = threadIdx.x;
-    const int a = i < half ? (interleaved ? 2 * i : i) : half + i, b = interleaved ? 2 * i + 1 : i + half;
+    const bool has = i < loose, pair = i < half, value = i < value_dim;
+    const int a = pair ? (interleaved ? 2 * i : i) : half + i, b = interleaved ? 2 * i + 1 : i + half;
+    const float* q_at = row + head * key_dim;
+    const float* k_at = q_at + qk;
+    float qa = 0.f, qb = 0.f, ka = 0.f, kb = 0.f, v = 0.f;
+    for (int s = 0; s < qkv.splits; s += 4) {
+      float d[4][5];
 #pragma unroll
-    for (int part = 0; part < 2; ++part) {
-      const int column = part * qk + head * key_dim;
-      const float scale = part ? key_scale : 1.f;
-      float* dst = part ? k_s : q_s;
-      const float u = qkv.at(t, column + a);
-      if (i < half) {
-        const float v = qkv.at(t, column + b);
-        dst[a] = (u * cs - v * sn) * scale;
-        dst[b] = (v * cs + u * sn) * scale;
-      } else {
-        dst[a] = u * scale;
+      for (int u = 0; u < 4; ++u) {
+        const size_t off = (size_t)(s + u) * qkv.split_stride;
+        const bool there = s + u < qkv.splits;
+        d[u][0] = there && has ? q_at[off + a] : 0.f;
+        d[u][1] = there && pair ? q_at[off + b] : 0.f;
+        d[u][2] = there && has ? k_at[off + a] : 0.f;
+        d[u][3] = there && pair ? k_at[off + b] : 0.f;
+        d[u][4] = there && value ? row[off + 2 * qk + head * value_dim + i] : 0.f;
       }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) { qa += d[u][0]; qb += d[u][1]; ka += d[u][2]; kb += d[u][3]; v += d[u][4]; }
     }
+    if (pair) {
+      q_s[a] = qa * cs - qb * sn;
+      q_s[b] = qb * cs + qa * sn;
+      k_s[a] = (ka * cs - kb * sn) * key_scale;
+      k_s[b] = (kb * cs + ka * sn) * key_scale;
+    } else if (has) {
+      q_s[a] = qa;
+      k_s[a] = ka * key_scale;
+    }
+    if (value) v_s[i] = v;
+    for (int e = i + blockDim.x; e < value_dim; e += blockDim.x)
+      v_s[e] = sum_slices(row + 2 * qk + head * value_dim + e, qkv.splits, qkv.split_stride);
   }
-  for (int e = threadIdx.x; e < value_dim; e += blockDim.x) v_s[e] = qkv.at(t, 2 * qk + head * value_dim + e);
+  const float z_first = (int)threadIdx.x < value_dim ? sum_slices(z_row + threadIdx.x, gate.splits, gate.split_stride) : 0.f;
   __syncthreads();
   float q[PER], k[PER];
 #pragma unroll
@@ -616,9 +637,10 @@ retention_single_kernel(Sliced qkv, Sliced gate, const int* __restrict__ positio
   float sq = 0.f;
   for (int e = threadIdx.x; e < value_dim; e += blockDim.x) sq += o_s[e] * o_s[e];
   const float unit = 1.f / sqrtf(block_sum(sq, scratch) / (float)value_dim + eps);
-  for (int e = threadIdx.x; e < value_dim; e += blockDim.x)
-    out[(size_t)t * out_stride + head * value_dim + e] =
-        from_float<T>(o_s[e] * unit * gate_f(gate_sigmoid, gate.at(t, head * value_dim + e)));
+  for (int e = threadIdx.x; e < value_dim; e += blockDim.x) {
+    const float z = e < (int)blockDim.x ? z_first : sum_slices(z_row + e, gate.splits, gate.split_stride);
+    out[(size_t)t * out_stride + head * value_dim + e] = from_float<T>(o_s[e] * unit * gate_f(gate_sigmoid, z));
+  }
 }
 
 }  // namespace distie
