@@ -85,13 +85,15 @@ latent_kv_write_kernel(const float* __restrict__ proj, int row_stride, int slice
 
 // A token's heads shared out over gridDim.y blocks: every head's plain columns to plain[head * head_stride + t * token_stride],
 // its rotated columns to rotated[t, head, :].  The token's angles are made once per block.  Shared memory: rotary_dim floats.
-template <typename T>
+// WHOLE: the projection is one matrix, not the slices of a split product.
+template <typename T, bool WHOLE>
 __global__ void __launch_bounds__(256)
 latent_q_prepare_kernel(const float* __restrict__ q, int row_stride, int slices, long long slice_stride, int heads, int dim,
                         int rot_dim, const int* __restrict__ positions, const float* __restrict__ inv_freq, float factor,
                         int rotary_dim, int interleaved, T* __restrict__ plain, long long head_stride, long long token_stride,
                         T* __restrict__ rotated, int quads) {
   extern __shared__ float row_s[];
+  if (WHOLE) slices = 1;
   const int t = blockIdx.x;
   const int per_block = (heads + gridDim.y - 1) / gridDim.y;
   const int h0 = blockIdx.y * per_block, count = min(heads, h0 + per_block) - h0;
@@ -486,16 +488,18 @@ extern "C" int distie_latent_q_prepare(const float* q, int row_stride, int slice
   const dim3 grid(tokens, tokens < 512 ? heads : 1);
   const int threads = tokens < 512 ? 128 : 256;
   const size_t shared = (size_t)rotary_dim * sizeof(float);
-  if (dtype == DISTIE_BF16)
-    latent_q_prepare_kernel<<<grid, threads, shared, stream>>>(q, row_stride, slices, slice_stride, heads, dim, rot_dim, positions,
-                                                               inv_freq, factor, rotary_dim, interleaved, (__nv_bfloat16*)plain,
-                                                               head_stride, token_stride, (__nv_bfloat16*)rotated, quads);
-  else if (dtype == DISTIE_F32)
-    latent_q_prepare_kernel<<<grid, threads, shared, stream>>>(q, row_stride, slices, slice_stride, heads, dim, rot_dim, positions,
-                                                               inv_freq, factor, rotary_dim, interleaved, (float*)plain, head_stride,
-                                                               token_stride, (float*)rotated, quads);
-  else
+#define DISTIE_Q_PREPARE(T, WHOLEV)                                                                                          \
+  latent_q_prepare_kernel<T, WHOLEV><<<grid, threads, shared, stream>>>(q, row_stride, slices, slice_stride, heads, dim, rot_dim, \
+                                                                        positions, inv_freq, factor, rotary_dim, interleaved,    \
+                                                                        (T*)plain, head_stride, token_stride, (T*)rotated, quads)
+  if (dtype == DISTIE_BF16) {
+    if (slices == 1) DISTIE_Q_PREPARE(__nv_bfloat16, true); else DISTIE_Q_PREPARE(__nv_bfloat16, false);
+  } else if (dtype == DISTIE_F32) {
+    if (slices == 1) DISTIE_Q_PREPARE(float, true); else DISTIE_Q_PREPARE(float, false);
+  } else {
     return DISTIE_ERR_UNSUPPORTED;
+  }
+#undef DISTIE_Q_PREPARE
   DISTIE_LAUNCH_CHECK();
   return 0;
 }

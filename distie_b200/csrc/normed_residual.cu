@@ -131,7 +131,8 @@ norm_add_rmsnorm_vec_kernel(ResidualTerms terms, const float* __restrict__ delta
 // measured, so the elements are spread over the machine whatever the rows are: four a thread (VEC: hidden a multiple of
 // 4, every pointer aligned to four elements) or one.  With a list of rows only those are made and the residual stays.
 // Launched as a dependent kernel: weight and bias are on their way before the producer of the terms has finished.
-template <typename T, bool VEC>
+// MANY: more than two terms, whose loads are in flight together.
+template <typename T, bool VEC, bool MANY>
 __global__ void __launch_bounds__(256)
 add_dynamic_tanh_kernel(ResidualTerms terms, float* residual, float alpha, const float* __restrict__ weight,
                         const float* __restrict__ bias, T* out, const int* rows_index, int hidden, long long units) {
@@ -150,8 +151,15 @@ add_dynamic_tanh_kernel(ResidualTerms terms, float* residual, float alpha, const
     float4 r = load4_cg(residual + at);
     if (terms.count > 0) {
       float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!MANY) {
+        for (int j = 0; j < terms.count; ++j) {
+          const float4 v = load4_cg(terms.ptr[j] + at);
+          const float s = terms.scale[j];
+          d.x += s * v.x; d.y += s * v.y; d.z += s * v.z; d.w += s * v.w;
+        }
+      }
 #pragma unroll
-      for (int j0 = 0; j0 < kResidualTerms; j0 += 12) {  // up to twelve terms in flight together
+      for (int j0 = 0; MANY && j0 < kResidualTerms; j0 += 12) {
         if (j0 >= terms.count) break;
         float4 v[12];
 #pragma unroll
@@ -541,8 +549,10 @@ extern "C" int distie_add_dynamic_tanh(const float* const* term_ptrs, const floa
   if (blocks > 0x7fffffffLL) return DISTIE_ERR_UNSUPPORTED;
   cudaError_t err;
 #define DISTIE_DYNAMIC_TANH(T, VECV)                                                                                        \
-  err = launch_dependent(add_dynamic_tanh_kernel<T, VECV>, dim3((unsigned)blocks), dim3(threads), 0, stream, terms, residual, \
-                         alpha, weight, bias, (T*)out, rows_index, hidden, units)
+  err = num_terms > 2 ? launch_dependent(add_dynamic_tanh_kernel<T, VECV, true>, dim3((unsigned)blocks), dim3(threads), 0, stream, \
+                                         terms, residual, alpha, weight, bias, (T*)out, rows_index, hidden, units)          \
+                      : launch_dependent(add_dynamic_tanh_kernel<T, VECV, false>, dim3((unsigned)blocks), dim3(threads), 0, stream, \
+                                         terms, residual, alpha, weight, bias, (T*)out, rows_index, hidden, units)
   if (dtype == DISTIE_BF16) {
     if (vec) DISTIE_DYNAMIC_TANH(__nv_bfloat16, true); else DISTIE_DYNAMIC_TANH(__nv_bfloat16, false);
   } else {

@@ -24,7 +24,8 @@
 namespace distie {
 
 constexpr int kChunk = 64;
-constexpr int kChunkThreads = 512;   // 16 warps: four groups of 16 rows by four groups of columns
+constexpr int kReadThreads = 512;    // 16 warps: four groups of 16 rows by four groups of columns
+constexpr int kWriteThreads = 256;   // (three blocks an SM)
 
 struct RetentionArgs {
   Sliced qkv;                 // [tokens, heads * (2 * key_dim) + heads * value_dim]
@@ -116,7 +117,7 @@ __device__ __forceinline__ float4 four_of(const Sliced& x, size_t t, int col) {
 
 // Rows t0 .. t0 + rows - 1 of one head's q or k (columns from `column`), rotated and times `scale`, into kChunk rows of
 // `dst`; rows past the chunk and columns key_dim .. up16(key_dim) - 1 become zeros.
-template <bool WHOLE>
+template <bool WHOLE, int kChunkThreads>
 __device__ __forceinline__ void load_rotated(const RetentionArgs& a, int t0, int rows, int column, float scale, const Parts& dst) {
   const int half = a.trig ? a.rotary_dim / 2 : 0, rot = 2 * half;
   const int key_dim = a.key_dim, padded = up16(key_dim);
@@ -179,7 +180,7 @@ __device__ __forceinline__ void load_rotated(const RetentionArgs& a, int t0, int
 
 // One head's v of the chunk into kChunk rows of `dst`, row r times weight_s[r] where weights are given; zeros in rows past
 // the chunk and in columns value_dim .. up16(value_dim) - 1.
-template <bool WHOLE>
+template <bool WHOLE, int kChunkThreads>
 __device__ __forceinline__ void load_values(const RetentionArgs& a, int t0, int rows, int column, const float* weight_s, const Parts& dst) {
   const int value_dim = a.value_dim, padded = up16(value_dim);
   const bool quads = (value_dim & 3) == 0 && (a.qkv.stride & 3) == 0 && (column & 3) == 0 && (a.qkv.split_stride & 3) == 0 &&
@@ -212,7 +213,7 @@ __device__ __forceinline__ int chunk_rows(const int* q_tiles, int chunk, int& t0
 
 // U^T [value_dim, key_dim] of a chunk: rows are value elements (V^T is the first operand), columns key elements.
 template <bool WHOLE>
-__global__ void __launch_bounds__(kChunkThreads) retention_chunk_write_kernel(RetentionArgs a) {
+__global__ void __launch_bounds__(kWriteThreads, 3) retention_chunk_write_kernel(RetentionArgs a) {
   extern __shared__ __align__(16) unsigned char chunk_s[];
   __shared__ float weight_s[kChunk];
   int t0;
@@ -223,8 +224,8 @@ __global__ void __launch_bounds__(kChunkThreads) retention_chunk_write_kernel(Re
   const int qk = a.heads * a.key_dim;
   if (threadIdx.x < kChunk) weight_s[threadIdx.x] = threadIdx.x < rows ? power_of(a.decay[head], rows - 1 - threadIdx.x) : 0.f;
   __syncthreads();
-  load_rotated<WHOLE>(a, t0, rows, qk + head * a.key_dim, a.key_scale, k);
-  load_values<WHOLE>(a, t0, rows, 2 * qk + head * a.value_dim, weight_s, v);
+  load_rotated<WHOLE, kWriteThreads>(a, t0, rows, qk + head * a.key_dim, a.key_scale, k);
+  load_values<WHOLE, kWriteThreads>(a, t0, rows, 2 * qk + head * a.value_dim, weight_s, v);
   __syncthreads();
 
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
@@ -234,7 +235,7 @@ __global__ void __launch_bounds__(kChunkThreads) retention_chunk_write_kernel(Re
   const int steps = (rows + 15) / 16;
   const int v_row = (lane & 7) + (lane >> 4) * 8, v_col = ((lane >> 3) & 1) * 8;  // what a lane names of V^T's 16 x 16 piece
   const int k_row = (lane & 7) + ((lane >> 3) & 1) * 8, k_col = (lane >> 4) * 8;  // and of K's
-  for (int unit = warp; unit < units; unit += kChunkThreads / 32) {
+  for (int unit = warp; unit < units; unit += kWriteThreads / 32) {
     const int m0 = (unit % m_tiles) * 16, n0 = (unit / m_tiles) * 32;
     float acc[4][4] = {};
     for (int s = 0; s < steps; ++s) {
@@ -276,8 +277,15 @@ __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float x, float y) {
   *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x, y);
 }
 
-// The chain from chunk to chunk of every request: a thread owns W neighbouring elements of one head's state.  A block
-// whose tile is not the first of its request has nothing to do.
+// 8 bytes into shared memory, asynchronously; zeros when not live.
+__device__ __forceinline__ void copy_8(__nv_bfloat16* dst, const float* src, bool live) {
+  const int bytes = live ? 8 : 0;
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes) : "memory");
+}
+
+// The chain from chunk to chunk of every request: a thread owns W neighbouring elements of one head's state.  What it
+// leaves for chunk_read is the state before the chunk in its two bfloat16 parts, in the bytes that held the chunk's U:
+// the W high parts, then the W low parts.  A block whose tile is not the first of its request has nothing to do.
 constexpr int kChainThreads = 256;
 template <int W>
 __global__ void __launch_bounds__(kChainThreads) retention_chunk_chain_kernel(RetentionArgs a) {
@@ -302,6 +310,18 @@ __global__ void __launch_bounds__(kChainThreads) retention_chunk_chain_kernel(Re
     if (W == 4) *reinterpret_cast<float4*>(p) = make_float4(x.v[0], x.v[W > 1 ? 1 : 0], x.v[W > 2 ? 2 : 0], x.v[W > 3 ? 3 : 0]);
     else *p = x.v[0];
   };
+  auto store_parts = [](float* p, const Piece& x) {
+    if (W == 4) {
+      const __nv_bfloat162 h0 = __floats2bfloat162_rn(x.v[0], x.v[W > 1 ? 1 : 0]), h1 = __floats2bfloat162_rn(x.v[W > 2 ? 2 : 0], x.v[W > 3 ? 3 : 0]);
+      const __nv_bfloat162 l0 = __floats2bfloat162_rn(x.v[0] - __low2float(h0), x.v[W > 1 ? 1 : 0] - __high2float(h0));
+      const __nv_bfloat162 l1 = __floats2bfloat162_rn(x.v[W > 2 ? 2 : 0] - __low2float(h1), x.v[W > 3 ? 3 : 0] - __high2float(h1));
+      *reinterpret_cast<uint4*>(p) = make_uint4(*reinterpret_cast<const uint32_t*>(&h0), *reinterpret_cast<const uint32_t*>(&h1),
+                                                *reinterpret_cast<const uint32_t*>(&l0), *reinterpret_cast<const uint32_t*>(&l1));
+    } else {
+      const __nv_bfloat16 h = __float2bfloat16_rn(x.v[0]), l = __float2bfloat16_rn(x.v[0] - __bfloat162float(h));
+      *reinterpret_cast<uint32_t*>(p) = (uint32_t)__bfloat16_as_ushort(h) | ((uint32_t)__bfloat16_as_ushort(l) << 16);
+    }
+  };
   const float decay = a.decay[head], whole = power_of(decay, kChunk);
   float* slot = a.state + ((size_t)a.seq_seat[seq] * a.heads + head) * size + at;
   Piece S = load(slot);
@@ -324,7 +344,7 @@ __global__ void __launch_bounds__(kChainThreads) retention_chunk_chain_kernel(Re
     for (int j = 0; j < 2 * kAhead; ++j) {
       const int n = min(kChunk, rows[j >> 1] - (j & 1) * kChunk);
       if (n > 0) {
-        store(mine + (size_t)(2 * tile + j) * stride, S);
+        store_parts(mine + (size_t)(2 * tile + j) * stride, S);
         const float factor = n == kChunk ? whole : power_of(decay, n);
 #pragma unroll
         for (int e = 0; e < W; ++e) S.v[e] = factor * S.v[e] + u[j].v[e];
@@ -337,7 +357,7 @@ __global__ void __launch_bounds__(kChainThreads) retention_chunk_chain_kernel(Re
 
 // O of a chunk from its own tokens and the state before it, normed per head and gated.
 template <typename T, bool WHOLE>
-__global__ void __launch_bounds__(kChunkThreads, 1)
+__global__ void __launch_bounds__(kReadThreads, 1)
 retention_chunk_read_kernel(RetentionArgs a, Sliced gate, int gate_sigmoid, float eps, T* __restrict__ out, int out_stride) {
   extern __shared__ __align__(16) unsigned char chunk_s[];
   __shared__ float power_s[kChunk + 1], square_s[4][kChunk];
@@ -356,23 +376,30 @@ retention_chunk_read_kernel(RetentionArgs a, Sliced gate, int gate_sigmoid, floa
   const int v0 = cq * 32;                    // the warp's value elements
 
   if (threadIdx.x <= kChunk) power_s[threadIdx.x] = power_of(a.decay[head], threadIdx.x);
+  // The state comes in its two parts already: four elements' high parts, then their low parts, in 16 bytes (or one element's
+  // in 4): it is copied while q, k and v are made.
   if ((a.key_dim & 3) == 0) {
-    const int per_row = key_padded / 4, e = 4 * (threadIdx.x % per_row), r_step = kChunkThreads / per_row;
+    const int per_row = key_padded / 4, e = 4 * (threadIdx.x % per_row), r_step = kReadThreads / per_row;
     const int r_first = threadIdx.x / per_row, r_end = r_first < r_step ? value_padded : 0;
-#pragma unroll 8
     for (int r = r_first; r < r_end; r += r_step) {
       const bool live = r < a.value_dim && e < a.key_dim;
-      S.put4(r, e, live ? *reinterpret_cast<const float4*>(before + (size_t)r * a.key_dim + e) : make_float4(0.f, 0.f, 0.f, 0.f));
+      const float* src = before + (live ? (size_t)r * a.key_dim + e : 0);
+      copy_8(S.high + r * S.ld + e, src, live);
+      copy_8(S.low + r * S.ld + e, src + 2, live);
     }
   } else {
-    for (int idx = threadIdx.x; idx < value_padded * key_padded; idx += kChunkThreads) {
+    for (int idx = threadIdx.x; idx < value_padded * key_padded; idx += kReadThreads) {
       const int r = idx / key_padded, e = idx % key_padded;
-      S.put(r, e, r < a.value_dim && e < a.key_dim ? before[(size_t)r * a.key_dim + e] : 0.f);
+      uint32_t both = 0u;
+      if (r < a.value_dim && e < a.key_dim) both = __float_as_uint(before[(size_t)r * a.key_dim + e]);
+      S.high[r * S.ld + e] = __ushort_as_bfloat16((unsigned short)(both & 0xffffu));
+      S.low[r * S.ld + e] = __ushort_as_bfloat16((unsigned short)(both >> 16));
     }
   }
-  load_rotated<WHOLE>(a, t0, rows, head * a.key_dim, 1.f, q);
-  load_rotated<WHOLE>(a, t0, rows, qk + head * a.key_dim, a.key_scale, k);
-  load_values<WHOLE>(a, t0, rows, 2 * qk + head * a.value_dim, nullptr, v);
+  cp_async_commit();
+  load_rotated<WHOLE, kReadThreads>(a, t0, rows, head * a.key_dim, 1.f, q);
+  load_rotated<WHOLE, kReadThreads>(a, t0, rows, qk + head * a.key_dim, a.key_scale, k);
+  load_values<WHOLE, kReadThreads>(a, t0, rows, 2 * qk + head * a.value_dim, nullptr, v);
   float z[4][4];  // the gate's inputs of what this thread will store, on their way during the products
 #pragma unroll
   for (int j = 0; j < 4; ++j)
@@ -383,6 +410,7 @@ retention_chunk_read_kernel(RetentionArgs a, Sliced gate, int gate_sigmoid, floa
       if (row < rows && col < a.value_dim)
         z[j][r] = WHOLE ? gate.p[(size_t)(t0 + row) * gate.stride + head * a.value_dim + col] : gate.at(t0 + row, head * a.value_dim + col);
     }
+  cp_async_wait<0>();
   __syncthreads();
 
   const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;  // what a lane names of a 16 x 16 piece of a
@@ -674,24 +702,24 @@ extern "C" int distie_retention_chunks(const float* qkv, int qkv_stride, int spl
   const size_t write_shared = parts_bytes(kChunk, key_dim) + parts_bytes(kChunk, value_dim);
   const size_t read_shared = 2 * parts_bytes(kChunk, key_dim) + parts_bytes(kChunk, value_dim) +
                              parts_bytes(up16(value_dim), key_dim) + parts_bytes(kChunk, kChunk);
-  auto launch = [&](auto kernel, size_t shared, auto... args) -> int {
+  auto launch = [&](auto kernel, int threads, size_t shared, auto... args) -> int {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     if (err != cudaSuccess) return (int)err;
-    kernel<<<grid, kChunkThreads, shared, stream>>>(args...);
+    kernel<<<grid, threads, shared, stream>>>(args...);
     return (int)cudaGetLastError();
   };
   const bool whole = splits == 1 && gate_splits == 1;
-  int status = whole ? launch(retention_chunk_write_kernel<true>, write_shared, a)
-                     : launch(retention_chunk_write_kernel<false>, write_shared, a);
+  int status = whole ? launch(retention_chunk_write_kernel<true>, kWriteThreads, write_shared, a)
+                     : launch(retention_chunk_write_kernel<false>, kWriteThreads, write_shared, a);
   if (status != 0) return status;
   const int size = key_dim * value_dim;
-  if (size % 4 == 0)
+  if (key_dim % 4 == 0)  // (groups of four lie in one row: the layout in which chunk_read takes them)
     retention_chunk_chain_kernel<4><<<dim3((size / 4 + kChainThreads - 1) / kChainThreads, heads, tiles), kChainThreads, 0, stream>>>(a);
   else
     retention_chunk_chain_kernel<1><<<dim3((size + kChainThreads - 1) / kChainThreads, heads, tiles), kChainThreads, 0, stream>>>(a);
   DISTIE_LAUNCH_CHECK();
 #define DISTIE_CHUNK_READ(T, WHOLEV) \
-  launch(retention_chunk_read_kernel<T, WHOLEV>, read_shared, a, gates, gate_sigmoid, eps, (T*)out, out_stride)
+  launch(retention_chunk_read_kernel<T, WHOLEV>, kReadThreads, read_shared, a, gates, gate_sigmoid, eps, (T*)out, out_stride)
   if (dtype == DISTIE_BF16) return whole ? DISTIE_CHUNK_READ(__nv_bfloat16, true) : DISTIE_CHUNK_READ(__nv_bfloat16, false);
   return whole ? DISTIE_CHUNK_READ(float, true) : DISTIE_CHUNK_READ(float, false);
 #undef DISTIE_CHUNK_READ
