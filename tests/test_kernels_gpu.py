@@ -373,7 +373,7 @@ def test_attention_mixed_batch(kernel_sets, dtype, heads, kv_heads, head_dim, pa
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize(
     "heads,kv_heads,head_dim,value_dim,page,window,chunk,keep_first,softcap,sink",
-    [(4, 4, 96, 32, 16, None, None, 0, 0.0, True), (6, 1, 64, 32, 16, None, None, 0, 0.0, False), (6, 3, 80, 48, 8, 37, None, 0, 0.0, True),
+    [(6, 6, 88, 40, 16, None, None, 0, 0.0, True), (6, 1, 64, 32, 16, None, None, 0, 0.0, False), (6, 3, 80, 48, 8, 37, None, 0, 0.0, True),
      (8, 2, 128, 64, 16, 100, None, 5, 0.0, False), (2, 2, 32, 96, 16, None, 50, 0, 0.0, False), (20, 1, 64, 128, 32, None, None, 0, 2.5, True),
      (18, 2, 96, 96, 16, 64, None, 17, 0.0, False), (3, 1, 112, 120, 4, 9, None, 2, 1.5, True), (5, 5, 40, 8, 16, None, 128, 0, 0.0, True),
      (1, 1, 8, 128, 64, 130, None, 0, 0.0, False), (10, 2, 48, 48, 128, None, None, 0, 0.0, False),
